@@ -77,6 +77,26 @@ class ModelConfig(C.Structure):
             "max_draft_tokens", "draft_vocab")]
 
 
+MIXER_LATENT_ATTENTION = 1
+MLP_NONE, MLP_RELU2 = 0, 1
+
+
+class LayerConfig(C.Structure):
+    """ctox_layer_config (include/ctox_b200.h)."""
+
+    _fields_ = [("rope_base", C.c_double)] + [(n, C.c_uint32) for n in (
+        "mixer", "heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "window")] + [
+        ("kv_from", C.c_int32), ("score_scale", C.c_float), ("mlp", C.c_uint32), ("ff", C.c_uint32)]
+
+
+class StackConfigC(C.Structure):
+    """ctox_stack_config (include/ctox_b200.h)."""
+
+    _fields_ = [("vocab_size", C.c_uint32), ("hidden_size", C.c_uint32), ("num_layers", C.c_uint32),
+                ("norm_eps", C.c_float), ("logit_softcap", C.c_float)] + [(n, C.c_uint32) for n in (
+                    "max_context_tokens", "kv_page_tokens", "kv_dtype", "pass_tokens")]
+
+
 class ExecStep(C.Structure):
     """ctox_exec_step (include/ctox_b200.h)."""
 
@@ -93,7 +113,8 @@ class ExecStep(C.Structure):
 
 (T_EMBED, T_LM_HEAD, T_FINAL_NORM, T_INPUT_NORM, T_POST_NORM, T_ATTN_QKV, T_ATTN_O, T_Q_NORM, T_K_NORM,
  T_LIN_IN, T_LIN_OUT, T_CONV_W, T_A_LOG, T_DT_BIAS, T_LIN_NORM, T_MLP_GATE_UP, T_MLP_DOWN, T_MTP_FC,
- T_MTP_NORM_E, T_MTP_NORM_H, T_MTP_NORM, T_DRAFT_IDS) = range(22)
+ T_MTP_NORM_E, T_MTP_NORM_H, T_MTP_NORM, T_DRAFT_IDS, T_Q_DOWN, T_Q_DOWN_NORM, T_Q_UP, T_KV_DOWN, T_KV_DOWN_NORM,
+ T_K_UP, T_V_UP, T_MIX_OUT_NORM, T_MLP_UP, T_MLP_OUT_NORM) = range(32)
 LAYER_GLOBAL = 0xFFFFFFFF
 
 
@@ -179,6 +200,12 @@ SIGNATURES = {
                                        C.c_uint64, C.c_uint64, C.c_uint32, C.c_void_p,
                                        C.POINTER(SpecRecord)]),
     "ctox_exec_create": (C.c_int32, [C.c_void_p, C.POINTER(ModelConfig), C.POINTER(C.c_void_p)]),
+    "ctox_exec_create_stack": (C.c_int32, [C.c_void_p, C.POINTER(StackConfigC), C.POINTER(LayerConfig),
+                                           C.POINTER(C.c_void_p)]),
+    "ctox_exec_extend": (C.c_int32, [C.c_void_p, C.c_void_p, C.c_uint64, C.c_void_p, C.c_uint64, C.c_void_p,
+                                     C.c_void_p]),
+    "ctox_exec_keep_streams": (C.c_int32, [C.c_void_p]),
+    "ctox_exec_last_stream": (C.c_int32, [C.c_void_p, C.c_uint32, C.c_uint64, C.c_uint64, C.c_void_p]),
     "ctox_exec_destroy": (C.c_int32, [C.c_void_p]),
     "ctox_exec_load_matrix": (C.c_int32, [C.c_void_p, C.c_uint32, C.c_uint32, C.POINTER(FusedMatVecOp)]),
     "ctox_exec_load_vector": (C.c_int32, [C.c_void_p, C.c_uint32, C.c_uint32, C.c_void_p, C.c_uint64]),

@@ -1,0 +1,513 @@
+// Matrix-vector products with dense bf16 weights for short passes, the norms of longer passes, and
+// the small kernels that go with them (embedding rows, weight layout).
+#include "dense.cuh"
+
+#include <map>
+#include <mutex>
+#include <tuple>
+
+namespace ctox {
+
+constexpr int kDvThreads = 256, kDvWarps = kDvThreads / 32;
+
+// Sum over the kDvThreads / M threads of a position (whole warps); every thread of the CTA calls it.
+template <int M>
+__device__ __forceinline__ float position_sum(float v, float *red) {
+    constexpr int W = kDvWarps / M;  // warps per position
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    if (W == 1) return v;
+    const int warp = threadIdx.x >> 5;
+    __syncthreads();
+    if ((threadIdx.x & 31) == 0) red[warp] = v;
+    __syncthreads();
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < W; ++i) s += red[warp / W * W + i];
+    return s;
+}
+
+__device__ void latent_append_row(const LatentAppend &a, uint32_t m, uint32_t tid, uint32_t nthreads, float *red) {
+    const float *row = a.fan + (size_t)m * a.fan_stride + a.fan_off;
+    float sq = 0.f;
+    for (uint32_t c = tid; c < a.kv_rank; c += nthreads) sq += row[c] * row[c];
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    __syncthreads();
+    if ((tid & 31) == 0) red[tid >> 5] = sq;
+    __syncthreads();
+    float total = 0.f;
+    for (uint32_t w = 0; w < nthreads / 32; ++w) total += red[w];
+    const float inv = 1.0f / sqrtf(total / (float)a.kv_rank + a.eps);
+    const uint32_t pos = a.pos0 + m;
+    const size_t base = paged_slot(a.page_table, a.page_tokens, pos) * (a.kv_pad + a.rot_pad);
+    auto store = [&](uint32_t c, float v) {
+        if (a.bf16)
+            ((__nv_bfloat16 *)a.cache)[base + c] = __float2bfloat16_rn(v);
+        else
+            ((float *)a.cache)[base + c] = v;
+    };
+    for (uint32_t c = tid; c < a.kv_pad; c += nthreads) store(c, c < a.kv_rank ? row[c] * inv * a.norm_w[c] : 0.f);
+    for (uint32_t i = tid; i < a.rot_pad / 2; i += nthreads) {
+        float u = 0.f, v = 0.f;
+        if (2 * i < a.rot_dim) {
+            u = row[a.kv_rank + 2 * i];
+            v = row[a.kv_rank + 2 * i + 1];
+            rope_pair(u, v, (float)pos * a.freq[i]);
+        }
+        store(a.kv_pad + 2 * i, u);
+        store(a.kv_pad + 2 * i + 1, v);
+    }
+}
+
+// One warp group of 2^lpr_log2 lanes per R rows, `ks` warps side by side on the columns of the same
+// rows. The activations sit in shared memory in the order the lanes read them: blocks of LPR * 8
+// columns as [half][lane][4]. The first weights of every warp are requested before the dependency
+// wait (they are constants), so they arrive while the prologue forms the input.
+template <int M, int R>
+__global__ void __launch_bounds__(kDvThreads, 2)
+    k_dense_matvec(const __nv_bfloat16 *__restrict__ W, uint32_t ld, uint32_t rows_per_group, uint32_t units_per_group,
+                   uint32_t units, uint32_t ks, uint32_t lpr_log2, uint32_t npos, VecIn in, VecOut out,
+                   LatentAppend ap, uint32_t append_positions) {
+    pdl_launch();
+    extern __shared__ __align__(16) float xs[];  // [M][ldx]
+    __shared__ float red[kDvWarps];
+    __shared__ float part[kDvWarps][32 * 4];  // partial sums of the column parts: [warp][subgroup rows x positions]
+    __shared__ float mw[M][kAttnSplitsDense];
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const uint32_t grid = gridDim.x - append_positions;
+    if (blockIdx.x >= grid) {
+        pdl_wait();
+        latent_append_row(ap, blockIdx.x - grid, tid, kDvThreads, red);
+        return;
+    }
+    const uint32_t lpr = 1u << lpr_log2, sub = lane >> lpr_log2, l = lane & (lpr - 1), nsub = 32u >> lpr_log2;
+    const uint32_t span = lpr * 8;                       // columns per step
+    const uint32_t nsteps = (ld + span - 1) / span, ldx = nsteps * span;
+    const uint32_t kp = warp % ks, rg = warp / ks;       // column part, row group of this warp
+    const uint32_t unit_rows = kDvWarps / ks * nsub * R;
+    const uint32_t cnt = kp < nsteps ? (nsteps - kp + ks - 1) / ks : 0;
+    constexpr int D = 8 / R;  // steps in flight
+    uint4 buf[D][R];
+    auto row_of = [&](uint32_t unit) { return (unit % units_per_group) * unit_rows + (rg * nsub + sub) * R; };
+    auto fetch = [&](const __nv_bfloat16 *base, uint32_t row0, uint32_t i, uint4 *dst) {
+        const uint32_t c = (kp + i * ks) * span + l * 8;
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            dst[r] = make_uint4(0, 0, 0, 0);
+            if (i < cnt && c < ld && row0 + r < rows_per_group)
+                dst[r] = __ldg(reinterpret_cast<const uint4 *>(base + (size_t)(row0 + r) * ld + c));
+        }
+    };
+    // ---- the input of `group`, normalised, into xs
+    auto stage = [&](uint32_t group) {
+        constexpr uint32_t T = kDvThreads / M;
+        const uint32_t m = tid / T, t = tid % T;
+        const bool live = m < npos;
+        float *xm = xs + m * ldx;
+        auto at = [&](uint32_t c) { return c / span * span + ((c >> 2) & 1) * (lpr * 4) + (c % span) / 8 * 4 + (c & 3); };
+        const uint32_t cols = in.cols;
+        if (in.ws_o) {
+            const size_t row = (size_t)m * in.groups + group;
+            if (live) {
+                float mx = -INFINITY;
+                for (uint32_t s = 0; s < in.splits; ++s) mx = fmaxf(mx, in.ws_ml[((size_t)s * in.ws_rows + row) * 2]);
+                float den = 0.f;
+                for (uint32_t s = 0; s < in.splits; ++s) {
+                    const float *ml = in.ws_ml + ((size_t)s * in.ws_rows + row) * 2;
+                    den += ml[1] * expf(ml[0] - mx);
+                }
+                for (uint32_t s = t; s < in.splits; s += T)
+                    mw[m][s] = expf(in.ws_ml[((size_t)s * in.ws_rows + row) * 2] - mx) / den;
+            }
+            __syncthreads();
+            for (uint32_t c = t; c < ldx; c += T) {
+                float v = 0.f;
+                if (live && c < cols)
+                    for (uint32_t s = 0; s < in.splits; ++s)
+                        v += mw[m][s] * in.ws_o[((size_t)s * in.ws_rows + row) * cols + c];
+                xm[at(c)] = v;
+            }
+            return;
+        }
+        const float *x = in.x + (size_t)m * in.x_stride + (size_t)group * in.x_group;
+        if (in.norm == NORM_NONE) {
+            for (uint32_t c = t; c < ldx; c += T) xm[at(c)] = live && c < cols ? x[c] : 0.f;
+            return;
+        }
+        float s = 0.f;
+        if (in.norm == NORM_RMS) {
+            for (uint32_t c = t; c < ldx; c += T) {
+                const float v = live && c < cols ? x[c] : 0.f;
+                xm[at(c)] = v;
+                s += v * v;
+            }
+            const float inv = 1.0f / sqrtf(position_sum<M>(s, red) / (float)cols + in.eps);
+            for (uint32_t c = t; c < cols; c += T) xm[at(c)] *= inv * in.w[c];
+            return;
+        }
+        const float n = (float)cols;
+        float mean = 0.f, inv = 0.f;
+        if (in.y) {
+            const float *y = in.y + (size_t)m * in.y_stride;
+            for (uint32_t c = t; c < cols; c += T) {
+                const float v = live ? y[c] : 0.f;
+                xm[at(c)] = v;
+                s += v;
+            }
+            mean = position_sum<M>(s, red) / n;
+            s = 0.f;
+            for (uint32_t c = t; c < cols; c += T) {
+                const float d = xm[at(c)] - mean;
+                s += d * d;
+            }
+            inv = 1.0f / sqrtf(position_sum<M>(s, red) / n + in.eps);
+        }
+        s = 0.f;
+        for (uint32_t c = t; c < ldx; c += T) {
+            float v = 0.f;
+            if (live && c < cols) {
+                v = x[c];
+                if (in.y) {
+                    v += (xm[at(c)] - mean) * inv * in.wb[c];
+                    if (blockIdx.x == 0) in.x_out[(size_t)m * in.x_stride + c] = v;
+                }
+            }
+            xm[at(c)] = v;
+            s += v;
+        }
+        mean = position_sum<M>(s, red) / n;
+        s = 0.f;
+        for (uint32_t c = t; c < cols; c += T) {
+            const float d = xm[at(c)] - mean;
+            s += d * d;
+        }
+        inv = 1.0f / sqrtf(position_sum<M>(s, red) / n + in.eps);
+        for (uint32_t c = t; c < cols; c += T) xm[at(c)] = (xm[at(c)] - mean) * inv * in.w[c];
+    };
+
+    uint32_t staged = 0xffffffffu;
+    for (uint32_t unit = blockIdx.x; unit < units; unit += grid) {
+        const uint32_t group = unit / units_per_group, row0 = row_of(unit);
+        const __nv_bfloat16 *base = W + (size_t)group * rows_per_group * ld;
+#pragma unroll
+        for (int d = 0; d < D; ++d) fetch(base, row0, d, buf[d]);
+        if (group != staged) {
+            if (staged == 0xffffffffu)
+                pdl_wait();
+            else
+                __syncthreads();
+            stage(group);
+            __syncthreads();
+            staged = group;
+        }
+        float acc[M][R];
+#pragma unroll
+        for (int m = 0; m < M; ++m)
+#pragma unroll
+            for (int r = 0; r < R; ++r) acc[m][r] = 0.f;
+        for (uint32_t i0 = 0; i0 < cnt; i0 += D) {
+#pragma unroll
+            for (int d = 0; d < D; ++d) {
+                uint4 w[R];
+#pragma unroll
+                for (int r = 0; r < R; ++r) w[r] = buf[d][r];
+                fetch(base, row0, i0 + d + D, buf[d]);
+                if (i0 + d < cnt) {
+                    const float *xp = xs + (kp + (i0 + d) * ks) * span + l * 4;
+#pragma unroll
+                    for (int m = 0; m < M; ++m) {
+                        const float4 a = *reinterpret_cast<const float4 *>(xp + m * ldx);
+                        const float4 b = *reinterpret_cast<const float4 *>(xp + m * ldx + lpr * 4);
+#pragma unroll
+                        for (int r = 0; r < R; ++r) {
+                            float s = acc[m][r];
+                            s = fmaf(__uint_as_float(w[r].x << 16), a.x, s);
+                            s = fmaf(__uint_as_float(w[r].x & 0xffff0000u), a.y, s);
+                            s = fmaf(__uint_as_float(w[r].y << 16), a.z, s);
+                            s = fmaf(__uint_as_float(w[r].y & 0xffff0000u), a.w, s);
+                            s = fmaf(__uint_as_float(w[r].z << 16), b.x, s);
+                            s = fmaf(__uint_as_float(w[r].z & 0xffff0000u), b.y, s);
+                            s = fmaf(__uint_as_float(w[r].w << 16), b.z, s);
+                            s = fmaf(__uint_as_float(w[r].w & 0xffff0000u), b.w, s);
+                            acc[m][r] = s;
+                        }
+                    }
+                }
+            }
+        }
+#pragma unroll
+        for (int m = 0; m < M; ++m)
+#pragma unroll
+            for (int r = 0; r < R; ++r)
+                for (uint32_t o = lpr >> 1; o > 0; o >>= 1) acc[m][r] += __shfl_xor_sync(0xffffffffu, acc[m][r], o);
+        if (ks > 1) {  // add the column parts of the rows up (part order), in the first of their warps
+            __syncthreads();
+            if (l == 0)
+#pragma unroll
+                for (int m = 0; m < M; ++m)
+#pragma unroll
+                    for (int r = 0; r < R; ++r) part[warp][sub * (M * R) + m * R + r] = acc[m][r];
+            __syncthreads();
+            if (kp == 0) {
+                for (uint32_t q = 1; q < ks; ++q)
+#pragma unroll
+                    for (int m = 0; m < M; ++m)
+#pragma unroll
+                        for (int r = 0; r < R; ++r) acc[m][r] += part[warp + q][sub * (M * R) + m * R + r];
+            }
+        }
+        if (kp == 0) {
+            for (uint32_t k = l; k < (uint32_t)(M * R); k += lpr) {
+                float v = 0.f, pair = 0.f;
+#pragma unroll
+                for (int m = 0; m < M; ++m)
+#pragma unroll
+                    for (int r = 0; r < R; ++r) {
+                        if (k == (uint32_t)(m * R + r)) v = acc[m][r];
+                        if ((k ^ 1u) == (uint32_t)(m * R + r)) pair = acc[m][r];
+                    }
+                const uint32_t m = k / R, row = row0 + k % R;
+                if (m >= npos || row >= rows_per_group) continue;
+                if (out.kind == OUT_RELU2) {
+                    v = v > 0.f ? v * v : 0.f;
+                } else if (out.kind == OUT_SOFTCAP) {
+                    v = out.cap * tanhf(v / out.cap);
+                } else if (out.kind == OUT_ROPE) {
+                    const uint32_t w = row % out.head_width;
+                    if (w >= out.rope0 && w < out.rope0 + out.rope_dims) {
+                        const float angle = (float)(out.pos0 + m) * out.freq[(w - out.rope0) >> 1];
+                        float a = (w & 1) ? pair : v, b = (w & 1) ? v : pair;
+                        rope_pair(a, b, angle);
+                        v = (w & 1) ? b : a;
+                    }
+                }
+                out.y[(size_t)m * out.y_stride + (size_t)group * rows_per_group + row] = v;
+            }
+        }
+    }
+}
+
+namespace {
+
+template <int M, int R>
+ctox_status matvec_launch(ctox_ctx *ctx, const DenseMat &w, uint32_t groups, uint32_t m, const VecIn &in,
+                          const VecOut &out, const LatentAppend *append, uint32_t append_positions, size_t smem,
+                          uint32_t ks, uint32_t lpr_log2) {
+    static std::mutex mu;
+    static std::map<std::tuple<int, size_t>, int> resident;  // CTAs per SM by (device, shared memory)
+    int per_sm = 0;
+    {
+        std::lock_guard<std::mutex> lock(mu);
+        auto it = resident.find({ctx->device, smem});
+        if (it == resident.end()) {
+            CTOX_CUDA(ctx, cudaFuncSetAttribute(k_dense_matvec<M, R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                                ctx->max_smem_optin - 8192));
+            CTOX_CUDA(ctx, cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, k_dense_matvec<M, R>, kDvThreads, smem));
+            if (per_sm < 1) return fail(ctx, CTOX_MEMORY_BUDGET, "dense matvec: %zu bytes of shared memory", smem);
+            resident[{ctx->device, smem}] = per_sm;
+        } else {
+            per_sm = it->second;
+        }
+    }
+    const uint32_t rows_per_group = w.rows / groups, unit_rows = kDvWarps / ks * (32u >> lpr_log2) * R;
+    const uint32_t units_per_group = (rows_per_group + unit_rows - 1) / unit_rows, units = units_per_group * groups;
+    const uint32_t fit = (uint32_t)(per_sm * ctx->sm_count), waves = (units + fit - 1) / fit;
+    const uint32_t grid = (units + waves - 1) / waves;
+    const LatentAppend ap = append ? *append : LatentAppend{};
+    CTOX_CUDA(ctx, launch_pdl(k_dense_matvec<M, R>, dim3(grid + append_positions), dim3(kDvThreads), smem, ctx->stream,
+                              (const __nv_bfloat16 *)w.w, w.ld, rows_per_group, units_per_group, units, ks, lpr_log2, m,
+                              in, out, ap, append_positions));
+    return CTOX_OK;
+}
+
+}  // namespace
+
+ctox_status launch_dense_matvec(ctox_ctx *ctx, const DenseMat &w, uint32_t groups, uint32_t m, const VecIn &in,
+                                const VecOut &out, const LatentAppend *append) {
+    uint32_t lpr_log2 = 5;  // lanes per row: fewer for narrow matrices
+    while (lpr_log2 > 3 && w.ld <= (8u << (lpr_log2 - 1))) --lpr_log2;
+    const uint32_t span = 8u << lpr_log2, nsteps = (w.ld + span - 1) / span;
+    const size_t row_bytes = (size_t)nsteps * span * 4;
+    uint32_t M = m <= 1 ? 1 : m <= 2 ? 2 : m <= 4 ? 4 : 8;
+    while (M > 1 && M * row_bytes + 8192 > (size_t)ctx->max_smem_optin) M /= 2;
+    if (M * row_bytes + 8192 > (size_t)ctx->max_smem_optin)
+        return fail(ctx, CTOX_MEMORY_BUDGET, "dense matvec: %u columns do not fit shared memory", w.ld);
+    for (uint32_t p = 0; p < m; p += M) {
+        const uint32_t n = m - p < M ? m - p : M;
+        VecIn i = in;
+        VecOut o = out;
+        if (i.x) i.x += (size_t)p * i.x_stride;
+        if (i.y) i.y += (size_t)p * i.y_stride;
+        if (i.x_out) i.x_out += (size_t)p * i.x_stride;
+        if (i.ws_o) {
+            i.ws_o += (size_t)p * i.groups * i.cols;
+            i.ws_ml += (size_t)p * i.groups * 2;
+        }
+        o.y += (size_t)p * o.y_stride;
+        o.pos0 += p;
+        // enough warps to cover the machine: fewer rows per warp, then several warps per row
+        const uint32_t want = (uint32_t)ctx->sm_count * 16, nsub = 32u >> lpr_log2;
+        const uint32_t R = M <= 2 && w.rows / (4 * nsub) >= want ? 4 : 2;
+        uint32_t ks = 1;
+        while (ks < kDvWarps && w.rows / (R * nsub) * ks < want && nsteps / (2 * ks) >= 2) ks *= 2;
+        const uint32_t na = append && p == 0 ? m : 0;
+        const size_t smem = M * row_bytes;
+        ctox_status rc;
+#define DV(MM, RR) matvec_launch<MM, RR>(ctx, w, groups, n, i, o, append, na, smem, ks, lpr_log2)
+        if (M == 1)
+            rc = R == 4 ? DV(1, 4) : DV(1, 2);
+        else if (M == 2)
+            rc = R == 4 ? DV(2, 4) : DV(2, 2);
+        else if (M == 4)
+            rc = DV(4, 2);
+        else
+            rc = DV(8, 2);
+#undef DV
+        if (rc) return rc;
+    }
+    return CTOX_OK;
+}
+
+// ------------------------------------------------------------------ norms of the residual stream
+constexpr int kSnThreads = 256;
+
+__global__ void __launch_bounds__(kSnThreads) k_stream_norm(StreamNorm a) {
+    pdl_launch();
+    pdl_wait();
+    extern __shared__ float v_s[];  // [width]
+    __shared__ float red[kDvWarps];
+    const uint32_t row = a.rows ? a.rows[blockIdx.x] : blockIdx.x, tid = threadIdx.x;
+    const float n = (float)a.width;
+    const float *x = a.x + (size_t)row * a.width;
+    float s = 0.f, mean = 0.f, inv = 0.f;
+    if (a.y) {
+        const float *y = a.y + (size_t)row * a.width;
+        for (uint32_t c = tid; c < a.width; c += kSnThreads) {
+            const float v = y[c];
+            v_s[c] = v;
+            s += v;
+        }
+        mean = position_sum<1>(s, red) / n;
+        s = 0.f;
+        for (uint32_t c = tid; c < a.width; c += kSnThreads) s += (v_s[c] - mean) * (v_s[c] - mean);
+        inv = 1.0f / sqrtf(position_sum<1>(s, red) / n + a.eps);
+    }
+    s = 0.f;
+    for (uint32_t c = tid; c < a.width; c += kSnThreads) {
+        float v = x[c];
+        if (a.y) v += (v_s[c] - mean) * inv * a.wb[c];
+        if (a.x_out) a.x_out[(size_t)row * a.width + c] = v;
+        v_s[c] = v;
+        s += v;
+    }
+    if (!a.w) return;
+    mean = position_sum<1>(s, red) / n;
+    s = 0.f;
+    for (uint32_t c = tid; c < a.width; c += kSnThreads) s += (v_s[c] - mean) * (v_s[c] - mean);
+    inv = 1.0f / sqrtf(position_sum<1>(s, red) / n + a.eps);
+    for (uint32_t c = tid; c < a.width; c += kSnThreads) {
+        const float v = (v_s[c] - mean) * inv * a.w[c];
+        if (a.f32_out) a.f32_out[(size_t)blockIdx.x * a.width + c] = v;
+        if (a.bf16_out) a.bf16_out[(size_t)blockIdx.x * a.bf16_ld + c] = __float2bfloat16_rn(v);
+    }
+}
+
+ctox_status launch_stream_norm(ctox_ctx *ctx, const StreamNorm &a, uint32_t m) {
+    const size_t smem = (size_t)a.width * 4;
+    if (smem + 1024 > (size_t)ctx->max_smem_optin)
+        return fail(ctx, CTOX_MEMORY_BUDGET, "stream norm: width %u does not fit shared memory", a.width);
+    if (smem > 40 * 1024)
+        CTOX_CUDA(ctx, cudaFuncSetAttribute(k_stream_norm, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    CTOX_CUDA(ctx, launch_pdl(k_stream_norm, dim3(m), dim3(kSnThreads), smem, ctx->stream, a));
+    return CTOX_OK;
+}
+
+__global__ void __launch_bounds__(kSnThreads) k_latent_split(const float *__restrict__ fan, uint32_t fan_stride,
+                                                             uint32_t q_rank, const float *__restrict__ q_norm,
+                                                             float eps, __nv_bfloat16 *__restrict__ cq, uint32_t cq_ld,
+                                                             LatentAppend ap, int has_append) {
+    pdl_launch();
+    pdl_wait();
+    __shared__ float red[kDvWarps];
+    const uint32_t m = blockIdx.x, tid = threadIdx.x;
+    const float *row = fan + (size_t)m * fan_stride;
+    float s = 0.f;
+    for (uint32_t c = tid; c < q_rank; c += kSnThreads) s += row[c] * row[c];
+    const float inv = 1.0f / sqrtf(position_sum<1>(s, red) / (float)q_rank + eps);
+    for (uint32_t c = tid; c < q_rank; c += kSnThreads)
+        cq[(size_t)m * cq_ld + c] = __float2bfloat16_rn(row[c] * inv * q_norm[c]);
+    if (has_append) latent_append_row(ap, m, tid, kSnThreads, red);
+}
+
+ctox_status launch_latent_split(ctox_ctx *ctx, const float *fan, uint32_t fan_stride, uint32_t q_rank,
+                                const float *q_norm, float eps, __nv_bfloat16 *cq, uint32_t cq_ld,
+                                const LatentAppend *append, uint32_t m) {
+    const LatentAppend ap = append ? *append : LatentAppend{};
+    CTOX_CUDA(ctx, launch_pdl(k_latent_split, dim3(m), dim3(kSnThreads), 0, ctx->stream, fan, fan_stride, q_rank, q_norm,
+                              eps, cq, cq_ld, ap, (int)(append != nullptr)));
+    return CTOX_OK;
+}
+
+// ------------------------------------------------------------------ embedding rows, weight layout
+__global__ void __launch_bounds__(256) k_embed_dense(const __nv_bfloat16 *__restrict__ embed, uint32_t ld,
+                                                     const uint32_t *__restrict__ tokens, uint32_t width,
+                                                     float *__restrict__ x) {
+    pdl_launch();
+    pdl_wait();
+    const __nv_bfloat16 *row = embed + (size_t)tokens[blockIdx.x] * ld;
+    for (uint32_t c = threadIdx.x; c < width; c += 256) x[(size_t)blockIdx.x * width + c] = __bfloat162float(row[c]);
+}
+
+ctox_status launch_embed_dense(ctox_ctx *ctx, const __nv_bfloat16 *embed, uint32_t ld, const uint32_t *tokens,
+                               uint32_t width, uint32_t m, float *x) {
+    CTOX_CUDA(ctx, launch_pdl(k_embed_dense, dim3(m), dim3(256), 0, ctx->stream, embed, ld, tokens, width, x));
+    return CTOX_OK;
+}
+
+__device__ __forceinline__ uint32_t pad_index(const PadAxis &a, uint32_t i) {
+    const uint32_t g = i / a.group, w = i % a.group;
+    return g * a.group_pad + (w < a.split ? w : w - a.split + a.split_pad);
+}
+
+__global__ void k_relayout(const __nv_bfloat16 *__restrict__ src, uint32_t rows, uint32_t cols, PadAxis ra, PadAxis ca,
+                           __nv_bfloat16 *__restrict__ dst, uint32_t dst_ld, uint32_t transpose_group,
+                           uint32_t transpose_cols) {
+    const uint64_t i = (uint64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (uint64_t)rows * cols) return;
+    const uint32_t r = pad_index(ra, (uint32_t)(i / cols)), c = pad_index(ca, (uint32_t)(i % cols));
+    if (transpose_group)
+        dst[((size_t)(r / transpose_group) * transpose_cols + c) * dst_ld + r % transpose_group] = src[i];
+    else
+        dst[(size_t)r * dst_ld + c] = src[i];
+}
+
+ctox_status launch_relayout(ctox_ctx *ctx, const __nv_bfloat16 *src, uint32_t rows, uint32_t cols, PadAxis ra,
+                            PadAxis ca, __nv_bfloat16 *dst, uint32_t dst_ld, uint32_t transpose_group,
+                            uint32_t transpose_cols) {
+    const uint64_t n = (uint64_t)rows * cols;
+    k_relayout<<<(unsigned)((n + 255) / 256), 256, 0, ctx->stream>>>(src, rows, cols, ra, ca, dst, dst_ld,
+                                                                     transpose_group, transpose_cols);
+    CTOX_CUDA(ctx, cudaGetLastError());
+    return CTOX_OK;
+}
+
+__global__ void k_fill_normal_bf16(__nv_bfloat16 *__restrict__ out, uint64_t n, float std, uint64_t seed) {
+    const uint64_t i = (uint64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n) return;
+    uint64_t x = seed + (i + 1) * 0x9E3779B97F4A7C15ull;  // splitmix64
+    x = (x ^ (x >> 30)) * 0xBF58476D1CE4E5B9ull;
+    x = (x ^ (x >> 27)) * 0x94D049BB133111EBull;
+    x ^= x >> 31;
+    const float u1 = ((float)(x >> 40) + 0.5f) * (1.0f / 16777216.0f);
+    const float u2 = (float)((x >> 16) & 0xffffff) * (1.0f / 16777216.0f);
+    out[i] = __float2bfloat16_rn(std * sqrtf(-2.0f * logf(u1)) * cosf(6.28318530718f * u2));
+}
+
+ctox_status launch_fill_normal_bf16(ctox_ctx *ctx, __nv_bfloat16 *out, uint64_t n, float std, uint64_t seed) {
+    k_fill_normal_bf16<<<(unsigned)((n + 255) / 256), 256, 0, ctx->stream>>>(out, n, std, seed);
+    CTOX_CUDA(ctx, cudaGetLastError());
+    return CTOX_OK;
+}
+
+}  // namespace ctox

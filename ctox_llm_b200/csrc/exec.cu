@@ -28,100 +28,12 @@
 #include <cstdlib>
 #include <vector>
 
-#include "common.cuh"
-#include "layers.cuh"
-#include "matvec.cuh"
-
-namespace ctox {
-constexpr uint32_t kMaxPass = 8;  // positions per pass (verify rows / prefill chunk)
-
-struct LayerW {
-    bool full = false;
-    float *in_ln = nullptr, *post_ln = nullptr;
-    ctox_matvec *in_fan = nullptr, *out = nullptr, *gate_up = nullptr, *down = nullptr;
-    float *conv_w = nullptr, *a_log = nullptr, *dt_bias = nullptr, *lin_norm = nullptr;
-    float *q_norm = nullptr, *k_norm = nullptr;
-};
-
-struct LayerS {
-    float *conv_state = nullptr;                  // [channels][kernel], committed
-    float *delta[2] = {nullptr, nullptr};         // [heads][128][128]; delta[cur] is committed
-    int cur = 0;
-    float *conv_in = nullptr;                     // [kMaxPass][channels] inputs of the last pass
-    float *q = nullptr, *k = nullptr, *v = nullptr, *g = nullptr, *beta = nullptr;  // last pass
-    void *k_cache = nullptr, *v_cache = nullptr;  // [slots][kv_heads][head_dim]
-};
-}  // namespace ctox
+#include "exec.cuh"
+#include "stack.cuh"
 
 using namespace ctox;
 
-struct ctox_exec {
-    ctox_ctx *ctx = nullptr;
-    ctox_model_config cfg{};  // this rank's shard: heads and FFN width divided by the group size
-    uint32_t tp_world = 1, tp_rank = 0;
-    uint32_t vocab_l = 0, vocab_off = 0;      // rows of lm_head on this rank
-    uint32_t kv_heads_global = 0;             // KV heads of the unsharded model
-    uint32_t draft_lo = 0, draft_n = 0;       // this rank's range of the draft id table
-    std::vector<uint32_t> draft_ids_host;
-    float *tp_buf = nullptr;                  // [kMaxPass][hidden] vector being summed over the group
-    uint32_t n_layers = 0;  // target layers; index n_layers is the MTP layer when present
-    uint32_t key_width = 0, value_width = 0, channels = 0, q_width = 0, kv_width = 0;
-    std::vector<LayerW> w;
-    std::vector<LayerS> s;
-    ctox_matvec *embed = nullptr, *lm_head = nullptr, *mtp_fc = nullptr, *draft_head = nullptr;
-    float *final_norm = nullptr, *mtp_norm_e = nullptr, *mtp_norm_h = nullptr, *mtp_norm = nullptr;
-    uint32_t *draft_ids = nullptr;  // device, [draft_vocab]
-    CommitLayer *commit_table = nullptr;  // device, one entry per linear-attention layer
-    uint32_t n_linear = 0;
-    bool lm_head_is_embed = false;
-    // session
-    uint64_t position = 0;     // tokens consumed by the target so far
-    bool have_hidden = false;  // hist_hidden[0 .. hist_n) holds the final hidden of the last hist_n positions
-    uint32_t hist_n = 0;       // committed positions of the last block (1..kMaxPass)
-    uint32_t hist_tokens[kMaxPass] = {0};  // tokens at positions position-hist_n+1 .. position-1 (drafts accepted)
-    uint64_t step_counter = 0;
-    bool warmed = false, keep_logits = false;
-    // Speculative transaction (engine.rs:322-362): an MTP decode resolves and commits its accepted
-    // prefix on the device and leaves the count here until commit_speculative confirms it.
-    int32_t pending = -1;
-    double last_enqueue_us = 0.0;  // host time the last decode spent enqueuing before it waited for the device
-    // Optional device times of the phases of a decode call (events at the phase boundaries):
-    // drafting, target pass, head + acceptance, commit.
-    bool phase_timing = false;
-    cudaEvent_t phase_ev[6] = {};
-    float phase_ms[4] = {0.f, 0.f, 0.f, 0.f};
-    bool commit_timed = false;
-    // A device error or a failed call after work was enqueued leaves the session state undefined:
-    // every call fails until reset_session (engine.rs:594-611 invalidates the session the same way).
-    bool poisoned = false;
-    // evidence of the last decode call (with keep_logits): the MTP layer's final hidden of every
-    // (token, hidden) pair it ran, in order, and the logits of every draft
-    float *mtp_trace = nullptr, *draft_trace = nullptr;
-    uint32_t mtp_trace_n = 0, draft_trace_n = 0, draft_rows = 0;
-    // buffers ([kMaxPass] rows each)
-    float *h = nullptr, *final_hidden = nullptr, *hist_hidden = nullptr, *embed_rows = nullptr;
-    float *mtp_h = nullptr, *mtp_hidden = nullptr;
-    float *aq = nullptr, *agate = nullptr, *attn_ws = nullptr;
-    float *lz = nullptr, *lcore = nullptr, *norm_scratch = nullptr;
-    float *draft_logits = nullptr, *logits = nullptr;
-    uint32_t *tokens_dev = nullptr;  // [kMaxPass + 1]: verify inputs = [token, drafts...]
-    uint32_t *mtp_tokens_dev = nullptr;
-    uint32_t *page_table = nullptr, *mtp_page_table = nullptr;
-    uint32_t attn_splits_max = kAttnMaxSplits;
-    uint64_t model_bytes = 0, session_bytes = 0;
-    std::vector<std::pair<void *, size_t>> owned;  // tracked raw allocations (vectors, buffers, states)
-};
-
 namespace {
-
-ctox_status xalloc(ctox_exec *e, void **p, size_t bytes, bool session, bool zero = true) {
-    ctox_status rc = dev_alloc(e->ctx, p, bytes);
-    if (rc) return rc;
-    e->owned.emplace_back(*p, bytes);
-    (session ? e->session_bytes : e->model_bytes) += bytes;
-    if (zero) CTOX_CUDA(e->ctx, cudaMemsetAsync(*p, 0, bytes, e->ctx->stream));
-    return CTOX_OK;
-}
 
 bool layer_is_full(const ctox_exec *e, uint32_t l) {
     if (l >= e->n_layers) return true;  // the MTP layer is a full-attention layer
@@ -201,6 +113,14 @@ ctox_status ctox_exec_create(ctox_ctx *ctx, const ctox_model_config *c_global, c
     return CTOX_OK;
 }
 
+ctox_status ctox_exec_create_stack(ctox_ctx *ctx, const ctox_stack_config *config, const ctox_layer_config *layers,
+                                   ctox_exec **out) {
+    if (!ctx || !config || !layers || !out) return CTOX_INVALID_STATE;
+    *out = nullptr;
+    CTOX_CUDA(ctx, cudaSetDevice(ctx->device));
+    return stack_create(ctx, config, layers, out);
+}
+
 ctox_status ctox_exec_destroy(ctox_exec *e) {
     if (!e) return CTOX_OK;
     cudaSetDevice(e->ctx->device);
@@ -218,6 +138,7 @@ ctox_status ctox_exec_destroy(ctox_exec *e) {
     for (auto &o : e->owned) dev_free(e->ctx, o.first, o.second);
     for (auto &ev : e->phase_ev)
         if (ev) cudaEventDestroy(ev);
+    stack_destroy(e);
     delete e;
     return CTOX_OK;
 }
@@ -322,6 +243,7 @@ extern "C" {
 ctox_status ctox_exec_load_matrix(ctox_exec *e, uint32_t layer, uint32_t tensor, const ctox_fused_matvec_op *op) {
     if (!e || !op) return CTOX_INVALID_STATE;
     ctox_ctx *ctx = e->ctx;
+    if (e->stack) return stack_load_matrix(e, layer, tensor, op);
     ctox_matvec **slot = nullptr;
     Shape shape{};
     if (!matrix_slot(e, layer, tensor, &slot, &shape))
@@ -346,7 +268,7 @@ ctox_status ctox_exec_load_matrix(ctox_exec *e, uint32_t layer, uint32_t tensor,
 ctox_status ctox_exec_load_vector(ctox_exec *e, uint32_t layer, uint32_t tensor, const float *values, uint64_t n) {
     if (!e || !values) return CTOX_INVALID_STATE;
     ctox_ctx *ctx = e->ctx;
-    if (layer == CTOX_LAYER_GLOBAL && tensor == CTOX_T_DRAFT_IDS) {
+    if (layer == CTOX_LAYER_GLOBAL && tensor == CTOX_T_DRAFT_IDS && !e->stack) {
         if (n != e->cfg.draft_vocab || n == 0)
             return fail(ctx, CTOX_SHAPE, "draft id table has %llu entries, expected %u", (unsigned long long)n,
                         e->cfg.draft_vocab);
@@ -365,8 +287,9 @@ ctox_status ctox_exec_load_vector(ctox_exec *e, uint32_t layer, uint32_t tensor,
         return CTOX_OK;
     }
     float **slot = nullptr;
-    uint64_t expect = 0;
-    if (!vector_slot(e, layer, tensor, &slot, &expect))
+    uint64_t expect = 0, *loaded = nullptr;
+    if (e->stack ? !stack_vector_slot(e, layer, tensor, &slot, &expect, &loaded)
+                 : !vector_slot(e, layer, tensor, &slot, &expect))
         return fail(ctx, CTOX_INVALID_ARTIFACT, "tensor %u is not a vector of layer %u", tensor, layer);
     if (n != expect)
         return fail(ctx, CTOX_SHAPE, "tensor %u of layer %u has %llu values, expected %llu", tensor, layer,
@@ -379,6 +302,7 @@ ctox_status ctox_exec_load_vector(ctox_exec *e, uint32_t layer, uint32_t tensor,
     }
     CTOX_CUDA(ctx, cudaMemcpyAsync(*slot, values, n * sizeof(float), cudaMemcpyHostToDevice, ctx->stream));
     CTOX_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+    if (loaded) *loaded |= 1ull << tensor;
     e->warmed = false;
     return CTOX_OK;
 }
@@ -628,6 +552,7 @@ ctox_status ctox_exec_fill_synthetic(ctox_exec *e, uint64_t seed, float mu, floa
     if (!e) return CTOX_INVALID_STATE;
     ctox_ctx *ctx = e->ctx;
     CTOX_CUDA(ctx, cudaSetDevice(ctx->device));
+    if (e->stack) return stack_fill_synthetic(e, seed);
     const ctox_model_config &c = e->cfg;
     // f16 block-scale quantile table of the log-normal(mu, sigma)
     std::vector<uint16_t> table(4096);
@@ -734,6 +659,11 @@ ctox_status ctox_exec_warmup(ctox_exec *e) {
     ctox_ctx *ctx = e->ctx;
     const ctox_model_config &c = e->cfg;
     CTOX_CUDA(ctx, cudaSetDevice(ctx->device));
+    if (e->stack) {
+        EX(stack_warmup(e));
+        e->warmed = true;
+        return ctox_exec_reset_session(e);
+    }
     if (!e->embed || !e->lm_head || !e->final_norm)
         return fail(ctx, CTOX_INVALID_STATE, "warmup: embedding, lm_head or final norm missing");
     if (!e->embed->parts[0].canon) return fail(ctx, CTOX_INVALID_STATE, "warmup: embedding rows not resident");
@@ -837,7 +767,7 @@ ctox_status ctox_exec_warmup(ctox_exec *e) {
 ctox_status ctox_exec_reset_session(ctox_exec *e) {
     if (!e) return CTOX_INVALID_STATE;
     ctox_ctx *ctx = e->ctx;
-    if (!e->h) return fail(ctx, CTOX_INVALID_STATE, "reset: executor is not warm");
+    if (!e->h && !(e->stack && e->warmed)) return fail(ctx, CTOX_INVALID_STATE, "reset: executor is not warm");
     const ctox_model_config &c = e->cfg;
     for (uint32_t l = 0; l < e->w.size(); ++l) {
         LayerS &ls = e->s[l];
@@ -871,6 +801,7 @@ ctox_status ctox_exec_prefill_synthetic(ctox_exec *e, uint64_t n, uint64_t seed)
     ctox_status rc = ctox_exec_reset_session(e);
     if (rc) return rc;
     uint64_t sd = seed;
+    if (e->stack) EX(stack_prefill_synthetic(e, n, seed));
     for (uint32_t l = 0; l < e->w.size(); ++l) {
         LayerS &ls = e->s[l];
         if (e->w[l].full) {
@@ -930,12 +861,6 @@ ctox_status ctox_exec_keep_logits(ctox_exec *e, int32_t enable) {
 
 // ------------------------------------------------------------------ passes
 namespace {
-
-#define EX(expr)               \
-    do {                       \
-        ctox_status rc_ = (expr); \
-        if (rc_) return rc_;   \
-    } while (0)
 
 AttnGeom attn_geom(const ctox_exec *e) {
     const ctox_model_config &c = e->cfg;
@@ -1035,6 +960,7 @@ ctox_status layer_body(ctox_exec *e, uint32_t l, float *h, uint32_t m, uint64_t 
 ctox_status target_pass(ctox_exec *e, uint32_t m, uint64_t pos0) {
     ctox_ctx *ctx = e->ctx;
     const ctox_model_config &c = e->cfg;
+    if (e->stack) return stack_pass(e, m, pos0);
     EX(matvec_embed_rows(e->embed, e->tokens_dev, m, e->h));
     const MvIn first = mv_in(e->w[0].in_fan);
     launch_residual_norm_prep(ctx->stream, e->h, nullptr, e->w[0].in_ln, c.rms_norm_epsilon, c.hidden_size, m, nullptr,
@@ -1052,6 +978,12 @@ ctox_status target_pass(ctox_exec *e, uint32_t m, uint64_t pos0) {
 ctox_status commit_positions(ctox_exec *e, uint32_t m, uint32_t n) {
     ctox_ctx *ctx = e->ctx;
     const ctox_model_config &c = e->cfg;
+    if (e->stack) {  // the cache only advances; the pass left the last position's hidden state in place
+        e->hist_n = 1;
+        e->have_hidden = true;
+        e->position += n;
+        return CTOX_OK;
+    }
     if (e->commit_table) {  // all linear-attention layers in one launch
         CommitCur cur{};
         uint32_t j = 0;
@@ -1146,25 +1078,60 @@ ctox_status session_usable(ctox_exec *e, const char *what) {
     return CTOX_OK;
 }
 
-ctox_status prefill_impl(ctox_exec *e, const uint32_t *tokens, uint64_t n, const volatile int32_t *cancel,
-                         bool *began) {
+// Positions the next pass may take of n remaining tokens.
+uint32_t pass_positions(const ctox_exec *e, uint64_t n) {
+    const uint32_t cap = e->stack ? e->stack->pass_cap : kMaxPass;
+    return (uint32_t)(n < cap ? n : cap);
+}
+
+// Logits of n positions (places in the pass) of the m of the last target pass, to host memory.
+ctox_status pass_logits(ctox_exec *e, uint32_t m, const uint32_t *places, uint32_t n, float *out) {
     ctox_ctx *ctx = e->ctx;
-    EX(ctox_exec_reset_session(e));
-    const uint64_t consume = n - 1;  // the last token is the input of the first decode
-    for (uint64_t a = 0; a < consume; a += kMaxPass) {
-        if (cancelled(cancel)) return fail(ctx, CTOX_CANCELLED, "prefill cancelled at token %llu", (unsigned long long)a);
-        const uint32_t m = (uint32_t)(consume - a < kMaxPass ? consume - a : kMaxPass);
-        *began = true;
-        EX(upload_u32(e, e->tokens_dev, tokens + a, m));
-        EX(target_pass(e, m, a));
-        EX(commit_positions(e, m, m));
-        for (uint32_t j = 0; j + 1 < m; ++j) e->hist_tokens[j] = tokens[a + 1 + j];
-        const bool last_chunk = a + m >= consume;
-        if (e->cfg.mtp_num_hidden_layers && !last_chunk) {
-            // keep the MTP cache exact: pairs (token p+1, final hidden p) of this chunk
-            EX(upload_u32(e, e->mtp_tokens_dev, tokens + a + 1, m));
-            EX(mtp_pass(e, m, a + 1, e->mtp_tokens_dev, e->hist_hidden, -1));
+    const size_t V = e->vocab_l;
+    if (e->stack) {
+        for (uint32_t i = 0; i < n; i += e->stack->head_rows) {
+            const uint32_t k = n - i < e->stack->head_rows ? n - i : e->stack->head_rows;
+            EX(stack_head_rows(e, places + i, k));
+            CTOX_CUDA(ctx, cudaMemcpyAsync(out + i * V, e->logits, k * V * 4, cudaMemcpyDeviceToHost, ctx->stream));
+            CTOX_CUDA(ctx, cudaStreamSynchronize(ctx->stream));  // the rows are used again
         }
+        return CTOX_OK;
+    }
+    if (!e->logits) EX(xalloc(e, (void **)&e->logits, (size_t)kMaxPass * V * 4, true));
+    EX(matvec_stream_prepared(e->lm_head, 0, m));
+    matvec_finish_enqueue(e->lm_head, m, e->logits, V);
+    for (uint32_t i = 0; i < n; ++i)
+        CTOX_CUDA(ctx, cudaMemcpyAsync(out + i * V, e->logits + places[i] * V, V * 4, cudaMemcpyDeviceToHost, ctx->stream));
+    return CTOX_OK;
+}
+
+ctox_status extend_impl(ctox_exec *e, const uint32_t *tokens, uint64_t n, const uint32_t *want, uint64_t n_want,
+                        float *logits_out, const volatile int32_t *cancel, bool *began) {
+    ctox_ctx *ctx = e->ctx;
+    std::vector<uint32_t> places;
+    uint64_t w = 0;
+    for (uint64_t a = 0; a < n;) {
+        if (cancelled(cancel)) return fail(ctx, CTOX_CANCELLED, "prefill cancelled at token %llu", (unsigned long long)a);
+        const uint32_t m = pass_positions(e, n - a);
+        *began = true;
+        if (e->cfg.mtp_num_hidden_layers && e->have_hidden && e->position > 0) {
+            // keep the MTP cache exact: pairs (token p+1, final hidden p) of the block before
+            uint32_t mt[kMaxPass];
+            for (uint32_t j = 0; j + 1 < e->hist_n; ++j) mt[j] = e->hist_tokens[j];
+            mt[e->hist_n - 1] = tokens[a];
+            EX(upload_u32(e, e->mtp_tokens_dev, mt, e->hist_n));
+            EX(mtp_pass(e, e->hist_n, e->position - e->hist_n + 1, e->mtp_tokens_dev, e->hist_hidden, -1));
+        }
+        EX(upload_u32(e, e->tokens_dev, tokens + a, m));
+        EX(target_pass(e, m, e->position));
+        places.clear();
+        for (; w < n_want && want[w] < a + m; ++w) places.push_back((uint32_t)(want[w] - a));
+        if (!places.empty())
+            EX(pass_logits(e, m, places.data(), (uint32_t)places.size(), logits_out + (w - places.size()) * e->vocab_l));
+        EX(commit_positions(e, m, m));
+        if (e->cfg.mtp_num_hidden_layers)
+            for (uint32_t j = 0; j + 1 < m; ++j) e->hist_tokens[j] = tokens[a + 1 + j];
+        a += m;
         // `tokens` may be pageable host memory: finish the chunk, and read the device error word
         int32_t dev_err = 0;
         EX(ctox_ctx_device_error(ctx, &dev_err));
@@ -1223,13 +1190,18 @@ ctox_status decode_impl(ctox_exec *e, uint32_t token, int32_t mtp_enabled, float
     if (e->phase_timing) cudaEventRecord(e->phase_ev[1], ctx->stream);
     EX(target_pass(e, m, P));
     if (e->phase_timing) cudaEventRecord(e->phase_ev[2], ctx->stream);
-    EX(matvec_stream_prepared(e->lm_head, 0, m));
     int32_t parent[kMaxPass];
     for (uint32_t i = 0; i < m; ++i) parent[i] = (int32_t)i - 1;
     const float inv_t = temperature > 0.f ? 1.0f / temperature : 0.f;
     const uint64_t step_id = e->step_counter++;
-    EX(head_verify_enqueue(e->lm_head, 0, m, m, parent, e->tokens_dev, inv_t, seed, step_id, e->vocab_l,
-                           e->keep_logits ? e->logits : nullptr, e->vocab_off));
+    if (e->stack) {
+        EX(stack_head_last(e));
+        EX(head_verify_logits_enqueue(ctx, e->logits, m, parent, e->tokens_dev, inv_t, seed, step_id, e->vocab_l));
+    } else {
+        EX(matvec_stream_prepared(e->lm_head, 0, m));
+        EX(head_verify_enqueue(e->lm_head, 0, m, m, parent, e->tokens_dev, inv_t, seed, step_id, e->vocab_l,
+                               e->keep_logits ? e->logits : nullptr, e->vocab_off));
+    }
     EX(head_tp_merge_enqueue(ctx, m, parent, e->tokens_dev, e->vocab_l));
     ctox_spec_record *rec_dev = nullptr;
     EX(head_accept_enqueue(ctx, m, parent, e->tokens_dev, inv_t, seed, step_id,
@@ -1293,9 +1265,37 @@ ctox_status ctox_exec_prefill(ctox_exec *e, const uint32_t *tokens, uint64_t n, 
     for (uint64_t i = 0; i < n; ++i)
         if (tokens[i] >= e->cfg.vocab_size) return fail(ctx, CTOX_SHAPE, "prefill: token %u out of range", tokens[i]);
     CTOX_CUDA(ctx, cudaSetDevice(ctx->device));
+    EX(ctox_exec_reset_session(e));
     bool began = false;
-    const ctox_status rc = prefill_impl(e, tokens, n, cancel, &began);
+    // the last token is the input of the first decode
+    const ctox_status rc = extend_impl(e, tokens, n - 1, nullptr, 0, nullptr, cancel, &began);
     // a prefill that stopped half way (cancelled or failed) leaves no usable session
+    if (rc && began) e->poisoned = true;
+    return rc;
+}
+
+ctox_status ctox_exec_extend(ctox_exec *e, const uint32_t *tokens, uint64_t n, const uint32_t *want, uint64_t n_want,
+                             float *logits_out, const volatile int32_t *cancel) {
+    if (!e || (n && !tokens) || (n_want && (!want || !logits_out))) return CTOX_INVALID_STATE;
+    ctox_ctx *ctx = e->ctx;
+    if (cancelled(cancel)) return fail(ctx, CTOX_CANCELLED, "extend cancelled");
+    if (!e->warmed) return fail(ctx, CTOX_INVALID_STATE, "extend: executor is not warm");
+    EX(session_usable(e, "extend"));
+    if (e->pending >= 0)
+        return fail(ctx, CTOX_INVALID_STATE, "extend requires the previous speculative branch to be committed");
+    if (n + e->position + 2 * kMaxPass > e->cfg.max_context_tokens)
+        return fail(ctx, CTOX_SHAPE, "extend: %llu tokens at position %llu do not fit the context", (unsigned long long)n,
+                    (unsigned long long)e->position);
+    for (uint64_t i = 0; i < n; ++i)
+        if (tokens[i] >= e->cfg.vocab_size) return fail(ctx, CTOX_SHAPE, "extend: token %u out of range", tokens[i]);
+    for (uint64_t i = 0; i < n_want; ++i)
+        if (want[i] >= n || (i && want[i] <= want[i - 1]))
+            return fail(ctx, CTOX_SHAPE, "extend: wanted places must ascend and lie among the tokens");
+    if (n_want && e->tp_world > 1)
+        return fail(ctx, CTOX_UNSUPPORTED_OPERATION, "extend: the logits of a group are vocabulary shards");
+    CTOX_CUDA(ctx, cudaSetDevice(ctx->device));
+    bool began = false;
+    const ctox_status rc = extend_impl(e, tokens, n, want, n_want, logits_out, cancel, &began);
     if (rc && began) e->poisoned = true;
     return rc;
 }
@@ -1421,6 +1421,25 @@ ctox_status ctox_exec_last_logits(ctox_exec *e, uint32_t position, float *out) {
         return fail(ctx, CTOX_INVALID_STATE, "logits are not kept (ctox_exec_keep_logits) or position out of range");
     CTOX_CUDA(ctx, cudaMemcpyAsync(out, e->logits + (size_t)position * e->vocab_l, (size_t)e->vocab_l * 4,
                                    cudaMemcpyDeviceToHost, ctx->stream));
+    CTOX_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+    return CTOX_OK;
+}
+
+ctox_status ctox_exec_keep_streams(ctox_exec *e) {
+    if (!e) return CTOX_INVALID_STATE;
+    if (!e->stack) return fail(e->ctx, CTOX_UNSUPPORTED_OPERATION, "keep_streams: not a layer-stack model");
+    CTOX_CUDA(e->ctx, cudaSetDevice(e->ctx->device));
+    return stack_keep_streams(e);
+}
+
+ctox_status ctox_exec_last_stream(ctox_exec *e, uint32_t layer, uint64_t position, uint64_t n, float *out) {
+    if (!e || !out) return CTOX_INVALID_STATE;
+    ctox_ctx *ctx = e->ctx;
+    if (!e->stack || !e->stack->streams || layer >= e->n_layers || position + n > e->position)
+        return fail(ctx, CTOX_INVALID_STATE, "streams are not kept (ctox_exec_keep_streams) or out of range");
+    const size_t H = e->cfg.hidden_size;
+    CTOX_CUDA(ctx, cudaMemcpyAsync(out, e->stack->streams + ((size_t)layer * e->cfg.max_context_tokens + position) * H,
+                                   n * H * 4, cudaMemcpyDeviceToHost, ctx->stream));
     CTOX_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
     return CTOX_OK;
 }

@@ -64,7 +64,7 @@ __global__ void __launch_bounds__(kHeadThreads) k_head_stats(
     uint32_t npos,
     float inv_temperature, unsigned long long seed, unsigned long long step, TreeDesc tree,
     NodeStat *__restrict__ cta_stats, float *__restrict__ child_z, float *__restrict__ logits_out,
-    unsigned long long logits_stride, uint32_t row_offset) {
+    unsigned long long logits_stride, uint32_t row_offset, const float *__restrict__ plain) {
     pdl_launch();
     pdl_wait();
     __shared__ NodeStat sh[kHeadThreads / 32][kMaxPosPerPass];
@@ -75,8 +75,9 @@ __global__ void __launch_bounds__(kHeadThreads) k_head_stats(
         const uint32_t pr = row / kPairRows, rl = row % kPairRows;
         float lg[kMaxPosPerPass];
 #pragma unroll
-        for (int m = 0; m < kMaxPosPerPass; ++m) lg[m] = 0.f;
-        for (uint32_t sl = 0; sl < slices; ++sl) {
+        for (int m = 0; m < kMaxPosPerPass; ++m)
+            lg[m] = plain && (uint32_t)m < npos ? plain[(size_t)m * logits_stride + row] : 0.f;
+        for (uint32_t sl = 0; sl < slices; ++sl) {  // no slices when the logits are given
             // a slot is [position][32 rows]: the 32 rows of a pair are one coalesced line per position
             const float *base = partial + ((size_t)pr * slices + sl) * max_pieces * (kPairRows * kMaxPosPerPass) + rl;
             const uint32_t n = pieces[pr * slices + sl];
@@ -638,10 +639,14 @@ ctox_status ctox_sample_topk_topp(ctox_ctx *ctx, const float *logits_dev, uint32
 
 namespace ctox {
 
-ctox_status head_verify_enqueue(ctox_matvec *mv, uint32_t node0, uint32_t npos, uint32_t n_nodes,
-                                const int32_t *parent, const uint32_t *tokens_dev, float inv_t, uint64_t seed,
-                                uint64_t step, uint32_t rows, float *logits_out_dev, uint32_t row_offset) {
-    ctox_ctx *ctx = mv->ctx;
+namespace {
+
+// Statistics of verify nodes node0 .. node0 + npos, from the partial sums of a streamed lm_head or from
+// finished logits (`plain`, [npos][logits_stride]).
+ctox_status head_stats_enqueue(ctox_ctx *ctx, const ctox_matvec *mv, const float *plain, uint64_t logits_stride,
+                               uint32_t node0, uint32_t npos, uint32_t n_nodes, const int32_t *parent,
+                               const uint32_t *tokens_dev, float inv_t, uint64_t seed, uint64_t step, uint32_t rows,
+                               float *logits_out_dev, uint32_t row_offset) {
     HeadScratch hs;
     ctox_status rc = head_scratch(ctx, hs);
     if (rc) return rc;
@@ -650,16 +655,32 @@ ctox_status head_verify_enqueue(ctox_matvec *mv, uint32_t node0, uint32_t npos, 
     tree.n_nodes = n_nodes;
     tree.token = tokens_dev;
     for (uint32_t i = 0; i < n_nodes; ++i) tree.parent[i] = parent[i];
-    MatvecPart &p = mv->parts[0];
+    const MatvecPart *p = mv ? &mv->parts[0] : nullptr;
     uint32_t grid = (rows + kHeadThreads - 1) / kHeadThreads;
     if (grid > kHeadGridMax) grid = kHeadGridMax;
-    launch_pdl(k_head_stats, dim3(grid), dim3(kHeadThreads), 0, ctx->stream, p.partial, p.split[npos > 4 ? 1 : 0].pieces, mv->s_out,
-                                                        mv->bias, rows, p.slices, p.max_pieces, node0, npos,
-                                                        inv_t, seed, step, tree, hs.cta_stats, hs.child_z,
-                                                        logits_out_dev, (unsigned long long)mv->rows, row_offset);
+    launch_pdl(k_head_stats, dim3(grid), dim3(kHeadThreads), 0, ctx->stream, p ? p->partial : nullptr,
+               p ? p->split[npos > 4 ? 1 : 0].pieces : nullptr, mv ? mv->s_out : nullptr, mv ? mv->bias : nullptr, rows,
+               p ? p->slices : 0u, p ? p->max_pieces : 0u, node0, npos, inv_t, seed, step, tree, hs.cta_stats, hs.child_z,
+               logits_out_dev, (unsigned long long)logits_stride, row_offset, plain);
     launch_pdl(k_head_merge, dim3(1), dim3(32 * kMaxPosPerPass), 0, ctx->stream, hs.cta_stats, grid, node0, npos, hs.node_stats);
     CTOX_CUDA(ctx, cudaGetLastError());
     return CTOX_OK;
+}
+
+}  // namespace
+
+ctox_status head_verify_enqueue(ctox_matvec *mv, uint32_t node0, uint32_t npos, uint32_t n_nodes,
+                                const int32_t *parent, const uint32_t *tokens_dev, float inv_t, uint64_t seed,
+                                uint64_t step, uint32_t rows, float *logits_out_dev, uint32_t row_offset) {
+    return head_stats_enqueue(mv->ctx, mv, nullptr, mv->rows, node0, npos, n_nodes, parent, tokens_dev, inv_t, seed, step,
+                              rows, logits_out_dev, row_offset);
+}
+
+ctox_status head_verify_logits_enqueue(ctox_ctx *ctx, const float *logits, uint32_t npos, const int32_t *parent,
+                                       const uint32_t *tokens_dev, float inv_t, uint64_t seed, uint64_t step,
+                                       uint32_t rows) {
+    return head_stats_enqueue(ctx, nullptr, logits, rows, 0, npos, npos, parent, tokens_dev, inv_t, seed, step, rows,
+                              nullptr, 0);
 }
 
 ctox_status head_accept_enqueue(ctox_ctx *ctx, uint32_t n_nodes, const int32_t *parent,

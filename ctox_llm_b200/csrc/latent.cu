@@ -1,0 +1,418 @@
+// Attention over the latent cache for short passes (decode and small portions of a prompt).
+#include "latent.cuh"
+
+#include <cmath>
+
+namespace ctox {
+
+constexpr int kLaThreads = 256, kLaWarps = 8;
+constexpr int kLaRowsMma = 16, kLaTileMma = 64;  // query rows per CTA, tokens per tile (tensor cores)
+constexpr int kLaRowsFma = 8, kLaTileFma = 32;   // the same on CUDA cores
+
+struct KeyRange {
+    uint32_t lo, hi;
+};
+__host__ __device__ inline KeyRange key_range(uint32_t pos0, uint32_t m, uint32_t window) {
+    KeyRange r;
+    r.hi = pos0 + m;
+    r.lo = window && pos0 + 1 > window ? pos0 + 1 - window : 0;
+    return r;
+}
+__device__ __forceinline__ bool key_visible(uint32_t key, uint32_t pos, uint32_t window) {
+    return key <= pos && (!window || pos - key < window);
+}
+
+template <typename T>
+__device__ __forceinline__ float cache_value(const T *p);
+template <>
+__device__ __forceinline__ float cache_value<float>(const float *p) { return *p; }
+template <>
+__device__ __forceinline__ float cache_value<__nv_bfloat16>(const __nv_bfloat16 *p) { return __bfloat162float(*p); }
+
+// CUDA cores, fp32 throughout: eight query rows against 32-token tiles; a warp scores one row (lane =
+// token), then every thread owns J latent columns of all eight rows.
+template <typename T, int J>
+__global__ void __launch_bounds__(kLaThreads) k_latent_attention(LatentAttn a, uint32_t splits) {
+    pdl_launch();
+    pdl_wait();
+    extern __shared__ __align__(16) float sm[];
+    const uint32_t D = a.kv_pad + a.rot_pad, ldk = D + 1, rows = a.m * a.heads;
+    float *q_s = sm;                           // [8][D]
+    float *k_s = q_s + kLaRowsFma * D;          // [32][D + 1]
+    float *p_s = k_s + kLaTileFma * ldk;        // [8][32]
+    float *al_s = p_s + kLaRowsFma * kLaTileFma;  // [8]
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const uint32_t row0 = blockIdx.x * kLaRowsFma, sp = blockIdx.y, row = row0 + warp;
+    const KeyRange kr = key_range(a.pos0, a.m, a.window);
+    const uint32_t tiles = (kr.hi - kr.lo + kLaTileFma - 1) / kLaTileFma;
+    const uint32_t t_beg = (uint32_t)((uint64_t)tiles * sp / splits), t_end = (uint32_t)((uint64_t)tiles * (sp + 1) / splits);
+    for (uint32_t i = tid; i < kLaRowsFma * D; i += kLaThreads) {
+        const uint32_t r = row0 + i / D, c = i % D;
+        q_s[i] = r >= rows ? 0.f
+                           : (c < a.kv_pad ? a.q_abs[(size_t)r * a.kv_pad + c] : a.q_rot[(size_t)r * a.q_stride + c - a.kv_pad]);
+    }
+    float o[kLaRowsFma][J];
+#pragma unroll
+    for (int r = 0; r < kLaRowsFma; ++r)
+#pragma unroll
+        for (int j = 0; j < J; ++j) o[r][j] = 0.f;
+    float mx = -INFINITY, sum = 0.f;
+    const uint32_t pos = a.pos0 + row / a.heads;
+    for (uint32_t tile = t_beg; tile < t_end; ++tile) {
+        const uint32_t t0 = kr.lo + tile * kLaTileFma;
+        __syncthreads();
+        for (uint32_t r = warp; r < kLaTileFma; r += kLaWarps) {
+            const uint32_t t = t0 + r;
+            const T *src = t < kr.hi ? (const T *)a.cache + paged_slot(a.page_table, a.page_tokens, t) * D : nullptr;
+            for (uint32_t c = lane; c < D; c += 32) k_s[r * ldk + c] = src ? cache_value(src + c) : 0.f;
+        }
+        __syncthreads();
+        const uint32_t t = t0 + lane;
+        float s = -INFINITY;
+        if (row < rows && t < kr.hi && key_visible(t, pos, a.window)) {
+            float s0 = 0.f, s1 = 0.f;
+            const float *q = q_s + warp * D, *k = k_s + lane * ldk;
+            for (uint32_t c = 0; c < D; c += 2) {
+                s0 = fmaf(q[c], k[c], s0);
+                s1 = fmaf(q[c + 1], k[c + 1], s1);
+            }
+            s = (s0 + s1) * a.scale;
+        }
+        float tm = s;
+#pragma unroll
+        for (int off = 16; off > 0; off >>= 1) tm = fmaxf(tm, __shfl_xor_sync(0xffffffffu, tm, off));
+        const float nm = fmaxf(mx, tm);
+        const float alpha = nm == -INFINITY ? 1.f : expf(mx - nm);
+        const float p = s == -INFINITY ? 0.f : expf(s - nm);
+        float ps = p;
+#pragma unroll
+        for (int off = 16; off > 0; off >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, off);
+        sum = sum * alpha + ps;
+        mx = nm;
+        p_s[warp * kLaTileFma + lane] = p;
+        if (lane == 0) al_s[warp] = alpha;
+        __syncthreads();
+#pragma unroll
+        for (int r = 0; r < kLaRowsFma; ++r) {
+            const float al = al_s[r];
+#pragma unroll
+            for (int j = 0; j < J; ++j) o[r][j] *= al;
+        }
+        for (uint32_t k = 0; k < kLaTileFma; ++k) {
+            float v[J];
+#pragma unroll
+            for (int j = 0; j < J; ++j) {
+                const uint32_t c = tid + j * kLaThreads;
+                v[j] = c < a.kv_pad ? k_s[k * ldk + c] : 0.f;
+            }
+#pragma unroll
+            for (int r = 0; r < kLaRowsFma; ++r) {
+                const float pr = p_s[r * kLaTileFma + k];
+#pragma unroll
+                for (int j = 0; j < J; ++j) o[r][j] = fmaf(pr, v[j], o[r][j]);
+            }
+        }
+    }
+    if (lane == 0 && row < rows) {
+        a.ws_ml[((size_t)sp * rows + row) * 2] = mx;
+        a.ws_ml[((size_t)sp * rows + row) * 2 + 1] = sum;
+    }
+#pragma unroll
+    for (int r = 0; r < kLaRowsFma; ++r)
+#pragma unroll
+        for (int j = 0; j < J; ++j) {
+            const uint32_t c = tid + j * kLaThreads;
+            if (c < a.kv_pad && row0 + r < rows) a.ws_o[((size_t)sp * rows + row0 + r) * a.kv_pad + c] = o[r][j];
+        }
+}
+
+// ------------------------------------------------------------------ tensor cores, bf16 cache
+__device__ __forceinline__ uint32_t smem_u32(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void ldsm_x4(uint32_t *r, uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+                 : "r"(addr)
+                 : "memory");
+}
+__device__ __forceinline__ void ldsm_x2(uint32_t *r, uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm_x4_t(uint32_t *r, uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+                 : "r"(addr)
+                 : "memory");
+}
+__device__ __forceinline__ void mma_bf16(float *c, const uint32_t *a, const uint32_t *b) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
+}
+__device__ __forceinline__ void split_bf16(float v, __nv_bfloat16 &hi, __nv_bfloat16 &lo) {
+    hi = __float2bfloat16_rn(v);
+    lo = __float2bfloat16_rn(v - __bfloat162float(hi));
+}
+
+// Sixteen query rows against 64-token tiles of cache rows. Scores: each warp eight tokens over the whole
+// row; weighted sum: each warp every eighth group of eight latent columns, the same tile read as the
+// transposed operand. Queries and weights are split into two bf16 parts (about 16 bits), so the only bf16
+// rounding is the cache's. NT: groups of eight columns per warp.
+template <int NT>
+__global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAttn a, uint32_t splits, uint32_t stages) {
+    pdl_launch();
+    extern __shared__ __align__(16) uint8_t smraw[];
+    constexpr uint32_t kLdP = kLaTileMma + 8;
+    const uint32_t D = a.kv_pad + a.rot_pad, ld = D + 8, rows = a.m * a.heads;
+    __nv_bfloat16 *k_s = reinterpret_cast<__nv_bfloat16 *>(smraw);                // [stages][64][ld]
+    __nv_bfloat16 *q_s = k_s + (size_t)stages * kLaTileMma * ld;                   // [hi, lo][16][ld]
+    __nv_bfloat16 *p_s = q_s + 2 * kLaRowsMma * ld;                                // [hi, lo][16][kLdP]
+    float *red = reinterpret_cast<float *>(p_s + 2 * kLaRowsMma * kLdP);           // [8][16]
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+    const uint32_t row0 = blockIdx.x * kLaRowsMma, sp = blockIdx.y;
+    const KeyRange kr = key_range(a.pos0, a.m, a.window);
+    const uint32_t tiles = (kr.hi - kr.lo + kLaTileMma - 1) / kLaTileMma;
+    const uint32_t t_beg = (uint32_t)((uint64_t)tiles * sp / splits), t_end = (uint32_t)((uint64_t)tiles * (sp + 1) / splits);
+    const uint32_t chunks = D / 8;
+    pdl_wait();
+    auto load_tile = [&](uint32_t tile, uint32_t stage) {
+        const uint32_t t0 = kr.lo + tile * kLaTileMma;
+        for (uint32_t r = warp; r < kLaTileMma; r += kLaWarps) {
+            const uint32_t t = t0 + r;
+            const bool in = t < kr.hi;
+            const __nv_bfloat16 *src =
+                (const __nv_bfloat16 *)a.cache + (in ? paged_slot(a.page_table, a.page_tokens, t) * D : 0);
+            __nv_bfloat16 *dst = k_s + ((size_t)stage * kLaTileMma + r) * ld;
+            for (uint32_t c = lane; c < chunks; c += 32)
+                asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + c * 8)), "l"(src + c * 8),
+                             "r"(in ? 16 : 0)
+                             : "memory");
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    if (t_beg < t_end) load_tile(t_beg, 0);
+    const float qscale = a.scale * 1.4426950408889634f;  // scores in units of log 2
+    for (uint32_t i = tid; i < kLaRowsMma * D; i += kLaThreads) {
+        const uint32_t r = i / D, c = i % D, row = row0 + r;
+        float v = 0.f;
+        if (row < rows)
+            v = (c < a.kv_pad ? a.q_abs[(size_t)row * a.kv_pad + c] : a.q_rot[(size_t)row * a.q_stride + c - a.kv_pad]) * qscale;
+        __nv_bfloat16 hi, lo;
+        split_bf16(v, hi, lo);
+        q_s[r * ld + c] = hi;
+        q_s[(kLaRowsMma + r) * ld + c] = lo;
+    }
+    float o[NT][4];
+#pragma unroll
+    for (int j = 0; j < NT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+    float mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.f, 0.f};  // rows g, g + 8
+    const uint32_t pos_a = a.pos0 + (row0 + g) / a.heads, pos_b = a.pos0 + (row0 + g + 8) / a.heads;
+    const uint32_t q_addr = smem_u32(q_s + (lane & 15) * ld + (lane >> 4) * 8);
+    const uint32_t p_addr = smem_u32(p_s + (lane & 15) * kLdP + (lane >> 4) * 8);
+    for (uint32_t tile = t_beg; tile < t_end; ++tile) {
+        const uint32_t st = stages == 2 ? (tile - t_beg) & 1 : 0;
+        const bool ahead = stages == 2 && tile + 1 < t_end;
+        if (ahead) load_tile(tile + 1, st ^ 1);
+        if (ahead)
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        else
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        const __nv_bfloat16 *kt = k_s + (size_t)st * kLaTileMma * ld;
+        // ---- scores of tokens warp * 8 .. + 8
+        float s4[4][4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) s4[i][0] = s4[i][1] = s4[i][2] = s4[i][3] = 0.f;
+        const uint32_t k_addr = smem_u32(kt + (warp * 8 + (lane & 7)) * ld + ((lane >> 3) & 1) * 8);
+        for (uint32_t k = 0; k < D; k += 16) {
+            uint32_t ah[4], al[4], b[2];
+            ldsm_x4(ah, q_addr + k * 2);
+            ldsm_x4(al, q_addr + kLaRowsMma * ld * 2 + k * 2);
+            ldsm_x2(b, k_addr + k * 2);
+            if ((k >> 4) & 1) {
+                mma_bf16(s4[2], ah, b);
+                mma_bf16(s4[3], al, b);
+            } else {
+                mma_bf16(s4[0], ah, b);
+                mma_bf16(s4[1], al, b);
+            }
+        }
+        float s[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            s[i] = (s4[0][i] + s4[2][i]) + (s4[1][i] + s4[3][i]);
+            const uint32_t t = kr.lo + tile * kLaTileMma + warp * 8 + t4 * 2 + (i & 1);
+            const uint32_t row = row0 + g + (i >= 2 ? 8 : 0);
+            if (row >= rows || t >= kr.hi || !key_visible(t, i >= 2 ? pos_b : pos_a, a.window)) s[i] = -INFINITY;
+        }
+        float tm[2] = {fmaxf(s[0], s[1]), fmaxf(s[2], s[3])};
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            tm[i] = fmaxf(tm[i], __shfl_xor_sync(0xffffffffu, tm[i], 1));
+            tm[i] = fmaxf(tm[i], __shfl_xor_sync(0xffffffffu, tm[i], 2));
+        }
+        if (t4 == 0) {
+            red[warp * kLaRowsMma + g] = tm[0];
+            red[warp * kLaRowsMma + g + 8] = tm[1];
+        }
+        __syncthreads();
+        float alpha[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            float nm = mx[i];
+#pragma unroll
+            for (int w = 0; w < kLaWarps; ++w) nm = fmaxf(nm, red[w * kLaRowsMma + g + i * 8]);
+            alpha[i] = nm == -INFINITY ? 1.f : exp2f(mx[i] - nm);
+            mx[i] = nm;
+            float p[2];
+#pragma unroll
+            for (int j = 0; j < 2; ++j) p[j] = s[i * 2 + j] == -INFINITY ? 0.f : exp2f(s[i * 2 + j] - nm);
+            sum[i] = sum[i] * alpha[i] + p[0] + p[1];
+            __nv_bfloat162 hi, lo;
+            split_bf16(p[0], hi.x, lo.x);
+            split_bf16(p[1], hi.y, lo.y);
+            __nv_bfloat16 *dst = p_s + (g + i * 8) * kLdP + warp * 8 + t4 * 2;
+            *reinterpret_cast<__nv_bfloat162 *>(dst) = hi;
+            *reinterpret_cast<__nv_bfloat162 *>(dst + kLaRowsMma * kLdP) = lo;
+        }
+        __syncthreads();
+        // ---- weighted sum of the cache rows
+#pragma unroll
+        for (int j = 0; j < NT; ++j) {
+            o[j][0] *= alpha[0];
+            o[j][1] *= alpha[0];
+            o[j][2] *= alpha[1];
+            o[j][3] *= alpha[1];
+        }
+#pragma unroll
+        for (uint32_t k = 0; k < kLaTileMma; k += 32) {
+            uint32_t ph[2][4], pl[2][4];
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                ldsm_x4(ph[i], p_addr + (k + i * 16) * 2);
+                ldsm_x4(pl[i], p_addr + kLaRowsMma * kLdP * 2 + (k + i * 16) * 2);
+            }
+            const uint32_t v_addr = smem_u32(kt + (k + lane) * ld);
+#pragma unroll
+            for (int j = 0; j < NT; ++j) {
+                const uint32_t n = (warp + j * kLaWarps) * 8;
+                if (n < a.kv_pad) {
+                    uint32_t b[4];
+                    ldsm_x4_t(b, v_addr + n * 2);
+                    mma_bf16(o[j], ph[0], b);
+                    mma_bf16(o[j], pl[0], b);
+                    mma_bf16(o[j], ph[1], b + 2);
+                    mma_bf16(o[j], pl[1], b + 2);
+                }
+            }
+        }
+        __syncthreads();
+        if (stages == 1 && tile + 1 < t_end) load_tile(tile + 1, 0);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 1);
+        sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 2);
+    }
+    __syncthreads();
+    if (t4 == 0) {
+        red[warp * kLaRowsMma + g] = sum[0];
+        red[warp * kLaRowsMma + g + 8] = sum[1];
+    }
+    __syncthreads();
+    if (warp == 0 && t4 == 0) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const uint32_t row = row0 + g + i * 8;
+            if (row >= rows) continue;
+            float total = 0.f;
+            for (int w = 0; w < kLaWarps; ++w) total += red[w * kLaRowsMma + g + i * 8];
+            a.ws_ml[((size_t)sp * rows + row) * 2] = mx[i] * 0.6931471805599453f;
+            a.ws_ml[((size_t)sp * rows + row) * 2 + 1] = total;
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+        const uint32_t n = (warp + j * kLaWarps) * 8;
+        if (n >= a.kv_pad) continue;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const uint32_t row = row0 + g + i * 8;
+            if (row < rows)
+                *reinterpret_cast<float2 *>(a.ws_o + ((size_t)sp * rows + row) * a.kv_pad + n + t4 * 2) =
+                    make_float2(o[j][i * 2], o[j][i * 2 + 1]);
+        }
+    }
+}
+
+namespace {
+
+size_t mma_smem(const LatentAttn &a, uint32_t stages) {
+    const size_t ld = a.kv_pad + a.rot_pad + 8;
+    return (stages * kLaTileMma + 2 * kLaRowsMma) * ld * 2 + 2 * kLaRowsMma * (kLaTileMma + 8) * 2 + kLaWarps * kLaRowsMma * 4;
+}
+// Tile stages of the tensor-core form (0: it does not apply).
+uint32_t mma_stages(const ctox_ctx *ctx, const LatentAttn &a) {
+    if (!a.bf16 || a.kv_pad > 1024) return 0;
+    for (uint32_t st = 2; st > 0; --st)
+        if (mma_smem(a, st) <= (size_t)ctx->max_smem_optin) return st;
+    return 0;
+}
+size_t fma_smem(const LatentAttn &a) {
+    const size_t D = a.kv_pad + a.rot_pad;
+    return (kLaRowsFma * D + kLaTileFma * (D + 1) + kLaRowsFma * kLaTileFma + kLaRowsFma) * 4;
+}
+
+template <typename T, int J>
+ctox_status fma_launch(ctox_ctx *ctx, const LatentAttn &a, uint32_t splits, uint32_t row_tiles, size_t smem) {
+    CTOX_CUDA(ctx, cudaFuncSetAttribute(k_latent_attention<T, J>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    CTOX_CUDA(ctx, launch_pdl(k_latent_attention<T, J>, dim3(row_tiles, splits), dim3(kLaThreads), smem, ctx->stream, a, splits));
+    return CTOX_OK;
+}
+template <int NT>
+ctox_status mma_launch(ctox_ctx *ctx, const LatentAttn &a, uint32_t splits, uint32_t row_tiles, size_t smem, uint32_t stages) {
+    CTOX_CUDA(ctx, cudaFuncSetAttribute(k_latent_attention_mma<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    CTOX_CUDA(ctx, launch_pdl(k_latent_attention_mma<NT>, dim3(row_tiles, splits), dim3(kLaThreads), smem, ctx->stream, a,
+                              splits, stages));
+    return CTOX_OK;
+}
+
+}  // namespace
+
+uint32_t latent_attn_splits(const ctox_ctx *ctx, const LatentAttn &a) {
+    const bool mma = mma_stages(ctx, a) > 0;
+    const uint32_t rows = a.m * a.heads, per = mma ? kLaRowsMma : kLaRowsFma, tile = mma ? kLaTileMma : kLaTileFma;
+    const uint32_t row_tiles = (rows + per - 1) / per;
+    const KeyRange kr = key_range(a.pos0, a.m, a.window);
+    const uint32_t tiles = (kr.hi - kr.lo + tile - 1) / tile;
+    uint32_t s = (uint32_t)ctx->sm_count / row_tiles;
+    if (s > kAttnSplitsDense) s = kAttnSplitsDense;
+    if (s > tiles) s = tiles;
+    return s ? s : 1;
+}
+
+ctox_status launch_latent_attention(ctox_ctx *ctx, const LatentAttn &a, uint32_t splits) {
+    const uint32_t rows = a.m * a.heads, stages = mma_stages(ctx, a);
+    if (stages) {
+        const uint32_t row_tiles = (rows + kLaRowsMma - 1) / kLaRowsMma, nt = (a.kv_pad + 63) / 64;
+        const size_t smem = mma_smem(a, stages);
+        if (nt <= 1) return mma_launch<1>(ctx, a, splits, row_tiles, smem, stages);
+        if (nt <= 2) return mma_launch<2>(ctx, a, splits, row_tiles, smem, stages);
+        if (nt <= 4) return mma_launch<4>(ctx, a, splits, row_tiles, smem, stages);
+        if (nt <= 8) return mma_launch<8>(ctx, a, splits, row_tiles, smem, stages);
+        return mma_launch<16>(ctx, a, splits, row_tiles, smem, stages);
+    }
+    const size_t smem = fma_smem(a);
+    const uint32_t row_tiles = (rows + kLaRowsFma - 1) / kLaRowsFma, j = (a.kv_pad + kLaThreads - 1) / kLaThreads;
+    if (smem > (size_t)ctx->max_smem_optin || j > 8)
+        return fail(ctx, CTOX_MEMORY_BUDGET, "latent attention: a latent of %u + %u values does not fit shared memory",
+                    a.kv_pad, a.rot_pad);
+#define FMA(T)                                                             \
+    (j <= 1 ? fma_launch<T, 1>(ctx, a, splits, row_tiles, smem)            \
+     : j <= 2 ? fma_launch<T, 2>(ctx, a, splits, row_tiles, smem)          \
+     : j <= 4 ? fma_launch<T, 4>(ctx, a, splits, row_tiles, smem)          \
+              : fma_launch<T, 8>(ctx, a, splits, row_tiles, smem))
+    return a.bf16 ? FMA(__nv_bfloat16) : FMA(float);
+#undef FMA
+}
+
+}  // namespace ctox

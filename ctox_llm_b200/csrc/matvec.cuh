@@ -78,6 +78,10 @@ void matvec_finish_enqueue(ctox_matvec *mv, uint32_t npos, float *y, uint64_t y_
 ctox_status head_verify_enqueue(ctox_matvec *mv, uint32_t node0, uint32_t npos, uint32_t n_nodes,
                                 const int32_t *parent, const uint32_t *tokens_dev, float inv_t, uint64_t seed,
                                 uint64_t step, uint32_t rows, float *logits_out_dev, uint32_t row_offset);
+// The same from finished logits [npos][rows] (a head that writes them).
+ctox_status head_verify_logits_enqueue(ctox_ctx *ctx, const float *logits, uint32_t npos, const int32_t *parent,
+                                       const uint32_t *tokens_dev, float inv_t, uint64_t seed, uint64_t step,
+                                       uint32_t rows);
 // Tensor-parallel vocabulary: merges the ranks' statistics (all-gather) before the acceptance walk.
 ctox_status head_tp_merge_enqueue(ctox_ctx *ctx, uint32_t n_nodes, const int32_t *parent,
                                   const uint32_t *tokens_dev, uint32_t shard_rows);

@@ -1,0 +1,554 @@
+// Layer-stack models: weights, buffers and the pass (see stack.cuh).
+#include "stack.cuh"
+
+#include <algorithm>
+#include <cmath>
+
+#include "latent.cuh"
+
+namespace ctox {
+
+namespace {
+
+uint32_t round_up(uint32_t v, uint32_t to) { return (v + to - 1) / to * to; }
+
+ctox_status dense_alloc(ctox_exec *e, DenseMat *d, uint64_t rows, uint64_t cols) {
+    if (d->w) return CTOX_OK;
+    d->rows = (uint32_t)rows;
+    d->cols = (uint32_t)cols;
+    d->ld = round_up((uint32_t)cols, 8);
+    return xalloc(e, (void **)&d->w, (size_t)rows * d->ld * 2, false);
+}
+
+// One tensor as the file holds it, and where it goes.
+struct Placement {
+    uint64_t rows = 0, cols = 0;
+    struct To {
+        DenseMat *mat;
+        uint64_t mat_rows, mat_cols;  // of the whole destination
+        uint32_t row0;
+        PadAxis ra, ca;
+        uint32_t transpose_group, transpose_cols;
+        uint32_t fill_rows;  // rows a synthetic fill writes (0: all of the destination)
+    } to[2];
+    int n = 0;
+    uint64_t *loaded = nullptr;
+};
+PadAxis plain_axis(uint64_t n) { return PadAxis{(uint32_t)n, (uint32_t)n, 0, (uint32_t)n}; }
+PadAxis head_axis(uint32_t per_head, uint32_t padded) { return PadAxis{per_head, per_head, 0, padded}; }
+
+bool place(ctox_exec *e, uint32_t layer, uint32_t tensor, Placement *p) {
+    StackModel *s = e->stack;
+    const uint32_t H = s->c.hidden_size;
+    auto whole = [&](DenseMat *m, uint64_t rows, uint64_t cols) {
+        p->rows = rows;
+        p->cols = cols;
+        p->to[0] = {m, rows, cols, 0, plain_axis(rows), plain_axis(cols), 0, 0, 0};
+        p->n = 1;
+        return true;
+    };
+    if (layer == CTOX_LAYER_GLOBAL) {
+        p->loaded = &s->loaded;
+        if (tensor == CTOX_T_EMBED) return whole(&s->embed, s->c.vocab_size, H);
+        if (tensor == CTOX_T_LM_HEAD) return whole(&s->head, s->c.vocab_size, H);
+        return false;
+    }
+    if (layer >= s->layers.size()) return false;
+    StackLayer &L = s->layers[layer];
+    const ctox_layer_config &c = L.c;
+    p->loaded = &L.loaded;
+    const uint64_t fan_rows = (uint64_t)c.q_rank + (c.kv_from < 0 ? c.kv_rank + c.rot_dim : 0);
+    switch (tensor) {
+        case CTOX_T_Q_DOWN:
+            whole(&L.fan, c.q_rank, H);
+            p->to[0].mat_rows = fan_rows;
+            p->to[0].fill_rows = c.q_rank;
+            return true;
+        case CTOX_T_KV_DOWN:
+            if (c.kv_from >= 0) return false;
+            whole(&L.fan, c.kv_rank + c.rot_dim, H);
+            p->to[0].mat_rows = fan_rows;
+            p->to[0].row0 = c.q_rank;
+            p->to[0].fill_rows = c.kv_rank + c.rot_dim;
+            return true;
+        case CTOX_T_Q_UP:
+            whole(&L.q_up, (uint64_t)c.heads * (c.dim + c.rot_dim), c.q_rank);
+            p->to[0].mat_rows = (uint64_t)c.heads * L.head_w;
+            p->to[0].ra = PadAxis{c.dim + c.rot_dim, c.dim, L.dim_pad, L.head_w};
+            return true;
+        case CTOX_T_K_UP:
+            whole(&L.k_up_t, (uint64_t)c.heads * c.dim, c.kv_rank);
+            p->to[0].mat_rows = (uint64_t)c.heads * L.kv_pad;
+            p->to[0].mat_cols = L.dim_pad;
+            p->to[0].ra = head_axis(c.dim, L.dim_pad);
+            p->to[0].transpose_group = L.dim_pad;
+            p->to[0].transpose_cols = L.kv_pad;
+            if (s->pass_cap > kDensePass) {
+                p->to[1] = {&L.k_up, (uint64_t)c.heads * L.dim_pad, L.kv_pad, 0, head_axis(c.dim, L.dim_pad),
+                            plain_axis(c.kv_rank), 0, 0, 0};
+                p->n = 2;
+            }
+            return true;
+        case CTOX_T_V_UP:
+            whole(&L.v_up, (uint64_t)c.heads * c.vdim, c.kv_rank);
+            p->to[0].mat_rows = (uint64_t)c.heads * L.vdim_pad;
+            p->to[0].mat_cols = L.kv_pad;
+            p->to[0].ra = head_axis(c.vdim, L.vdim_pad);
+            return true;
+        case CTOX_T_ATTN_O:
+            whole(&L.o, H, (uint64_t)c.heads * c.vdim);
+            p->to[0].mat_cols = (uint64_t)c.heads * L.vdim_pad;
+            p->to[0].ca = head_axis(c.vdim, L.vdim_pad);
+            return true;
+        case CTOX_T_MLP_UP: return c.mlp != CTOX_MLP_NONE && whole(&L.up, c.ff, H);
+        case CTOX_T_MLP_DOWN: return c.mlp != CTOX_MLP_NONE && whole(&L.down, H, c.ff);
+        default: return false;
+    }
+}
+
+uint64_t bit(uint32_t tensor) { return 1ull << tensor; }
+
+uint64_t layer_needs(const ctox_layer_config &c) {
+    uint64_t m = bit(CTOX_T_INPUT_NORM) | bit(CTOX_T_MIX_OUT_NORM) | bit(CTOX_T_Q_DOWN) | bit(CTOX_T_Q_DOWN_NORM) |
+                 bit(CTOX_T_Q_UP) | bit(CTOX_T_K_UP) | bit(CTOX_T_V_UP) | bit(CTOX_T_ATTN_O);
+    if (c.kv_from < 0) m |= bit(CTOX_T_KV_DOWN) | bit(CTOX_T_KV_DOWN_NORM);
+    if (c.mlp != CTOX_MLP_NONE)
+        m |= bit(CTOX_T_POST_NORM) | bit(CTOX_T_MLP_OUT_NORM) | bit(CTOX_T_MLP_UP) | bit(CTOX_T_MLP_DOWN);
+    return m;
+}
+constexpr uint64_t kGlobalNeeds = (1ull << CTOX_T_EMBED) | (1ull << CTOX_T_LM_HEAD) | (1ull << CTOX_T_FINAL_NORM);
+
+}  // namespace
+
+ctox_status stack_create(ctox_ctx *ctx, const ctox_stack_config *c, const ctox_layer_config *layers, ctox_exec **out) {
+    if (ctx->tp_world > 1)
+        return fail(ctx, CTOX_UNSUPPORTED_OPERATION, "layer-stack models run on one GPU (the context has joined a group)");
+    if (!c->vocab_size || !c->hidden_size || !c->num_layers || !c->kv_page_tokens || c->max_context_tokens < 2 * kMaxPass ||
+        !(c->norm_eps >= 0.f) || !(c->logit_softcap >= 0.f))
+        return fail(ctx, CTOX_SHAPE, "layer stack: sizes, page and context must be set");
+    if (c->kv_dtype != CTOX_F32 && c->kv_dtype != CTOX_BF16)
+        return fail(ctx, CTOX_UNSUPPORTED_DTYPE, "layer stack: kv dtype %u", c->kv_dtype);
+    for (uint32_t l = 0; l < c->num_layers; ++l) {
+        const ctox_layer_config &y = layers[l];
+        if (y.mixer != CTOX_MIXER_LATENT_ATTENTION)
+            return fail(ctx, CTOX_UNSUPPORTED_OPERATION, "layer %u: unknown mixer %u", l, y.mixer);
+        if (y.mlp != CTOX_MLP_NONE && y.mlp != CTOX_MLP_RELU2)
+            return fail(ctx, CTOX_UNSUPPORTED_OPERATION, "layer %u: unknown feed-forward %u", l, y.mlp);
+        if (!y.heads || !y.dim || !y.vdim || !y.q_rank || !y.kv_rank || y.rot_dim % 2 || !(y.rope_base > 0.0) ||
+            !std::isfinite(y.score_scale) || (y.mlp != CTOX_MLP_NONE && !y.ff))
+            return fail(ctx, CTOX_SHAPE, "layer %u: unsupported latent-attention or feed-forward sizes", l);
+        if (y.kv_from >= 0) {
+            if ((uint32_t)y.kv_from >= l || layers[y.kv_from].kv_from >= 0)
+                return fail(ctx, CTOX_SHAPE, "layer %u: kv_from must name an earlier layer with its own cache", l);
+            const ctox_layer_config &o = layers[y.kv_from];
+            if (o.kv_rank != y.kv_rank || o.rot_dim != y.rot_dim || o.rope_base != y.rope_base)
+                return fail(ctx, CTOX_SHAPE, "layer %u: latent and rotation differ from those of layer %d", l, y.kv_from);
+        }
+    }
+    ctox_exec *e = new ctox_exec();
+    StackModel *s = new StackModel();
+    e->ctx = ctx;
+    e->stack = s;
+    s->c = *c;
+    s->pass_cap = kDensePass;
+    s->layers.resize(c->num_layers);
+    for (uint32_t l = 0; l < c->num_layers; ++l) {
+        StackLayer &L = s->layers[l];
+        L.c = layers[l];
+        L.owner = L.c.kv_from < 0 ? l : (uint32_t)L.c.kv_from;
+        L.dim_pad = round_up(L.c.dim, 16);
+        L.rot_pad = round_up(L.c.rot_dim, 16);
+        L.vdim_pad = round_up(L.c.vdim, 16);
+        L.kv_pad = round_up(L.c.kv_rank, 16);
+        L.head_w = L.dim_pad + L.rot_pad;
+    }
+    // what the executor's own calls read of the model
+    e->cfg.vocab_size = c->vocab_size;
+    e->cfg.hidden_size = c->hidden_size;
+    e->cfg.num_hidden_layers = c->num_layers;
+    e->cfg.max_context_tokens = c->max_context_tokens;
+    e->cfg.kv_page_tokens = c->kv_page_tokens;
+    e->cfg.kv_dtype = c->kv_dtype;
+    e->n_layers = c->num_layers;
+    e->vocab_l = c->vocab_size;
+    *out = e;
+    return CTOX_OK;
+}
+
+void stack_destroy(ctox_exec *e) {
+    delete e->stack;
+    e->stack = nullptr;
+}
+
+ctox_status stack_load_matrix(ctox_exec *e, uint32_t layer, uint32_t tensor, const ctox_fused_matvec_op *op) {
+    ctox_ctx *ctx = e->ctx;
+    CTOX_CUDA(ctx, cudaSetDevice(ctx->device));
+    Placement p;
+    if (!place(e, layer, tensor, &p))
+        return fail(ctx, CTOX_INVALID_ARTIFACT, "tensor %u is not a matrix of layer %u", tensor, layer);
+    if (op->rows != p.rows || op->columns != p.cols)
+        return fail(ctx, CTOX_SHAPE, "tensor %u of layer %u is %llux%llu, expected %llux%llu", tensor, layer,
+                    (unsigned long long)op->rows, (unsigned long long)op->columns, (unsigned long long)p.rows,
+                    (unsigned long long)p.cols);
+    if (op->dtype != CTOX_BF16 || op->weights_len != p.rows * p.cols * 2 || !op->weights)
+        return fail(ctx, CTOX_UNSUPPORTED_DTYPE, "matrices of a layer stack are dense bf16 rows");
+    if (op->activation != CTOX_ACT_IDENTITY || op->bias || op->s_in || op->s_out)
+        return fail(ctx, CTOX_UNSUPPORTED_OPERATION, "matrices of a layer stack carry no bias, scales or activation");
+    __nv_bfloat16 *tmp = nullptr;
+    ctox_status rc = dev_alloc(ctx, (void **)&tmp, op->weights_len);
+    if (rc) return rc;
+    auto upload = [&]() -> ctox_status {
+        CTOX_CUDA(ctx, cudaMemcpyAsync(tmp, op->weights, op->weights_len, cudaMemcpyHostToDevice, ctx->stream));
+        for (int i = 0; i < p.n; ++i) {
+            const Placement::To &t = p.to[i];
+            EX(dense_alloc(e, t.mat, t.mat_rows, t.mat_cols));
+            EX(launch_relayout(ctx, tmp, (uint32_t)p.rows, (uint32_t)p.cols, t.ra, t.ca,
+                               t.mat->w + (size_t)t.row0 * t.mat->ld, t.mat->ld, t.transpose_group, t.transpose_cols));
+        }
+        CTOX_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+        return CTOX_OK;
+    };
+    rc = upload();
+    dev_free(ctx, tmp, op->weights_len);
+    if (rc) return rc;
+    *p.loaded |= bit(tensor);
+    e->warmed = false;
+    return CTOX_OK;
+}
+
+bool stack_vector_slot(ctox_exec *e, uint32_t layer, uint32_t tensor, float ***slot, uint64_t *n, uint64_t **loaded) {
+    StackModel *s = e->stack;
+    *n = s->c.hidden_size;
+    if (layer == CTOX_LAYER_GLOBAL) {
+        *loaded = &s->loaded;
+        *slot = &s->final_norm;
+        return tensor == CTOX_T_FINAL_NORM;
+    }
+    if (layer >= s->layers.size()) return false;
+    StackLayer &L = s->layers[layer];
+    *loaded = &L.loaded;
+    switch (tensor) {
+        case CTOX_T_INPUT_NORM: *slot = &L.norm1; return true;
+        case CTOX_T_MIX_OUT_NORM: *slot = &L.norm1b; return true;
+        case CTOX_T_POST_NORM: *slot = &L.norm2; return L.c.mlp != CTOX_MLP_NONE;
+        case CTOX_T_MLP_OUT_NORM: *slot = &L.norm2b; return L.c.mlp != CTOX_MLP_NONE;
+        case CTOX_T_Q_DOWN_NORM: *slot = &L.q_norm; *n = L.c.q_rank; return true;
+        case CTOX_T_KV_DOWN_NORM: *slot = &L.kv_norm; *n = L.c.kv_rank; return L.c.kv_from < 0;
+        default: return false;
+    }
+}
+
+ctox_status stack_fill_synthetic(ctox_exec *e, uint64_t seed) {
+    ctox_ctx *ctx = e->ctx;
+    StackModel *s = e->stack;
+    uint64_t sd = seed * 1000003ull + 29;
+    auto fill = [&](uint32_t layer, uint32_t tensor) -> ctox_status {
+        Placement p;
+        if (!place(e, layer, tensor, &p)) return CTOX_OK;
+        for (int i = 0; i < p.n; ++i) {
+            const Placement::To &t = p.to[i];
+            EX(dense_alloc(e, t.mat, t.mat_rows, t.mat_cols));
+            const uint64_t rows = t.fill_rows ? t.fill_rows : t.mat_rows;
+            sd = sd * 6364136223846793005ull + 1442695040888963407ull;
+            EX(launch_fill_normal_bf16(ctx, t.mat->w + (size_t)t.row0 * t.mat->ld, rows * t.mat->ld,
+                                       1.0f / std::sqrt((float)p.cols), sd));
+        }
+        *p.loaded |= bit(tensor);
+        return CTOX_OK;
+    };
+    auto ones = [&](uint32_t layer, uint32_t tensor) -> ctox_status {
+        float **slot = nullptr;
+        uint64_t n = 0, *loaded = nullptr;
+        if (!stack_vector_slot(e, layer, tensor, &slot, &n, &loaded)) return CTOX_OK;
+        if (!*slot) EX(xalloc(e, (void **)slot, n * 4, false));
+        const std::vector<float> v(n, 1.0f);
+        CTOX_CUDA(ctx, cudaMemcpyAsync(*slot, v.data(), n * 4, cudaMemcpyHostToDevice, ctx->stream));
+        CTOX_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+        *loaded |= bit(tensor);
+        return CTOX_OK;
+    };
+    for (uint32_t t : {CTOX_T_EMBED, CTOX_T_LM_HEAD}) EX(fill(CTOX_LAYER_GLOBAL, t));
+    EX(ones(CTOX_LAYER_GLOBAL, CTOX_T_FINAL_NORM));
+    for (uint32_t l = 0; l < s->layers.size(); ++l) {
+        for (uint32_t t : {CTOX_T_Q_DOWN, CTOX_T_KV_DOWN, CTOX_T_Q_UP, CTOX_T_K_UP, CTOX_T_V_UP, CTOX_T_ATTN_O,
+                           CTOX_T_MLP_UP, CTOX_T_MLP_DOWN})
+            EX(fill(l, t));
+        for (uint32_t t : {CTOX_T_INPUT_NORM, CTOX_T_MIX_OUT_NORM, CTOX_T_POST_NORM, CTOX_T_MLP_OUT_NORM,
+                           CTOX_T_Q_DOWN_NORM, CTOX_T_KV_DOWN_NORM})
+            EX(ones(l, t));
+    }
+    CTOX_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+    e->warmed = false;
+    return CTOX_OK;
+}
+
+namespace {
+
+LatentAttn latent_args(const ctox_exec *e, const StackLayer &L, uint32_t m, uint32_t pos0) {
+    const StackModel *s = e->stack;
+    const StackLayer &O = s->layers[L.owner];
+    LatentAttn a{};
+    a.q_abs = s->q_abs;
+    a.q_rot = s->q + L.dim_pad;
+    a.q_stride = L.head_w;
+    a.cache = O.cache;
+    a.bf16 = s->c.kv_dtype == CTOX_BF16;
+    a.page_table = O.page_table;
+    a.page_tokens = s->c.kv_page_tokens;
+    a.heads = L.c.heads;
+    a.kv_pad = L.kv_pad;
+    a.rot_pad = L.rot_pad;
+    a.pos0 = pos0;
+    a.m = m;
+    a.window = L.c.window;
+    a.scale = L.c.score_scale;
+    a.ws_o = s->ws_o;
+    a.ws_ml = s->ws_ml;
+    return a;
+}
+
+}  // namespace
+
+ctox_status stack_warmup(ctox_exec *e) {
+    ctox_ctx *ctx = e->ctx;
+    StackModel *s = e->stack;
+    const ctox_stack_config &c = s->c;
+    if ((s->loaded & kGlobalNeeds) != kGlobalNeeds)
+        return fail(ctx, CTOX_INVALID_STATE, "warmup: embedding, lm_head or final norm missing");
+    for (uint32_t l = 0; l < s->layers.size(); ++l) {
+        const uint64_t need = layer_needs(s->layers[l].c);
+        if ((s->layers[l].loaded & need) != need)
+            return fail(ctx, CTOX_INVALID_STATE, "warmup: layer %u has missing tensors (mask %llx)", l,
+                        (unsigned long long)(need & ~s->layers[l].loaded));
+    }
+    if (s->x[0]) return CTOX_OK;
+    const uint64_t H = c.hidden_size, P = s->pass_cap, S = kDensePass;
+    uint64_t fan_w = 0, q_w = 0, abs_w = 0, att_w = 0, ff = 1, ws_o = 0, ws_ml = 0;
+    for (StackLayer &L : s->layers) {
+        fan_w = std::max<uint64_t>(fan_w, L.fan.rows);
+        q_w = std::max<uint64_t>(q_w, (uint64_t)L.c.heads * L.head_w);
+        abs_w = std::max<uint64_t>(abs_w, (uint64_t)L.c.heads * L.kv_pad);
+        att_w = std::max<uint64_t>(att_w, (uint64_t)L.c.heads * L.vdim_pad);
+        ff = std::max<uint64_t>(ff, L.c.mlp != CTOX_MLP_NONE ? L.c.ff : 1);
+        for (uint32_t m = 1; m <= S; ++m) {
+            LatentAttn a = latent_args(e, L, m, c.max_context_tokens);
+            const uint64_t rows = (uint64_t)latent_attn_splits(ctx, a) * m * L.c.heads;
+            ws_o = std::max<uint64_t>(ws_o, rows * L.kv_pad);
+            ws_ml = std::max<uint64_t>(ws_ml, rows * 2);
+        }
+        const uint32_t pairs = std::max<uint32_t>(L.c.rot_dim / 2, 1);
+        std::vector<float> freq(pairs, 0.f);
+        for (uint32_t i = 0; i < L.c.rot_dim / 2; ++i)
+            freq[i] = (float)std::pow(L.c.rope_base, -2.0 * (double)i / (double)L.c.rot_dim);
+        EX(xalloc(e, (void **)&L.freq, pairs * 4, false));
+        CTOX_CUDA(ctx, cudaMemcpyAsync(L.freq, freq.data(), pairs * 4, cudaMemcpyHostToDevice, ctx->stream));
+        CTOX_CUDA(ctx, cudaStreamSynchronize(ctx->stream));  // `freq` is a local
+    }
+#define WALLOC(ptr, bytes) EX(xalloc(e, (void **)&(ptr), (bytes), true))
+    WALLOC(s->x[0], P * H * 4);
+    WALLOC(s->x[1], P * H * 4);
+    WALLOC(s->y, P * H * 4);
+    WALLOC(s->fan, P * fan_w * 4);
+    WALLOC(s->q, S * q_w * 4);
+    WALLOC(s->q_abs, S * abs_w * 4);
+    WALLOC(s->att, S * att_w * 4);
+    WALLOC(s->u, S * ff * 4);
+    WALLOC(s->ws_o, ws_o * 4);
+    WALLOC(s->ws_ml, ws_ml * 4);
+    WALLOC(s->rows_dev, P * 4);
+    WALLOC(e->tokens_dev, (P + 1) * 4);
+    WALLOC(e->hist_hidden, kMaxPass * H * 4);
+    s->head_rows = (uint32_t)S;
+    WALLOC(s->head_in, S * H * 4);
+    WALLOC(e->logits, (size_t)s->head_rows * c.vocab_size * 4);
+    // caches: a ring of pages that holds the widest window read from it and one pass
+    const uint32_t pt = c.kv_page_tokens, pages_total = (c.max_context_tokens + pt - 1) / pt;
+    for (uint32_t l = 0; l < s->layers.size(); ++l) {
+        StackLayer &O = s->layers[l];
+        if (O.owner != l) continue;
+        uint64_t reach = 0;
+        for (const StackLayer &L : s->layers)
+            if (L.owner == l) reach = std::max<uint64_t>(reach, L.c.window ? L.c.window : c.max_context_tokens);
+        const uint32_t ring = (uint32_t)std::min<uint64_t>(pages_total, (reach + P + pt - 1) / pt + 1);
+        O.slots = ring * pt;
+        WALLOC(O.cache, (size_t)O.slots * (O.kv_pad + O.rot_pad) * (c.kv_dtype == CTOX_BF16 ? 2 : 4));
+        WALLOC(O.page_table, (size_t)pages_total * 4);
+        std::vector<uint32_t> table(pages_total);
+        for (uint32_t p = 0; p < pages_total; ++p) table[p] = p % ring;
+        CTOX_CUDA(ctx, cudaMemcpyAsync(O.page_table, table.data(), (size_t)pages_total * 4, cudaMemcpyHostToDevice, ctx->stream));
+        CTOX_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+    }
+#undef WALLOC
+    return CTOX_OK;
+}
+
+ctox_status stack_prefill_synthetic(ctox_exec *e, uint64_t n, uint64_t seed) {
+    ctox_ctx *ctx = e->ctx;
+    StackModel *s = e->stack;
+    uint64_t sd = seed + 1;
+    if (s->c.kv_dtype != CTOX_BF16)
+        return fail(ctx, CTOX_UNSUPPORTED_OPERATION, "synthetic prefill of a layer stack needs a bf16 cache");
+    for (StackLayer &L : s->layers) {
+        if (!L.cache) continue;
+        sd = sd * 6364136223846793005ull + 1442695040888963407ull;
+        EX(launch_fill_normal_bf16(ctx, (__nv_bfloat16 *)L.cache, (uint64_t)L.slots * (L.kv_pad + L.rot_pad), 1.f, sd));
+    }
+    (void)n;
+    return CTOX_OK;
+}
+
+ctox_status stack_keep_streams(ctox_exec *e) {
+    StackModel *s = e->stack;
+    if (s->streams) return CTOX_OK;
+    return xalloc(e, (void **)&s->streams,
+                  (size_t)s->layers.size() * s->c.max_context_tokens * s->c.hidden_size * 4, true);
+}
+
+// ------------------------------------------------------------------ passes
+namespace {
+
+VecIn vec_plain(const float *x, uint32_t stride, uint32_t cols) {
+    VecIn v{};
+    v.x = x;
+    v.x_stride = stride;
+    v.cols = cols;
+    return v;
+}
+VecOut vec_out(float *y, uint32_t stride, int kind = OUT_PLAIN) {
+    VecOut o{};
+    o.y = y;
+    o.y_stride = stride;
+    o.kind = kind;
+    return o;
+}
+
+// The stream with the last sublayer's output added (its layer norm applied), normalised by w: the prologue
+// of the next product. The updated stream goes to the other buffer.
+VecIn stream_in(StackModel *s, const float *w) {
+    VecIn v = vec_plain(s->x[s->cur], s->c.hidden_size, s->c.hidden_size);
+    v.norm = NORM_LAYER;
+    v.w = w;
+    v.eps = s->c.norm_eps;
+    if (s->y_norm) {
+        v.y = s->y;
+        v.y_stride = s->c.hidden_size;
+        v.wb = s->y_norm;
+        v.x_out = s->x[s->cur ^ 1];
+        s->cur ^= 1;
+        s->y_norm = nullptr;
+    }
+    return v;
+}
+
+LatentAppend append_args(const ctox_exec *e, const StackLayer &L, uint32_t pos0) {
+    const StackModel *s = e->stack;
+    return LatentAppend{s->fan, L.fan.rows, L.c.q_rank, L.c.kv_rank, L.c.rot_dim, L.kv_pad, L.rot_pad, L.kv_norm,
+                        s->c.norm_eps, L.cache, s->c.kv_dtype == CTOX_BF16, L.page_table, s->c.kv_page_tokens, pos0,
+                        L.freq};
+}
+
+// One layer for up to kDensePass positions, eight kernels: down projections (residual add and norms in
+// their prologue), query up projection (norm in its prologue, rotation in its epilogue, cache append in
+// its extra CTAs), queries into the latent space, attention, values (merge of the splits in the prologue),
+// output projection, feed-forward up and down.
+ctox_status layer_short(ctox_exec *e, uint32_t l, uint32_t m, uint32_t pos0) {
+    ctox_ctx *ctx = e->ctx;
+    StackModel *s = e->stack;
+    StackLayer &L = s->layers[l];
+    const ctox_layer_config &c = L.c;
+    const uint32_t H = s->c.hidden_size, qw = c.heads * L.head_w, vw = c.heads * L.vdim_pad;
+    EX(launch_dense_matvec(ctx, L.fan, 1, m, stream_in(s, L.norm1), vec_out(s->fan, L.fan.rows), nullptr));
+    VecIn in = vec_plain(s->fan, L.fan.rows, c.q_rank);
+    in.norm = NORM_RMS;
+    in.w = L.q_norm;
+    in.eps = s->c.norm_eps;
+    VecOut out = vec_out(s->q, qw, OUT_ROPE);
+    out.head_width = L.head_w;
+    out.rope0 = L.dim_pad;
+    out.rope_dims = c.rot_dim;
+    out.pos0 = pos0;
+    out.freq = L.freq;
+    const LatentAppend ap = append_args(e, L, pos0);
+    EX(launch_dense_matvec(ctx, L.q_up, 1, m, in, out, L.owner == l ? &ap : nullptr));
+    in = vec_plain(s->q, qw, L.dim_pad);
+    in.x_group = L.head_w;
+    EX(launch_dense_matvec(ctx, L.k_up_t, c.heads, m, in, vec_out(s->q_abs, c.heads * L.kv_pad), nullptr));
+    const LatentAttn a = latent_args(e, L, m, pos0);
+    const uint32_t splits = latent_attn_splits(ctx, a);
+    EX(launch_latent_attention(ctx, a, splits));
+    in = VecIn{};
+    in.cols = L.kv_pad;
+    in.ws_o = s->ws_o;
+    in.ws_ml = s->ws_ml;
+    in.splits = splits;
+    in.ws_rows = m * c.heads;
+    in.groups = c.heads;
+    EX(launch_dense_matvec(ctx, L.v_up, c.heads, m, in, vec_out(s->att, vw), nullptr));
+    EX(launch_dense_matvec(ctx, L.o, 1, m, vec_plain(s->att, vw, vw), vec_out(s->y, H), nullptr));
+    s->y_norm = L.norm1b;
+    if (c.mlp != CTOX_MLP_NONE) {
+        EX(launch_dense_matvec(ctx, L.up, 1, m, stream_in(s, L.norm2), vec_out(s->u, c.ff, OUT_RELU2), nullptr));
+        EX(launch_dense_matvec(ctx, L.down, 1, m, vec_plain(s->u, c.ff, c.ff), vec_out(s->y, H), nullptr));
+        s->y_norm = L.norm2b;
+    }
+    return CTOX_OK;
+}
+
+StreamNorm stream_norm(const StackModel *s, const float *w) {
+    StreamNorm n{};
+    n.x = s->x[s->cur];
+    n.y = s->y_norm ? s->y : nullptr;
+    n.wb = s->y_norm;
+    n.w = w;
+    n.eps = s->c.norm_eps;
+    n.width = s->c.hidden_size;
+    return n;
+}
+
+}  // namespace
+
+ctox_status stack_pass(ctox_exec *e, uint32_t m, uint64_t pos0) {
+    ctox_ctx *ctx = e->ctx;
+    StackModel *s = e->stack;
+    const uint32_t H = s->c.hidden_size;
+    s->cur = 0;
+    s->y_norm = nullptr;
+    EX(launch_embed_dense(ctx, s->embed.w, s->embed.ld, e->tokens_dev, H, m, s->x[0]));
+    for (uint32_t l = 0; l < s->layers.size(); ++l) {
+        EX(layer_short(e, l, m, (uint32_t)pos0));
+        if (s->streams) {  // evidence: the stream after this layer
+            StreamNorm n = stream_norm(s, nullptr);
+            n.x_out = s->streams + ((size_t)l * s->c.max_context_tokens + pos0) * H;
+            EX(launch_stream_norm(ctx, n, m));
+        }
+    }
+    StreamNorm n = stream_norm(s, s->final_norm);
+    n.x += (size_t)(m - 1) * H;
+    if (n.y) n.y += (size_t)(m - 1) * H;
+    n.f32_out = e->hist_hidden;
+    return launch_stream_norm(ctx, n, 1);
+}
+
+ctox_status stack_head_last(ctox_exec *e) {
+    StackModel *s = e->stack;
+    VecOut out = vec_out(e->logits, s->c.vocab_size, s->c.logit_softcap > 0.f ? OUT_SOFTCAP : OUT_PLAIN);
+    out.cap = s->c.logit_softcap;
+    return launch_dense_matvec(e->ctx, s->head, 1, 1, vec_plain(e->hist_hidden, s->c.hidden_size, s->c.hidden_size), out,
+                               nullptr);
+}
+
+ctox_status stack_head_rows(ctox_exec *e, const uint32_t *rows, uint32_t n) {
+    ctox_ctx *ctx = e->ctx;
+    StackModel *s = e->stack;
+    const uint32_t H = s->c.hidden_size;
+    CTOX_CUDA(ctx, cudaMemcpyAsync(s->rows_dev, rows, n * 4, cudaMemcpyHostToDevice, ctx->stream));
+    StreamNorm a = stream_norm(s, s->final_norm);
+    a.rows = s->rows_dev;
+    a.f32_out = s->head_in;
+    EX(launch_stream_norm(ctx, a, n));
+    VecOut out = vec_out(e->logits, s->c.vocab_size, s->c.logit_softcap > 0.f ? OUT_SOFTCAP : OUT_PLAIN);
+    out.cap = s->c.logit_softcap;
+    return launch_dense_matvec(ctx, s->head, 1, n, vec_plain(s->head_in, H, H), out, nullptr);
+}
+
+}  // namespace ctox

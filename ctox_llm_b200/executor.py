@@ -11,7 +11,7 @@ from __future__ import annotations
 
 import ctypes as C
 from dataclasses import dataclass
-from typing import List, Optional, Sequence
+from typing import Iterator, List, Optional, Sequence
 
 import numpy as np
 
@@ -55,6 +55,28 @@ def qwen38_27b_config(**overrides) -> N.ModelConfig:
 
 
 @dataclass
+class StackConfig:
+    """A model described layer by layer (ctox_stack_config plus its ctox_layer_config list)."""
+
+    vocab_size: int
+    hidden_size: int
+    layers: List[N.LayerConfig]
+    norm_eps: float
+    logit_softcap: float
+    max_context_tokens: int
+    kv_page_tokens: int = 128
+    kv_dtype: int = N.BF16
+    pass_tokens: int = 0
+    mtp_num_hidden_layers: int = 0  # such a model has no MTP layer
+
+    def create(self, backend: B200Backend, handle) -> int:
+        c = N.StackConfigC(self.vocab_size, self.hidden_size, len(self.layers), self.norm_eps, self.logit_softcap,
+                           self.max_context_tokens, self.kv_page_tokens, self.kv_dtype, self.pass_tokens)
+        layers = (N.LayerConfig * len(self.layers))(*self.layers)
+        return backend._lib.ctox_exec_create_stack(backend._ctx, C.byref(c), layers, C.byref(handle))
+
+
+@dataclass
 class GeneratedBlock:
     """One decode call: engine.rs GeneratedStep / ResolvedGreedyMtpVerification."""
 
@@ -71,12 +93,19 @@ class GeneratedBlock:
 
 
 class B200Executor:
-    def __init__(self, backend: B200Backend, config: N.ModelConfig):
+    """One model and one session. config: ModelConfig (the hybrid model) or StackConfig."""
+
+    _h = None
+
+    def __init__(self, backend: B200Backend, config):
         self._b = backend
         self._lib = backend._lib
         self.config = config
         handle = C.c_void_p()
-        backend._check(self._lib.ctox_exec_create(backend._ctx, C.byref(config), C.byref(handle)))
+        if isinstance(config, StackConfig):
+            backend._check(config.create(backend, handle))
+        else:
+            backend._check(self._lib.ctox_exec_create(backend._ctx, C.byref(config), C.byref(handle)))
         self._h = handle
 
     # -- load ------------------------------------------------------------------------------
@@ -101,6 +130,44 @@ class B200Executor:
         t = np.ascontiguousarray(tokens, dtype=np.uint32)
         self._b._check(self._lib.ctox_exec_prefill(self._h, t.ctypes.data_as(C.c_void_p), t.size,
                                                    _cancel_ptr(cancellation)))
+
+    def extend(self, tokens: Sequence[int], want: Sequence[int] = (),
+               cancellation: Optional[CancellationToken] = None) -> np.ndarray:
+        """Consumes more tokens at the current position; returns the logits [len(want), vocab] at the
+        wanted places (ascending, counted from the first of these tokens)."""
+        t = np.ascontiguousarray(tokens, dtype=np.uint32)
+        w = np.ascontiguousarray(want, dtype=np.uint32)
+        out = np.zeros((w.size, self.config.vocab_size), dtype=np.float32)
+        self._b._check(self._lib.ctox_exec_extend(
+            self._h, t.ctypes.data_as(C.c_void_p), t.size, w.ctypes.data_as(C.c_void_p) if w.size else None, w.size,
+            out.ctypes.data_as(C.c_void_p) if w.size else None, _cancel_ptr(cancellation)))
+        return out
+
+    def generate(self, prompt: Sequence[int], max_new_tokens: int, temperature: float = 0.0, top_k: int = 0,
+                 top_p: float = 1.0, seed: int = 0, stop_tokens: Sequence[int] = (),
+                 cancellation: Optional[CancellationToken] = None) -> Iterator[int]:
+        """Prefills the prompt and yields up to max_new_tokens tokens. temperature 0 is greedy; otherwise
+        tokens follow softmax(logits / temperature), drawn on the device, or with top_k in 1..1024 among
+        the top_k best inside the top_p nucleus. Models with an MTP layer emit speculative blocks."""
+        self.prefill(prompt, cancellation)
+        restricted = temperature > 0.0 and top_k > 0
+        draws = np.random.Generator(np.random.Philox(key=[seed, 0]))
+        if restricted:
+            self.keep_logits(True)
+        mtp = self.config.mtp_num_hidden_layers > 0 and not restricted
+        token, produced = int(prompt[-1]), 0
+        while produced < max_new_tokens:
+            block = self.decode(token, mtp_enabled=mtp, temperature=0.0 if restricted else temperature, seed=seed,
+                                cancellation=cancellation)
+            emitted = block.emitted
+            if restricted:
+                draw = float(draws.integers(0, 1 << 24)) / (1 << 24)
+                emitted = [self.select_target_token(temperature, top_k, top_p, draw)]
+            for token in emitted:
+                yield int(token)
+                produced += 1
+                if produced >= max_new_tokens or token in stop_tokens:
+                    return
 
     def prefill_synthetic(self, n: int, seed: int = 0) -> None:
         self._b._check(self._lib.ctox_exec_prefill_synthetic(self._h, n, seed))
@@ -178,6 +245,15 @@ class B200Executor:
         out = np.zeros(self.config.vocab_size // self._b.tp_world, dtype=np.float32)
         self._b._check(self._lib.ctox_exec_last_logits(self._h, position,
                                                        out.ctypes.data_as(C.c_void_p)))
+        return out
+
+    def keep_streams(self) -> None:
+        """Keeps the residual stream after every layer (layer-stack models)."""
+        self._b._check(self._lib.ctox_exec_keep_streams(self._h))
+
+    def last_stream(self, layer: int, position: int, n: int) -> np.ndarray:
+        out = np.zeros((n, self.config.hidden_size), dtype=np.float32)
+        self._b._check(self._lib.ctox_exec_last_stream(self._h, layer, position, n, out.ctypes.data_as(C.c_void_p)))
         return out
 
     def last_mtp_hidden(self) -> np.ndarray:

@@ -391,10 +391,56 @@ enum {
     CTOX_T_MTP_NORM_E = 18,    /* global, vector hidden (pre_fc_norm_embedding) */
     CTOX_T_MTP_NORM_H = 19,    /* global, vector hidden (pre_fc_norm_hidden) */
     CTOX_T_MTP_NORM = 20,      /* global, vector hidden (mtp.norm) */
-    CTOX_T_DRAFT_IDS = 21      /* global, draft_vocab strictly increasing token ids (as uint32) */
+    CTOX_T_DRAFT_IDS = 21,     /* global, draft_vocab strictly increasing token ids (as uint32) */
+    /* layer-stack models (ctox_exec_create_stack); matrices are dense CTOX_BF16 rows. They also use
+     * EMBED, LM_HEAD, FINAL_NORM, INPUT_NORM (before the mixer), POST_NORM (before the feed-forward),
+     * ATTN_O (hidden x heads*vdim) and MLP_DOWN (hidden x ff). */
+    CTOX_T_Q_DOWN = 22,        /* layer, matrix q_rank x hidden */
+    CTOX_T_Q_DOWN_NORM = 23,   /* layer, vector q_rank */
+    CTOX_T_Q_UP = 24,          /* layer, matrix heads*(dim+rot_dim) x q_rank, per head [dim | rot_dim] */
+    CTOX_T_KV_DOWN = 25,       /* layer with its own cache, matrix (kv_rank+rot_dim) x hidden */
+    CTOX_T_KV_DOWN_NORM = 26,  /* layer with its own cache, vector kv_rank */
+    CTOX_T_K_UP = 27,          /* layer, matrix heads*dim x kv_rank */
+    CTOX_T_V_UP = 28,          /* layer, matrix heads*vdim x kv_rank */
+    CTOX_T_MIX_OUT_NORM = 29,  /* layer, vector hidden (after the mixer) */
+    CTOX_T_MLP_UP = 30,        /* layer, matrix ff x hidden */
+    CTOX_T_MLP_OUT_NORM = 31   /* layer, vector hidden (after the feed-forward) */
 };
 #define CTOX_LAYER_GLOBAL 0xffffffffu
 /* layer index of the MTP decoder layer = num_hidden_layers */
+
+/* ---- models described layer by layer (no counterpart in the reference) ----
+ * Every layer is x += norm(mixer(norm(x))), then, with a feed-forward, x += norm(ff(norm(x))); the
+ * norms are layer norms with a weight. They run through the same executor calls as the hybrid model:
+ * prefill, extend, decode, select_target, evidence. One GPU, no MTP layer. */
+enum { CTOX_MIXER_LATENT_ATTENTION = 1 };
+enum { CTOX_MLP_NONE = 0, CTOX_MLP_RELU2 = 1 /* down(relu(up x)^2) */ };
+
+/* Latent attention: queries through a q_rank latent with an RMS norm; keys and values of all heads are
+ * made from one cached row per token, an RMS-normed latent of kv_rank values and a rotated key part of
+ * rot_dim values (interleaved pairs, base rope_base). kv_from >= 0 reads the cache of that earlier layer
+ * (same kv_rank, rot_dim and rope_base) instead of writing its own. */
+typedef struct {
+    double rope_base;
+    uint32_t mixer;  /* CTOX_MIXER_* */
+    uint32_t heads, dim, rot_dim, vdim, q_rank, kv_rank;
+    uint32_t window; /* a token sees itself and window - 1 tokens before it; 0: all of them */
+    int32_t kv_from; /* -1: own cache */
+    float score_scale;
+    uint32_t mlp; /* CTOX_MLP_* */
+    uint32_t ff;
+} ctox_layer_config;
+
+typedef struct {
+    uint32_t vocab_size, hidden_size, num_layers;
+    float norm_eps;
+    float logit_softcap; /* logits = cap * tanh(logits / cap); 0: none */
+    uint32_t max_context_tokens;
+    uint32_t kv_page_tokens;
+    uint32_t kv_dtype;    /* CTOX_BF16: 16-bit products; CTOX_F32: everything in 32-bit, passes of 8 tokens */
+    uint32_t pass_tokens; /* most prompt tokens of one pass (0: a default); cached pages cover the widest
+                             window and one pass */
+} ctox_stack_config;
 
 /* One speculative block (engine.rs:110-116 ResolvedGreedyMtpVerification). */
 typedef struct {
@@ -408,9 +454,13 @@ typedef struct {
 } ctox_exec_step;
 
 ctox_status ctox_exec_create(ctox_ctx *ctx, const ctox_model_config *config, ctox_exec **out);
+/* A layer-stack model: config->num_layers layer descriptions. Not available in a tensor-parallel group. */
+ctox_status ctox_exec_create_stack(ctox_ctx *ctx, const ctox_stack_config *config,
+                                   const ctox_layer_config *layers, ctox_exec **out);
 ctox_status ctox_exec_destroy(ctox_exec *exec); /* unload: frees every allocation */
 /* load(): one tensor at a time, host memory. Matrices are FusedMatVec descriptions
- * without input (weights, s_in, s_out, optional bias). */
+ * without input (weights, s_in, s_out, optional bias); those of a layer stack are dense: dtype CTOX_BF16,
+ * row-major weights, no scales. */
 ctox_status ctox_exec_load_matrix(ctox_exec *exec, uint32_t layer, uint32_t tensor,
                                   const ctox_fused_matvec_op *op);
 ctox_status ctox_exec_load_vector(ctox_exec *exec, uint32_t layer, uint32_t tensor, const float *values,
@@ -432,6 +482,13 @@ ctox_status ctox_exec_reset_session(ctox_exec *exec);
  * the last token is NOT consumed: it is the input of the first decode. */
 ctox_status ctox_exec_prefill(ctox_exec *exec, const uint32_t *tokens, uint64_t n,
                               const volatile int32_t *cancel);
+/* Consumes `n` more tokens at the current position, in passes, on top of what the session holds (which
+ * may be nothing: position 0 after reset_session). `want` names `n_want` of them, ascending places 0 ..
+ * n-1, whose logits are copied to logits_out [n_want][vocab_size] (host memory; both NULL with n_want 0).
+ * prefill() is a reset and this over all tokens but the last. Not while a speculative block is pending,
+ * and not in a tensor-parallel group when logits are wanted. */
+ctox_status ctox_exec_extend(ctox_exec *exec, const uint32_t *tokens, uint64_t n, const uint32_t *want,
+                             uint64_t n_want, float *logits_out, const volatile int32_t *cancel);
 /* Benchmark prefill: fills `n` cache positions with random K/V ~ N(0,1) and random
  * recurrent state instead of running the model, and sets the position. */
 ctox_status ctox_exec_prefill_synthetic(ctox_exec *exec, uint64_t n, uint64_t seed);
@@ -493,6 +550,11 @@ ctox_status ctox_exec_last_logits(ctox_exec *exec, uint32_t position, float *out
 ctox_status ctox_exec_last_mtp_hidden(ctox_exec *exec, uint32_t index, float *out, uint32_t *count);
 ctox_status ctox_exec_last_draft_logits(ctox_exec *exec, uint32_t draft, float *out, uint32_t *rows,
                                         uint32_t *count);
+/* Evidence of a layer stack: once enabled, the residual stream after every layer is kept for every
+ * position ([layer][max_context_tokens][hidden] floats of device memory). _last_stream copies `n`
+ * positions from `position` on. */
+ctox_status ctox_exec_keep_streams(ctox_exec *exec);
+ctox_status ctox_exec_last_stream(ctox_exec *exec, uint32_t layer, uint64_t position, uint64_t n, float *out);
 /* ModelExecutor::select_target_token (engine.rs:322-362): samples the target token of verify
  * position `position` of the last decode call from the logits the executor kept on the device
  * (ctox_exec_keep_logits must be on), with the same rules as ctox_sample_topk_topp. In a
