@@ -68,6 +68,12 @@ inline ctox_status fail(ctox_ctx *ctx, ctox_status code, const char *fmt, ...) {
                               cudaGetErrorString(e_));                                    \
     } while (0)
 
+#define EX(expr)               \
+    do {                       \
+        ctox_status rc_ = (expr); \
+        if (rc_) return rc_;   \
+    } while (0)
+
 // Tracked allocation: every byte is accounted on the context so that a caller
 // can assert "nothing left" after destroying its handles.
 ctox_status dev_alloc(ctox_ctx *ctx, void **ptr, size_t bytes);

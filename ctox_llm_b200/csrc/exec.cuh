@@ -96,12 +96,6 @@ struct ctox_exec {
 
 namespace ctox {
 
-#define EX(expr)               \
-    do {                       \
-        ctox_status rc_ = (expr); \
-        if (rc_) return rc_;   \
-    } while (0)
-
 // Tracked allocation owned by the executor (freed by ctox_exec_destroy), zeroed unless told otherwise.
 inline ctox_status xalloc(ctox_exec *e, void **p, size_t bytes, bool session, bool zero = true) {
     ctox_status rc = dev_alloc(e->ctx, p, bytes);

@@ -1,0 +1,299 @@
+// Latent attention of long passes: 128 queries of one head per CTA against 64-token key tiles.
+//
+// Scores and the weighted sum run on tcgen05.mma with operands staged by TMA; scores (double-buffered) and
+// the output accumulate in tensor memory. One warp loads, one issues the products, four hold one query
+// row per thread for the softmax: they read the scores from tensor memory, write the weights to shared
+// memory as the next product's operand, and rescale the output only when a row's maximum has grown by more
+// than 2^8 since its last reference (the final division is exact either way). Two CTAs share an SM when
+// their buffers fit, so one's softmax overlaps the other's products.
+#include "latent.cuh"
+#include "umma.cuh"
+
+#include <cmath>
+
+namespace ctox {
+
+constexpr int kLpThreads = 192;
+constexpr uint32_t kLpQ = 128, kLpK = 64;
+
+struct LpBox {  // a segment of the head dimension, cut into boxes one swizzle atom wide
+    uint32_t width, n;
+};
+__host__ __device__ inline LpBox lp_box(uint32_t dims) {
+    const uint32_t w = dims % 64 == 0 ? 64 : dims % 32 == 0 ? 32 : 16;
+    return LpBox{w, dims / w};
+}
+
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+__global__ void __launch_bounds__(kLpThreads)
+    k_latent_prefill(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_qr,
+                     const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_kr,
+                     const __grid_constant__ CUtensorMap map_v, LatentPrefill a, uint32_t stages, uint32_t tmem_cols,
+                     int32_t *error_word) {
+    using namespace umma;
+    pdl_launch();
+    extern __shared__ uint8_t raw[];
+    __shared__ __align__(8) uint64_t bars[14];
+    __shared__ uint32_t tmem_slot;
+    __shared__ volatile int dead;
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const uint32_t D = a.dim_pad + a.rot_pad;
+    const LpBox bd = lp_box(a.dim_pad), br = lp_box(a.rot_pad);
+    const uint32_t q_bytes = kLpQ * D * 2, k_bytes = kLpK * D * 2, v_bytes = a.vdim_pad * kLpK * 2;
+    const uint32_t base = (smem_addr(raw) + 1023) & ~1023u;
+    const uint32_t q_s = base, p_s = q_s + q_bytes, k_s = p_s + kLpQ * kLpK * 2, v_s = k_s + stages * k_bytes;
+    const uint32_t b0 = smem_addr(bars), q_full = b0, k_full = b0 + 8, k_empty = b0 + 24, v_full = b0 + 40,
+                   v_empty = b0 + 56, s_full = b0 + 72, p_full = b0 + 88, o_done = b0 + 96, drained = b0 + 104;
+    if (tid == 0) {
+        dead = 0;
+        bar_init(q_full, 1);
+        for (uint32_t i = 0; i < 2; ++i) {
+            bar_init(k_full + i * 8, 1);
+            bar_init(k_empty + i * 8, 1);
+            bar_init(v_full + i * 8, 1);
+            bar_init(v_empty + i * 8, 1);
+            bar_init(s_full + i * 8, 1);
+        }
+        bar_init(p_full, 4);
+        bar_init(o_done, 1);
+        bar_init(drained, 1);
+        bar_init_fence();
+    }
+    if (warp == 1) tmem_alloc(smem_addr(&tmem_slot), tmem_cols);
+    fence_before();
+    __syncthreads();
+    fence_after();
+    const uint32_t tmem = tmem_slot, tmem_o = tmem + 2 * kLpK;
+    const uint32_t q_tiles = (a.m + kLpQ - 1) / kLpQ;
+    const uint32_t i0 = (q_tiles - 1 - blockIdx.x % q_tiles) * kLpQ, head = blockIdx.x / q_tiles;
+    const uint32_t p_first = a.pos0 + i0, p_last = a.pos0 + min(i0 + kLpQ, a.m) - 1;
+    const uint32_t key_lo = a.window && p_first + 1 > a.window ? p_first + 1 - a.window : 0;
+    const uint32_t t_lo = (key_lo - a.row0) / kLpK, n = (p_last - a.row0) / kLpK - t_lo + 1;
+    pdl_wait();
+    if (warp == 0) {
+        if (lane == 0) {
+            bar_expect(q_full, q_bytes);
+            for (uint32_t i = 0; i < bd.n; ++i)
+                tma_load(q_s + i * kLpQ * bd.width * 2, &map_q, q_full, (int)(head * D + i * bd.width), (int)i0);
+            for (uint32_t i = 0; i < br.n; ++i)
+                tma_load(q_s + kLpQ * a.dim_pad * 2 + i * kLpQ * br.width * 2, &map_qr, q_full,
+                         (int)(head * D + a.dim_pad + i * br.width), (int)i0);
+            uint32_t k_issued = 0, v_issued = 0;
+            bool ok = true;
+            for (uint32_t j = 0; j < n; ++j) {
+                const uint32_t s = j % stages, round = j / stages, row = (t_lo + j) * kLpK;
+                if (round > 0 && !(ok = bar_wait(k_empty + s * 8, (round - 1) & 1, &dead))) break;
+                const uint32_t pos = a.row0 + row;
+                const int slot = (int)(a.page_table[pos / a.page_tokens] * a.page_tokens + pos % a.page_tokens);
+                const uint32_t kd = k_s + s * k_bytes;
+                bar_expect(k_full + s * 8, k_bytes);
+                for (uint32_t i = 0; i < bd.n; ++i)
+                    tma_load(kd + i * kLpK * bd.width * 2, &map_k, k_full + s * 8, (int)(head * a.dim_pad + i * bd.width), (int)row);
+                for (uint32_t i = 0; i < br.n; ++i)
+                    tma_load(kd + kLpK * a.dim_pad * 2 + i * kLpK * br.width * 2, &map_kr, k_full + s * 8,
+                             (int)(a.kv_pad + i * br.width), slot);
+                ++k_issued;
+                if (round > 0 && !(ok = bar_wait(v_empty + s * 8, (round - 1) & 1, &dead))) break;
+                bar_expect(v_full + s * 8, v_bytes);
+                tma_load(v_s + s * v_bytes, &map_v, v_full + s * 8, (int)row, (int)(head * a.vdim_pad));
+                ++v_issued;
+            }
+            if (!ok) {  // leave no copy in flight behind
+                bar_drain(q_full, 0);
+                for (uint32_t s = 0; s < stages && s < k_issued; ++s) bar_drain(k_full + s * 8, ((k_issued - 1 - s) / stages) & 1);
+                for (uint32_t s = 0; s < stages && s < v_issued; ++s) bar_drain(v_full + s * 8, ((v_issued - 1 - s) / stages) & 1);
+            }
+        }
+    } else if (warp == 1) {
+        if (lane == 0) {
+            const uint32_t idesc_s = idesc_bf16(kLpQ, kLpK), idesc_o = idesc_bf16(kLpQ, a.vdim_pad);
+            auto scores = [&](uint32_t j) -> bool {
+                const uint32_t s = j % stages;
+                if (!bar_wait(k_full + s * 8, (j / stages) & 1, &dead)) return false;
+                fence_after();
+                const uint32_t d = tmem + (j & 1) * kLpK, kd = k_s + s * k_bytes;
+                bool acc = false;
+                for (uint32_t i = 0; i < bd.n; ++i)
+                    for (uint32_t k = 0; k < bd.width; k += 16, acc = true)
+                        mma_f16(d, smem_desc(q_s + i * kLpQ * bd.width * 2 + k * 2, bd.width * 2),
+                                smem_desc(kd + i * kLpK * bd.width * 2 + k * 2, bd.width * 2), idesc_s, acc);
+                for (uint32_t i = 0; i < br.n; ++i)
+                    for (uint32_t k = 0; k < br.width; k += 16, acc = true)
+                        mma_f16(d, smem_desc(q_s + kLpQ * a.dim_pad * 2 + i * kLpQ * br.width * 2 + k * 2, br.width * 2),
+                                smem_desc(kd + kLpK * a.dim_pad * 2 + i * kLpK * br.width * 2 + k * 2, br.width * 2), idesc_s,
+                                acc);
+                commit(k_empty + s * 8);
+                commit(s_full + (j & 1) * 8);
+                return true;
+            };
+            bool ok = bar_wait(q_full, 0, &dead) && scores(0);
+            for (uint32_t j = 0; j < n && ok; ++j) {
+                if (j + 1 < n && !(ok = scores(j + 1))) break;
+                const uint32_t s = j % stages;
+                if (!(ok = bar_wait(p_full, j & 1, &dead) && bar_wait(v_full + s * 8, (j / stages) & 1, &dead))) break;
+                fence_after();
+                const uint64_t dp = smem_desc(p_s, 128), dv = smem_desc(v_s + s * v_bytes, 128);
+#pragma unroll
+                for (uint32_t k = 0; k < kLpK / 16; ++k) mma_f16(tmem_o, dp + k * 2, dv + k * 2, idesc_o, j > 0 || k > 0);
+                commit(v_empty + s * 8);
+                commit(o_done);
+            }
+            if (!ok) {
+                commit(drained);
+                bar_drain(drained, 0);
+            }
+        }
+    } else {
+        const uint32_t quarter = warp & 3, row = quarter * 32 + lane;
+        const uint32_t lanes = (quarter * 32) << 16;
+        const uint32_t pos = a.pos0 + i0 + row;
+        const float c = a.scale * 1.4426950408889634f;
+        float ref = -INFINITY, sum = 0.f;
+        bool ok = true;
+        for (uint32_t j = 0; j < n; ++j) {
+            if (!(ok = __all_sync(0xffffffffu, bar_wait(s_full + (j & 1) * 8, (j >> 1) & 1, &dead)))) break;
+            fence_after();
+            float s[kLpK];
+            tmem_ld32(tmem + (j & 1) * kLpK + lanes, s);
+            tmem_ld32(tmem + (j & 1) * kLpK + 32 + lanes, s + 32);
+            tmem_ld_wait();
+            const uint32_t t0 = a.row0 + (t_lo + j) * kLpK;
+            const bool all = t0 + kLpK - 1 <= p_first && (!a.window || p_last < t0 + a.window);
+            if (!all) {
+#pragma unroll
+                for (uint32_t k = 0; k < kLpK; ++k) {
+                    const uint32_t t = t0 + k;
+                    if (t > pos || (a.window && pos - t >= a.window)) s[k] = -INFINITY;
+                }
+            }
+            float mx = s[0];
+#pragma unroll
+            for (uint32_t k = 1; k < kLpK; ++k) mx = fmaxf(mx, s[k]);
+            mx *= c;
+            // P and O belong to the product of the tile before until it has finished
+            if (j > 0) {
+                if (!(ok = __all_sync(0xffffffffu, bar_wait(o_done, (j - 1) & 1, &dead)))) break;
+                fence_after();
+            }
+            const bool grow = mx > ref + 8.f || (ref == -INFINITY && mx > ref);
+            if (__any_sync(0xffffffffu, grow)) {
+                const float f = grow ? ex2(ref - mx) : 1.f;  // ref = -inf: 0, and nothing but zeros was added
+                if (grow) {
+                    ref = mx;
+                    sum *= f;
+                }
+                if (j > 0) {
+                    for (uint32_t d = 0; d < a.vdim_pad; d += 16) {
+                        float o[16];
+                        tmem_ld16(tmem_o + d + lanes, o);
+                        tmem_ld_wait();
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) o[i] *= f;
+                        tmem_st16(tmem_o + d + lanes, o);
+                    }
+                    tmem_st_wait();
+                }
+            }
+            const float r = ref == -INFINITY ? 0.f : ref;
+            const uint32_t dst = p_s + row * 128;
+#pragma unroll
+            for (uint32_t k = 0; k < kLpK; k += 8) {
+                float p[8];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    p[i] = ex2(fmaf(s[k + i], c, -r));
+                    sum += p[i];
+                }
+                uint32_t h[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const __nv_bfloat162 b = __floats2bfloat162_rn(p[2 * i], p[2 * i + 1]);
+                    h[i] = *reinterpret_cast<const uint32_t *>(&b);
+                }
+                asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(dst + (((k >> 3) ^ (row & 7)) << 4)), "r"(h[0]),
+                             "r"(h[1]), "r"(h[2]), "r"(h[3])
+                             : "memory");
+            }
+            fence_smem_async();
+            fence_before();
+            __syncwarp();
+            if (lane == 0) bar_arrive(p_full);
+        }
+        if (ok && (ok = __all_sync(0xffffffffu, bar_wait(o_done, (n - 1) & 1, &dead)))) {
+            fence_after();
+            const float inv = 1.0f / sum;
+            __nv_bfloat16 *out = a.out + ((size_t)(i0 + row) * a.heads + head) * a.vdim_pad;
+            for (uint32_t d = 0; d < a.vdim_pad; d += 16) {
+                float o[16];
+                tmem_ld16(tmem_o + d + lanes, o);
+                tmem_ld_wait();
+                uint32_t h[8];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    const __nv_bfloat162 b = __floats2bfloat162_rn(o[2 * i] * inv, o[2 * i + 1] * inv);
+                    h[i] = *reinterpret_cast<const uint32_t *>(&b);
+                }
+                if (i0 + row < a.m) {
+                    *reinterpret_cast<uint4 *>(out + d) = make_uint4(h[0], h[1], h[2], h[3]);
+                    *reinterpret_cast<uint4 *>(out + d + 8) = make_uint4(h[4], h[5], h[6], h[7]);
+                }
+            }
+            fence_before();
+        }
+    }
+    __syncwarp();
+    __syncthreads();
+    if (warp == 1) {
+        fence_after();
+        tmem_free(tmem, tmem_cols);
+    }
+    if (tid == 0 && dead) *error_word = DEV_ERR_WAIT_TIMEOUT;
+}
+
+namespace {
+
+size_t lp_smem(uint32_t dim_pad, uint32_t rot_pad, uint32_t vdim_pad, uint32_t stages) {
+    const size_t D = dim_pad + rot_pad;
+    return 1024 + kLpQ * D * 2 + kLpQ * kLpK * 2 + stages * (kLpK * D * 2 + (size_t)vdim_pad * kLpK * 2);
+}
+
+}  // namespace
+
+bool latent_prefill_fits(const ctox_ctx *ctx, uint32_t dim_pad, uint32_t rot_pad, uint32_t vdim_pad) {
+    return vdim_pad <= 256 && lp_smem(dim_pad, rot_pad, vdim_pad, 1) + 1024 <= (size_t)ctx->max_smem_optin;
+}
+
+ctox_status launch_latent_prefill(ctox_ctx *ctx, const LatentPrefill &a) {
+    if (!latent_prefill_fits(ctx, a.dim_pad, a.rot_pad, a.vdim_pad) || a.page_tokens % kLpQ || a.row0 % kLpQ || a.vt_ld % 8)
+        return fail(ctx, CTOX_SHAPE, "latent prefill: unsupported sizes");
+    const size_t half = ((size_t)ctx->max_smem_optin - 2048) / 2 - 1024;  // two CTAs on an SM
+    uint32_t stages = 2;
+    size_t smem = lp_smem(a.dim_pad, a.rot_pad, a.vdim_pad, 2);
+    if (smem > half && (lp_smem(a.dim_pad, a.rot_pad, a.vdim_pad, 1) <= half || smem + 1024 > (size_t)ctx->max_smem_optin)) {
+        stages = 1;
+        smem = lp_smem(a.dim_pad, a.rot_pad, a.vdim_pad, 1);
+    }
+    uint32_t cols = 256;  // scores 2 x 64 and the output
+    if (2 * kLpK + a.vdim_pad > 256) cols = 512;
+    const LpBox bd = lp_box(a.dim_pad), br = a.rot_pad ? lp_box(a.rot_pad) : LpBox{16, 0};
+    const uint64_t qw = (uint64_t)a.heads * (a.dim_pad + a.rot_pad), kw = (uint64_t)a.heads * a.dim_pad,
+                   cw = a.kv_pad + a.rot_pad;
+    CUtensorMap mq, mqr, mk, mkr, mv;
+    EX(tensor_map_bf16(ctx, &mq, a.q, a.m, qw, qw, kLpQ, bd.width));
+    EX(tensor_map_bf16(ctx, &mqr, a.q, a.m, qw, qw, kLpQ, br.width));
+    EX(tensor_map_bf16(ctx, &mk, a.k, a.span, kw, kw, kLpK, bd.width));
+    EX(tensor_map_bf16(ctx, &mkr, a.cache, a.slots, cw, cw, kLpK, br.width));
+    EX(tensor_map_bf16(ctx, &mv, a.vt, (uint64_t)a.heads * a.vdim_pad, a.span, a.vt_ld, a.vdim_pad, kLpK));
+    CTOX_CUDA(ctx, cudaFuncSetAttribute(k_latent_prefill, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    const uint32_t grid = (a.m + kLpQ - 1) / kLpQ * a.heads;
+    CTOX_CUDA(ctx, launch_pdl(k_latent_prefill, dim3(grid), dim3(kLpThreads), smem, ctx->stream, mq, mqr, mk, mkr, mv, a,
+                              stages, cols, ctx->dev_error));
+    return CTOX_OK;
+}
+
+}  // namespace ctox

@@ -4,9 +4,12 @@
 #include <algorithm>
 #include <cmath>
 
+#include "gemm.cuh"
 #include "latent.cuh"
 
 namespace ctox {
+
+constexpr uint32_t kDefaultPass = 2048, kHeadRowsLong = 64;
 
 namespace {
 
@@ -135,7 +138,7 @@ ctox_status stack_create(ctox_ctx *ctx, const ctox_stack_config *c, const ctox_l
         if (y.mlp != CTOX_MLP_NONE && y.mlp != CTOX_MLP_RELU2)
             return fail(ctx, CTOX_UNSUPPORTED_OPERATION, "layer %u: unknown feed-forward %u", l, y.mlp);
         if (!y.heads || !y.dim || !y.vdim || !y.q_rank || !y.kv_rank || y.rot_dim % 2 || !(y.rope_base > 0.0) ||
-            !std::isfinite(y.score_scale) || (y.mlp != CTOX_MLP_NONE && !y.ff))
+            !std::isfinite(y.score_scale) || !(y.score_scale > 0.f) || (y.mlp != CTOX_MLP_NONE && !y.ff))
             return fail(ctx, CTOX_SHAPE, "layer %u: unsupported latent-attention or feed-forward sizes", l);
         if (y.kv_from >= 0) {
             if ((uint32_t)y.kv_from >= l || layers[y.kv_from].kv_from >= 0)
@@ -162,6 +165,11 @@ ctox_status stack_create(ctox_ctx *ctx, const ctox_stack_config *c, const ctox_l
         L.kv_pad = round_up(L.c.kv_rank, 16);
         L.head_w = L.dim_pad + L.rot_pad;
     }
+    // Passes longer than kDensePass use the tensor-core products; in 32-bit mode, with pages that are not
+    // whole tiles or with heads too large for its shared memory, every pass is a short one.
+    bool longer = c->kv_dtype == CTOX_BF16 && c->kv_page_tokens % 128 == 0;
+    for (const StackLayer &L : s->layers) longer = longer && latent_prefill_fits(ctx, L.dim_pad, L.rot_pad, L.vdim_pad);
+    if (longer) s->pass_cap = std::max(kDensePass, std::min(c->pass_tokens ? c->pass_tokens : kDefaultPass, c->max_context_tokens));
     // what the executor's own calls read of the model
     e->cfg.vocab_size = c->vocab_size;
     e->cfg.hidden_size = c->hidden_size;
@@ -345,6 +353,32 @@ ctox_status stack_warmup(ctox_exec *e) {
         CTOX_CUDA(ctx, cudaStreamSynchronize(ctx->stream));  // `freq` is a local
     }
 #define WALLOC(ptr, bytes) EX(xalloc(e, (void **)&(ptr), (bytes), true))
+    const bool longer = P > kDensePass;
+    if (longer) {
+        uint64_t span = 0, k_w = 0, cq_w = 0;
+        for (uint32_t l = 0; l < s->layers.size(); ++l) {
+            StackLayer &L = s->layers[l];
+            const uint64_t reach = L.c.window ? L.c.window : c.max_context_tokens;
+            span = std::max<uint64_t>(span, std::min<uint64_t>(reach + P, c.max_context_tokens));
+            k_w = std::max<uint64_t>(k_w, (uint64_t)L.c.heads * L.dim_pad);
+            cq_w = std::max<uint64_t>(cq_w, round_up(L.c.q_rank, 8));
+            for (uint32_t other : s->table_layers)
+                if (s->layers[other].c.rot_dim == L.c.rot_dim && s->layers[other].c.rope_base == L.c.rope_base)
+                    L.table = s->layers[other].table;
+            if (L.table || !L.c.rot_dim) continue;
+            WALLOC(L.table, P * (L.c.rot_dim / 2) * sizeof(float2));
+            s->table_layers.push_back(l);
+        }
+        s->span_cap = round_up((uint32_t)span, 128) + 128;
+        WALLOC(s->h_b, P * round_up(c.hidden_size, 8) * 2);
+        WALLOC(s->cq_b, P * cq_w * 2);
+        WALLOC(s->q_b, P * q_w * 2);
+        WALLOC(s->k_b, s->span_cap * k_w * 2);
+        WALLOC(s->vt_b, s->span_cap * att_w * 2);
+        WALLOC(s->att_b, P * att_w * 2);
+        WALLOC(s->u_b, P * round_up((uint32_t)ff, 8) * 2);
+        WALLOC(s->head_b, (size_t)kHeadRowsLong * round_up(c.hidden_size, 8) * 2);
+    }
     WALLOC(s->x[0], P * H * 4);
     WALLOC(s->x[1], P * H * 4);
     WALLOC(s->y, P * H * 4);
@@ -358,7 +392,7 @@ ctox_status stack_warmup(ctox_exec *e) {
     WALLOC(s->rows_dev, P * 4);
     WALLOC(e->tokens_dev, (P + 1) * 4);
     WALLOC(e->hist_hidden, kMaxPass * H * 4);
-    s->head_rows = (uint32_t)S;
+    s->head_rows = longer ? kHeadRowsLong : (uint32_t)S;
     WALLOC(s->head_in, S * H * 4);
     WALLOC(e->logits, (size_t)s->head_rows * c.vocab_size * 4);
     // caches: a ring of pages that holds the widest window read from it and one pass
@@ -494,6 +528,19 @@ ctox_status layer_short(ctox_exec *e, uint32_t l, uint32_t m, uint32_t pos0) {
     return CTOX_OK;
 }
 
+GemmOperand rows_of(const __nv_bfloat16 *p, uint32_t rows, uint32_t cols, uint32_t ld) {
+    return GemmOperand{p, rows, cols, ld, nullptr, 0, 0, 0};
+}
+GemmOperand weight_of(const DenseMat &w) { return rows_of(w.w, w.rows, w.cols, w.ld); }
+GemmOut gemm_out(void *d, uint32_t ld, bool bf16, int kind = OUT_PLAIN) {
+    GemmOut o{};
+    o.d = d;
+    o.ld = ld;
+    o.bf16 = bf16;
+    o.kind = kind;
+    return o;
+}
+
 StreamNorm stream_norm(const StackModel *s, const float *w) {
     StreamNorm n{};
     n.x = s->x[s->cur];
@@ -505,6 +552,77 @@ StreamNorm stream_norm(const StackModel *s, const float *w) {
     return n;
 }
 
+// One layer for a long pass: the products on the tensor cores over bf16 activations, keys and values of
+// the visible span expanded from the cache.
+ctox_status layer_long(ctox_exec *e, uint32_t l, uint32_t m, uint32_t pos0) {
+    ctox_ctx *ctx = e->ctx;
+    StackModel *s = e->stack;
+    StackLayer &L = s->layers[l];
+    const StackLayer &O = s->layers[L.owner];
+    const ctox_layer_config &c = L.c;
+    const uint32_t H = s->c.hidden_size, h_ld = round_up(H, 8), qw = c.heads * L.head_w, vw = c.heads * L.vdim_pad,
+                   cq_ld = round_up(c.q_rank, 8), ff_ld = round_up(c.ff, 8);
+    auto norm_into_h = [&](const float *w) -> ctox_status {  // the stream in place, its norm as bf16
+        StreamNorm n = stream_norm(s, w);
+        n.x_out = n.y ? s->x[s->cur] : nullptr;
+        n.bf16_out = s->h_b;
+        n.bf16_ld = h_ld;
+        s->y_norm = nullptr;
+        return launch_stream_norm(ctx, n, m);
+    };
+    EX(norm_into_h(L.norm1));
+    const GemmOperand h = rows_of(s->h_b, m, H, h_ld);
+    EX(launch_gemm(ctx, h, weight_of(L.fan), gemm_out(s->fan, L.fan.rows, false)));
+    const LatentAppend ap = append_args(e, L, pos0);
+    EX(launch_latent_split(ctx, s->fan, L.fan.rows, c.q_rank, L.q_norm, s->c.norm_eps, s->cq_b, cq_ld,
+                           L.owner == l ? &ap : nullptr, m));
+    GemmOut q = gemm_out(s->q_b, qw, true, c.rot_dim ? OUT_ROPE : OUT_PLAIN);
+    q.head_width = L.head_w;
+    q.rope0 = L.dim_pad;
+    q.rope_dims = c.rot_dim;
+    q.table = L.table;
+    EX(launch_gemm(ctx, rows_of(s->cq_b, m, c.q_rank, cq_ld), weight_of(L.q_up), q));
+    const uint32_t first = c.window && pos0 + 1 > c.window ? pos0 + 1 - c.window : 0;
+    LatentPrefill a{};
+    a.row0 = first / 128 * 128;
+    a.span = pos0 + m - a.row0;
+    GemmOperand latents = rows_of((const __nv_bfloat16 *)O.cache, a.span, L.kv_pad, L.kv_pad + L.rot_pad);
+    latents.page_table = O.page_table;
+    latents.page_tokens = s->c.kv_page_tokens;
+    latents.row0 = a.row0;
+    latents.store_rows = O.slots;
+    EX(launch_gemm(ctx, latents, weight_of(L.k_up), gemm_out(s->k_b, c.heads * L.dim_pad, true)));
+    EX(launch_gemm(ctx, weight_of(L.v_up), latents, gemm_out(s->vt_b, s->span_cap, true)));
+    a.q = s->q_b;
+    a.k = s->k_b;
+    a.vt = s->vt_b;
+    a.vt_ld = s->span_cap;
+    a.cache = (const __nv_bfloat16 *)O.cache;
+    a.out = s->att_b;
+    a.page_table = O.page_table;
+    a.page_tokens = s->c.kv_page_tokens;
+    a.slots = O.slots;
+    a.heads = c.heads;
+    a.dim_pad = L.dim_pad;
+    a.rot_pad = L.rot_pad;
+    a.vdim_pad = L.vdim_pad;
+    a.kv_pad = L.kv_pad;
+    a.pos0 = pos0;
+    a.m = m;
+    a.window = c.window;
+    a.scale = c.score_scale;
+    EX(launch_latent_prefill(ctx, a));
+    EX(launch_gemm(ctx, rows_of(s->att_b, m, vw, vw), weight_of(L.o), gemm_out(s->y, H, false)));
+    s->y_norm = L.norm1b;
+    if (c.mlp != CTOX_MLP_NONE) {
+        EX(norm_into_h(L.norm2));
+        EX(launch_gemm(ctx, h, weight_of(L.up), gemm_out(s->u_b, ff_ld, true, OUT_RELU2)));
+        EX(launch_gemm(ctx, rows_of(s->u_b, m, c.ff, ff_ld), weight_of(L.down), gemm_out(s->y, H, false)));
+        s->y_norm = L.norm2b;
+    }
+    return CTOX_OK;
+}
+
 }  // namespace
 
 ctox_status stack_pass(ctox_exec *e, uint32_t m, uint64_t pos0) {
@@ -514,8 +632,13 @@ ctox_status stack_pass(ctox_exec *e, uint32_t m, uint64_t pos0) {
     s->cur = 0;
     s->y_norm = nullptr;
     EX(launch_embed_dense(ctx, s->embed.w, s->embed.ld, e->tokens_dev, H, m, s->x[0]));
+    if (m > kDensePass)
+        for (uint32_t l : s->table_layers) {
+            const StackLayer &L = s->layers[l];
+            EX(launch_rope_table(ctx, L.freq, L.c.rot_dim / 2, (uint32_t)pos0, m, L.table));
+        }
     for (uint32_t l = 0; l < s->layers.size(); ++l) {
-        EX(layer_short(e, l, m, (uint32_t)pos0));
+        EX(m > kDensePass ? layer_long(e, l, m, (uint32_t)pos0) : layer_short(e, l, m, (uint32_t)pos0));
         if (s->streams) {  // evidence: the stream after this layer
             StreamNorm n = stream_norm(s, nullptr);
             n.x_out = s->streams + ((size_t)l * s->c.max_context_tokens + pos0) * H;
@@ -544,6 +667,14 @@ ctox_status stack_head_rows(ctox_exec *e, const uint32_t *rows, uint32_t n) {
     CTOX_CUDA(ctx, cudaMemcpyAsync(s->rows_dev, rows, n * 4, cudaMemcpyHostToDevice, ctx->stream));
     StreamNorm a = stream_norm(s, s->final_norm);
     a.rows = s->rows_dev;
+    if (n > kDensePass) {
+        a.bf16_out = s->head_b;
+        a.bf16_ld = round_up(H, 8);
+        EX(launch_stream_norm(ctx, a, n));
+        GemmOut o = gemm_out(e->logits, s->c.vocab_size, false, s->c.logit_softcap > 0.f ? OUT_SOFTCAP : OUT_PLAIN);
+        o.cap = s->c.logit_softcap;
+        return launch_gemm(ctx, rows_of(s->head_b, n, H, a.bf16_ld), weight_of(s->head), o);
+    }
     a.f32_out = s->head_in;
     EX(launch_stream_norm(ctx, a, n));
     VecOut out = vec_out(e->logits, s->c.vocab_size, s->c.logit_softcap > 0.f ? OUT_SOFTCAP : OUT_PLAIN);

@@ -23,7 +23,8 @@ struct StackLayer {
     DenseMat up, down;
     float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr, *q_norm = nullptr,
           *kv_norm = nullptr;
-    float *freq = nullptr;  // [rot_dim / 2]
+    float *freq = nullptr;     // [rot_dim / 2]
+    float2 *table = nullptr;   // [position of the pass][rot_dim / 2] (cos, sin), shared by layers that rotate alike
     uint64_t loaded = 0;    // bit per tensor id
     // cache of an owner: ring of pages through the page table, rows [kv_pad | rot_pad]
     void *cache = nullptr;
@@ -44,6 +45,7 @@ struct StackModel {
     __nv_bfloat16 *h_b = nullptr, *cq_b = nullptr, *q_b = nullptr, *k_b = nullptr, *vt_b = nullptr, *att_b = nullptr,
                   *u_b = nullptr, *head_b = nullptr;
     uint32_t span_cap = 0;  // key rows of k_b, columns of vt_b
+    std::vector<uint32_t> table_layers;  // one layer of every distinct rotation
     float *head_in = nullptr;
     uint32_t *rows_dev = nullptr;
     uint32_t head_rows = 0;  // rows of e->logits
