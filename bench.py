@@ -812,6 +812,135 @@ def run_micro(args):
     be.close()
 
 
+LATENT_SIZES = {
+    # width, layers, vocabulary, feed-forward | heads, dim, rot_dim, vdim, q_rank, kv_rank, window | the hybrid
+    # model's query and KV heads (of 256) at the same width
+    "2k": dict(width=2048, layers=8, vocab=32768, ff=8192, heads=16, dim=128, rot_dim=64, vdim=128, q_rank=768,
+               kv_rank=512, window=4096, hybrid_heads=(8, 2)),
+    "5k": dict(width=5120, layers=8, vocab=32768, ff=17408, heads=40, dim=128, rot_dim=64, vdim=128, q_rank=1536,
+               kv_rank=512, window=4096, hybrid_heads=(24, 4)),
+    "7k": dict(width=7168, layers=4, vocab=32768, ff=18432, heads=128, dim=128, rot_dim=64, vdim=128, q_rank=1536,
+               kv_rank=512, window=4096, hybrid_heads=(32, 8)),
+}
+
+
+def run_latent(args):
+    """The layer-stack model (Lomelorn: latent attention, window 4096, bf16 weights) beside the closest
+    existing model, the hybrid with full attention in every layer, at the same width, depth, feed-forward
+    and vocabulary: decode at a context of 8192 tokens and prefill of one 4096-token prompt, through the
+    executor's own calls, random weights. Per kernel family: device time with an event pair around every
+    launch (serialised), and the fraction of its roofline (the larger of bytes / measured copy bandwidth and
+    flops / measured bf16 product)."""
+    import torch
+    import ctox_llm_b200 as ctox
+    from ctox_llm_b200 import _native as N
+    local = int(os.environ.get("LOCAL_RANK", "0"))
+    if int(os.environ.get("RANK", "0")) != 0:
+        return
+    torch.cuda.set_device(local)
+    stream = torch.cuda.Stream(device=local)
+    be = ctox.B200Backend(local, stream=stream.cuda_stream)
+    peak, peak_kind = load_peaks()
+    tflops = 1590.0
+    if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")):
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+            tflops = float(json.load(f)["bf16_tflops"])
+    context, prompt_n = 8192, 4096
+    prompt = [int(t) for t in np.random.default_rng(0).integers(0, 32768, prompt_n)]
+
+    def stack(z):
+        layer = dict(rope_base=10000.0, mixer=N.MIXER_LATENT_ATTENTION, heads=z["heads"], dim=z["dim"], rot_dim=z["rot_dim"],
+                     vdim=z["vdim"], q_rank=z["q_rank"], kv_rank=z["kv_rank"], window=z["window"], kv_from=-1,
+                     score_scale=(z["dim"] + z["rot_dim"]) ** -0.5, mlp=N.MLP_RELU2, ff=z["ff"])
+        return ctox.StackConfig(vocab_size=z["vocab"], hidden_size=z["width"], norm_eps=1e-6, logit_softcap=30.0,
+                                layers=[N.LayerConfig(**layer) for _ in range(z["layers"])],
+                                max_context_tokens=context + 1024, pass_tokens=args.pass_tokens)
+
+    def hybrid(z):
+        return ctox.qwen38_27b_config(
+            vocab_size=z["vocab"], hidden_size=z["width"], intermediate_size=z["ff"], num_hidden_layers=z["layers"],
+            num_attention_heads=z["hybrid_heads"][0], num_key_value_heads=z["hybrid_heads"][1], full_attention_interval=1,
+            mtp_num_hidden_layers=0, draft_vocab=0, max_draft_tokens=0, max_context_tokens=context + 1024)
+
+    def families(work):
+        be.kernel_timing(True)
+        work()
+        out = be.kernel_timing_classes()
+        be.kernel_timing(False)
+        for k in out.values():
+            ideal = max(k["bytes"] / (peak * 1e9), k["flops"] / (tflops * 1e12)) * 1e3
+            k["us_per_launch"] = k["ms"] * 1e3 / k["launches"]
+            if ideal > 0:
+                k["roofline_frac"] = ideal / k["ms"]
+        return out
+
+    def measure(config):
+        ex = ctox.B200Executor(be, config)
+        ex.fill_synthetic(seed=0)
+        ex.warmup()
+
+        def prefill():
+            ex.reset_session()
+            ex.extend(prompt)
+
+        def timed(work, n):
+            torch.cuda.synchronize()
+            ev0, ev1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            t0 = time.perf_counter()
+            ev0.record(stream)
+            for _ in range(n):
+                work()
+            ev1.record(stream)
+            torch.cuda.synchronize()
+            return ev0.elapsed_time(ev1), time.perf_counter() - t0
+
+        res = {"allocations": ex.allocations()}
+        for _ in range(2):
+            prefill()
+        ms, wall = timed(prefill, 3)
+        res["prefill"] = {"tokens_per_s": 3 * prompt_n / (ms * 1e-3), "e2e_tokens_per_s": 3 * prompt_n / wall, "ms": ms / 3,
+                          "families": families(prefill)}
+        tok = [1]
+
+        def decode():
+            tok[0] = ex.decode(tok[0], mtp_enabled=False).token_id
+
+        ex.prefill_synthetic(context, seed=1)
+        for _ in range(max(args.warmup, 3)):
+            decode()
+        launches0 = be.kernel_launches()
+        ms, wall = timed(decode, args.steps)
+        res["decode"] = {"tokens_per_s": args.steps / (ms * 1e-3), "e2e_tokens_per_s": args.steps / wall,
+                         "ms": ms / args.steps, "launches_per_token": (be.kernel_launches() - launches0) / args.steps,
+                         "enqueue_us": ex.last_enqueue_us(), "families": families(decode)}
+        ex.unload()
+        return res
+
+    sampler = ClockSampler(local)
+    sampler.start()
+    sweep = {}
+    launches0 = be.kernel_launches()
+    with torch.cuda.stream(stream):
+        for name in args.sizes.split(","):
+            z = LATENT_SIZES[name]
+            sweep[name] = {"shape": z, "lomelorn": measure(stack(z))}
+            if not args.quick:
+                sweep[name]["hybrid"] = measure(hybrid(z))
+    last = sweep[args.sizes.split(",")[-1] if "5k" not in sweep else "5k"]["lomelorn"]
+    line = {"metric": "latent_decode_tokens_per_s", "value": last["decode"]["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
+            "steps": args.steps, "warmup": max(args.warmup, 3), "ms_per_step": last["decode"]["ms"], "higher_is_better": True,
+            "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+            "config": {"workload": "layer stack (latent attention) beside the hybrid model with full attention at equal width, "
+                                   f"depth, feed-forward and vocabulary; decode at context {context}, prefill of {prompt_n} tokens",
+                       "l2": "a pass streams more weights than twice the L2"},
+            "e2e": {"value": last["decode"]["e2e_tokens_per_s"], "unit": "tokens/s", "h2d_bytes_per_step": 4,
+                    "d2h_bytes_per_step": 300},
+            "sweep": sweep, "peaks": {"hbm_gbs": peak, "bf16_tflops": tflops, "kind": f"of {peak_kind}"},
+            "gpu_launches": be.kernel_launches() - launches0, "clocks": sampler.stop(), "cpu_baseline": None}
+    print(json.dumps(line), flush=True)
+    be.close()
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -819,7 +948,7 @@ def main():
     ap.add_argument("--warmup", type=int, default=None)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--workload", default="decode",
-                    choices=["decode", "q4_matvec", "q2_matvec", "matvec", "verify_layer", "gated_delta", "kv_pack"])
+                    choices=["decode", "q4_matvec", "q2_matvec", "matvec", "verify_layer", "gated_delta", "kv_pack", "latent"])
     ap.add_argument("--dtype", default="q4", choices=["q4", "q2"], help="matvec: code format")
     ap.add_argument("--rows", type=int, default=17408)
     ap.add_argument("--cols", type=int, default=5120)
@@ -828,6 +957,8 @@ def main():
     ap.add_argument("--replicas", type=int, default=0,
                     help="matvec: weight replicas to rotate (default: enough to exceed twice the L2; 1 = weights "
                          "stay in L2, a diagnostic that separates the instruction cost from the HBM stream)")
+    ap.add_argument("--sizes", default="2k,5k,7k", help="latent: sizes to run")
+    ap.add_argument("--pass-tokens", type=int, default=0, help="latent: prompt tokens per pass (0: the default)")
     ap.add_argument("--context", type=int, default=32768)
     ap.add_argument("--drafts", type=int, default=3,
                     help="decode: chained MTP drafts per block (3 = 4 verify positions, BASELINE config 2; "
@@ -838,13 +969,15 @@ def main():
                     help="decode: only the timed region and one kernel-timing block (for launch lists)")
     args = ap.parse_args()
     if args.steps is None:
-        args.steps = {"decode": 256, "verify_layer": 400, "gated_delta": 50, "kv_pack": 50}.get(args.workload, 2000)
+        args.steps = {"decode": 256, "verify_layer": 400, "gated_delta": 50, "kv_pack": 50, "latent": 64}.get(args.workload, 2000)
     if args.warmup is None:
-        args.warmup = {"decode": 4, "gated_delta": 5, "kv_pack": 5}.get(args.workload, 50)
+        args.warmup = {"decode": 4, "gated_delta": 5, "kv_pack": 5, "latent": 4}.get(args.workload, 50)
     if args.impl == "reference":
         run_reference(args)
     elif args.workload == "decode":
         run_decode(args)
+    elif args.workload == "latent":
+        run_latent(args)
     elif args.workload == "q4_matvec":
         run_b200(args)
     else:

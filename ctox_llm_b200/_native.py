@@ -77,6 +77,15 @@ class ModelConfig(C.Structure):
             "max_draft_tokens", "draft_vocab")]
 
 
+KERNEL_CLASSES = ("stream_matvec", "attention", "dense_matvec", "latent_attention", "gemm", "latent_prefill", "norm", "other")
+
+
+class KernelClass(C.Structure):
+    """ctox_kernel_class (include/ctox_b200.h)."""
+
+    _fields_ = [("ms", C.c_double), ("launches", C.c_uint64), ("bytes", C.c_double), ("flops", C.c_double)]
+
+
 MIXER_LATENT_ATTENTION = 1
 MLP_NONE, MLP_RELU2 = 0, 1
 
@@ -161,6 +170,7 @@ SIGNATURES = {
     "ctox_ctx_kernel_timing": (C.c_int32, [C.c_void_p, C.c_int32]),
     "ctox_ctx_kernel_timing_read": (C.c_int32, [C.c_void_p, C.POINTER(C.c_double),
                                                 C.POINTER(C.c_uint64)]),
+    "ctox_ctx_kernel_timing_classes": (C.c_int32, [C.c_void_p, C.POINTER(KernelClass)]),
     "ctox_fused_matvec": (C.c_int32, [C.c_void_p, C.POINTER(FusedMatVecOp), C.c_void_p]),
     "ctox_fused_matvec_fanout": (C.c_int32, [C.c_void_p, C.POINTER(FusedMatVecOp), C.c_uint64,
                                              C.POINTER(C.c_void_p)]),

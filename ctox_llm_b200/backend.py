@@ -256,6 +256,13 @@ class B200Backend:
     def kernel_timing(self, enable: bool) -> None:
         self._check(self._lib.ctox_ctx_kernel_timing(self._ctx, int(enable)))
 
+    def kernel_timing_classes(self) -> dict:
+        """{family: {ms, launches, bytes, flops}} of the bracketed launches since the last read."""
+        c = (N.KernelClass * len(N.KERNEL_CLASSES))()
+        self._check(self._lib.ctox_ctx_kernel_timing_classes(self._ctx, c))
+        return {name: {"ms": k.ms, "launches": int(k.launches), "bytes": k.bytes, "flops": k.flops}
+                for name, k in zip(N.KERNEL_CLASSES, c) if k.launches}
+
     def kernel_timing_read(self):
         """(total milliseconds, launches) of the dominant kernel since the last read."""
         ms, n = C.c_double(), C.c_uint64()

@@ -15,6 +15,22 @@
 
 namespace ctox {
 struct TpPeer;
+// Kernel families of the optional timing (benchmark support).
+enum KernelClass : int {
+    KC_STREAM_MATVEC = 0,   // packed weights
+    KC_ATTENTION = 1,       // hybrid model's attention with its merge
+    KC_DENSE_MATVEC = 2,    // bf16 weights, short passes
+    KC_LATENT_ATTENTION = 3,  // latent cache, short passes
+    KC_GEMM = 4,            // tensor-core product, long passes
+    KC_LATENT_PREFILL = 5,  // tensor-core attention, long passes
+    KC_NORM = 6,            // norms of long passes
+    KC_COUNT = 8
+};
+struct TimedLaunch {
+    cudaEvent_t begin, end;
+    int kind;
+    double bytes, flops;
+};
 }
 struct ctox_ctx {
     int device = 0;
@@ -40,7 +56,7 @@ struct ctox_ctx {
     bool tp_silent = false;
     // optional per-kernel timing of the dominant kernel (benchmark support)
     bool timing = false;
-    std::vector<std::pair<cudaEvent_t, cudaEvent_t>> timing_events;
+    std::vector<ctox::TimedLaunch> timing_events;
 };
 
 namespace ctox {
@@ -92,7 +108,7 @@ void tp_peer_destroy(ctox_ctx *ctx);
 // When timing is enabled, brackets the next launches with a CUDA event pair on
 // the context's stream; both are no-ops otherwise.
 void timing_begin(ctox_ctx *ctx);
-void timing_end(ctox_ctx *ctx);
+void timing_end(ctox_ctx *ctx, int kind = KC_STREAM_MATVEC, double bytes = 0, double flops = 0);
 
 // Programmatic dependent launch. A kernel launched through launch_pdl may begin while the kernel
 // before it in the stream is still running; it must execute pdl_wait() before it touches memory

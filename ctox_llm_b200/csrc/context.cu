@@ -59,12 +59,16 @@ void timing_begin(ctox_ctx *ctx) {
     cudaEvent_t a = nullptr, b = nullptr;
     if (cudaEventCreate(&a) != cudaSuccess || cudaEventCreate(&b) != cudaSuccess) return;
     cudaEventRecord(a, ctx->stream);
-    ctx->timing_events.emplace_back(a, b);
+    ctx->timing_events.push_back(TimedLaunch{a, b, KC_STREAM_MATVEC, 0, 0});
 }
 
-void timing_end(ctox_ctx *ctx) {
+void timing_end(ctox_ctx *ctx, int kind, double bytes, double flops) {
     if (!ctx->timing || ctx->timing_events.empty()) return;
-    cudaEventRecord(ctx->timing_events.back().second, ctx->stream);
+    TimedLaunch &t = ctx->timing_events.back();
+    t.kind = kind;
+    t.bytes = bytes;
+    t.flops = flops;
+    cudaEventRecord(t.end, ctx->stream);
 }
 }  // namespace ctox
 
@@ -145,8 +149,8 @@ ctox_status ctox_ctx_destroy(ctox_ctx *ctx) {
     if (ctx->stream) cudaStreamSynchronize(ctx->stream);
     ctox_tp_destroy(ctx);
     for (auto &ev : ctx->timing_events) {
-        cudaEventDestroy(ev.first);
-        cudaEventDestroy(ev.second);
+        cudaEventDestroy(ev.begin);
+        cudaEventDestroy(ev.end);
     }
     if (ctx->dev_error) cudaFree(ctx->dev_error);
     if (ctx->host_error) cudaFreeHost(ctx->host_error);
@@ -175,23 +179,32 @@ ctox_status ctox_ctx_kernel_timing(ctox_ctx *ctx, int32_t enable) {
     return CTOX_OK;
 }
 
-ctox_status ctox_ctx_kernel_timing_read(ctox_ctx *ctx, double *total_ms, uint64_t *launches) {
-    if (!ctx || !total_ms || !launches) return CTOX_INVALID_STATE;
+ctox_status ctox_ctx_kernel_timing_classes(ctox_ctx *ctx, ctox_kernel_class *classes) {
+    if (!ctx || !classes) return CTOX_INVALID_STATE;
     CTOX_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
-    double sum = 0.0;
-    uint64_t n = 0;
+    memset(classes, 0, sizeof(ctox_kernel_class) * CTOX_KERNEL_CLASSES);
     for (auto &ev : ctx->timing_events) {
         float ms = 0.f;
-        if (cudaEventElapsedTime(&ms, ev.first, ev.second) == cudaSuccess) {
-            sum += ms;
-            ++n;
+        if (cudaEventElapsedTime(&ms, ev.begin, ev.end) == cudaSuccess && ev.kind < CTOX_KERNEL_CLASSES) {
+            ctox_kernel_class &c = classes[ev.kind];
+            c.ms += ms;
+            c.launches += 1;
+            c.bytes += ev.bytes;
+            c.flops += ev.flops;
         }
-        cudaEventDestroy(ev.first);
-        cudaEventDestroy(ev.second);
+        cudaEventDestroy(ev.begin);
+        cudaEventDestroy(ev.end);
     }
     ctx->timing_events.clear();
-    *total_ms = sum;
-    *launches = n;
+    return CTOX_OK;
+}
+
+ctox_status ctox_ctx_kernel_timing_read(ctox_ctx *ctx, double *total_ms, uint64_t *launches) {
+    if (!ctx || !total_ms || !launches) return CTOX_INVALID_STATE;
+    ctox_kernel_class classes[CTOX_KERNEL_CLASSES];
+    EX(ctox_ctx_kernel_timing_classes(ctx, classes));
+    *total_ms = classes[KC_STREAM_MATVEC].ms;
+    *launches = classes[KC_STREAM_MATVEC].launches;
     return CTOX_OK;
 }
 

@@ -315,9 +315,11 @@ ctox_status matvec_launch(ctox_ctx *ctx, const DenseMat &w, uint32_t groups, uin
     const uint32_t fit = (uint32_t)(per_sm * ctx->sm_count), waves = (units + fit - 1) / fit;
     const uint32_t grid = (units + waves - 1) / waves;
     const LatentAppend ap = append ? *append : LatentAppend{};
+    timing_begin(ctx);
     CTOX_CUDA(ctx, launch_pdl(k_dense_matvec<M, R>, dim3(grid + append_positions), dim3(kDvThreads), smem, ctx->stream,
                               (const __nv_bfloat16 *)w.w, w.ld, rows_per_group, units_per_group, units, ks, lpr_log2, m,
                               in, out, ap, append_positions));
+    timing_end(ctx, KC_DENSE_MATVEC, 2.0 * w.rows * w.ld, 2.0 * w.rows * w.ld * m);
     return CTOX_OK;
 }
 
@@ -419,7 +421,10 @@ ctox_status launch_stream_norm(ctox_ctx *ctx, const StreamNorm &a, uint32_t m) {
         return fail(ctx, CTOX_MEMORY_BUDGET, "stream norm: width %u does not fit shared memory", a.width);
     if (smem > 40 * 1024)
         CTOX_CUDA(ctx, cudaFuncSetAttribute(k_stream_norm, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    timing_begin(ctx);
     CTOX_CUDA(ctx, launch_pdl(k_stream_norm, dim3(m), dim3(kSnThreads), smem, ctx->stream, a));
+    timing_end(ctx, KC_NORM,
+               (double)m * a.width * (4 + (a.y ? 4 : 0) + (a.x_out ? 4 : 0) + (a.f32_out ? 4 : 0) + (a.bf16_out ? 2 : 0)), 0);
     return CTOX_OK;
 }
 

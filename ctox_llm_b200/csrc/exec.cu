@@ -942,8 +942,11 @@ ctox_status layer_body(ctox_exec *e, uint32_t l, float *h, uint32_t m, uint64_t 
                         ls.v_cache, c.kv_dtype == CTOX_BF16, page_table, c.kv_page_tokens);
         const uint64_t tiles = (slot0 + m + 63) / 64;
         const uint32_t splits = (uint32_t)(tiles < e->attn_splits_max ? (tiles ? tiles : 1) : e->attn_splits_max);
+        timing_begin(ctx);
         launch_attention(st, g, e->aq, e->agate, ls.k_cache, ls.v_cache, c.kv_dtype == CTOX_BF16, page_table,
                          c.kv_page_tokens, slot0, m, splits, e->attn_ws, out_in);
+        timing_end(ctx, KC_ATTENTION, 2.0 * (double)(slot0 + m) * e->kv_width * kv_elem(e),
+                   4.0 * (double)(slot0 + m) * e->q_width * m);
     }
     EX(matvec_stream_prepared(lw.out, 0, m));
     EX(add_and_norm(e, h, lw.out, m, lw.post_ln, nullptr, lw.gate_up, false));

@@ -259,9 +259,12 @@ ctox_status launch_gemm(ctox_ctx *ctx, const GemmOperand &a, const GemmOperand &
             best = bn;
         }
     }
-    if (best == 256) return gemm_launch<256>(ctx, a, b, out);
-    if (best == 128) return gemm_launch<128>(ctx, a, b, out);
-    return gemm_launch<64>(ctx, a, b, out);
+    timing_begin(ctx);
+    EX(best == 256 ? gemm_launch<256>(ctx, a, b, out) : best == 128 ? gemm_launch<128>(ctx, a, b, out)
+                                                                   : gemm_launch<64>(ctx, a, b, out));
+    timing_end(ctx, KC_GEMM, 2.0 * ((double)a.rows + b.rows) * a.cols + (out.bf16 ? 2.0 : 4.0) * a.rows * b.rows,
+               2.0 * a.rows * b.rows * a.cols);
+    return CTOX_OK;
 }
 
 __global__ void k_rope_table(const float *__restrict__ freq, uint32_t pairs, uint32_t pos0, uint32_t rows,

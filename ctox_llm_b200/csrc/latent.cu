@@ -390,7 +390,7 @@ uint32_t latent_attn_splits(const ctox_ctx *ctx, const LatentAttn &a) {
     return s ? s : 1;
 }
 
-ctox_status launch_latent_attention(ctox_ctx *ctx, const LatentAttn &a, uint32_t splits) {
+static ctox_status latent_attention_any(ctox_ctx *ctx, const LatentAttn &a, uint32_t splits) {
     const uint32_t rows = a.m * a.heads, stages = mma_stages(ctx, a);
     if (stages) {
         const uint32_t row_tiles = (rows + kLaRowsMma - 1) / kLaRowsMma, nt = (a.kv_pad + 63) / 64;
@@ -413,6 +413,16 @@ ctox_status launch_latent_attention(ctox_ctx *ctx, const LatentAttn &a, uint32_t
               : fma_launch<T, 8>(ctx, a, splits, row_tiles, smem))
     return a.bf16 ? FMA(__nv_bfloat16) : FMA(float);
 #undef FMA
+}
+
+ctox_status launch_latent_attention(ctox_ctx *ctx, const LatentAttn &a, uint32_t splits) {
+    const KeyRange kr = key_range(a.pos0, a.m, a.window);
+    const double keys = kr.hi - kr.lo;
+    timing_begin(ctx);
+    EX(latent_attention_any(ctx, a, splits));
+    timing_end(ctx, KC_LATENT_ATTENTION, keys * (a.kv_pad + a.rot_pad) * (a.bf16 ? 2 : 4),
+               2.0 * keys * a.m * a.heads * (2 * a.kv_pad + a.rot_pad));
+    return CTOX_OK;
 }
 
 }  // namespace ctox

@@ -291,8 +291,17 @@ ctox_status launch_latent_prefill(ctox_ctx *ctx, const LatentPrefill &a) {
     EX(tensor_map_bf16(ctx, &mv, a.vt, (uint64_t)a.heads * a.vdim_pad, a.span, a.vt_ld, a.vdim_pad, kLpK));
     CTOX_CUDA(ctx, cudaFuncSetAttribute(k_latent_prefill, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     const uint32_t grid = (a.m + kLpQ - 1) / kLpQ * a.heads;
+    timing_begin(ctx);
     CTOX_CUDA(ctx, launch_pdl(k_latent_prefill, dim3(grid), dim3(kLpThreads), smem, ctx->stream, mq, mqr, mk, mkr, mv, a,
                               stages, cols, ctx->dev_error));
+    double pairs = 0;  // visible (query, key) pairs
+    if (ctx->timing)
+        for (uint32_t i = 0; i < a.m; ++i) {
+            const uint32_t seen = a.pos0 + i + 1;
+            pairs += a.window && seen > a.window ? a.window : seen;
+        }
+    timing_end(ctx, KC_LATENT_PREFILL, 2.0 * (a.m * (qw + (double)a.heads * a.vdim_pad) + a.span * (kw + (double)a.heads * a.vdim_pad)),
+               2.0 * pairs * a.heads * (a.dim_pad + a.rot_pad + a.vdim_pad));
     return CTOX_OK;
 }
 

@@ -46,7 +46,11 @@ def open_model(folder: str, backend: Optional[B200Backend] = None, dtype: str = 
     config = read_config(folder)
     backend = backend or B200Backend()
     executor = _OPENERS[config["architecture"]](backend, folder, config, dtype, max_context_tokens, **options)
-    executor.warmup()
+    try:
+        executor.warmup()
+    except Exception:
+        executor.unload()
+        raise
     return executor
 
 

@@ -80,7 +80,11 @@ def load_weights(weights: SafetensorsFile, ex: B200Executor) -> None:
 
 def open_lomelorn(backend, folder, config, dtype, max_context_tokens, **options):
     ex = B200Executor(backend, stack_config(config, dtype, max_context_tokens, **options))
-    load_weights(SafetensorsFile(os.path.join(folder, "model.safetensors")), ex)
+    try:
+        load_weights(SafetensorsFile(os.path.join(folder, "model.safetensors")), ex)
+    except Exception:
+        ex.unload()
+        raise
     return ex
 
 

@@ -158,6 +158,17 @@ uint64_t ctox_kernel_launches(void);
  * summed duration and the number of launches since the last read, and clears. */
 ctox_status ctox_ctx_kernel_timing(ctox_ctx *ctx, int32_t enable);
 ctox_status ctox_ctx_kernel_timing_read(ctox_ctx *ctx, double *total_ms, uint64_t *launches);
+/* The same for every kernel family that is bracketed (the read above reports class 0 alone); both reads
+ * clear. Classes: 0 packed streaming matvec, 1 attention of the hybrid model (with its merge), 2 dense
+ * matvec, 3 latent attention of short passes, 4 tensor-core product, 5 latent attention of long passes,
+ * 6 norms of long passes. bytes / flops: algorithmic work (0 where not counted). */
+#define CTOX_KERNEL_CLASSES 8
+typedef struct {
+    double ms;
+    uint64_t launches;
+    double bytes, flops;
+} ctox_kernel_class;
+ctox_status ctox_ctx_kernel_timing_classes(ctox_ctx *ctx, ctox_kernel_class *classes);
 /* backend/mod.rs:153-156: kind()/promotion_state()/profile() */
 const char *ctox_backend_profile(void);
 uint32_t ctox_abi_version(void);

@@ -48,6 +48,37 @@ def test_plain_greedy_decode_matches_oracle(setup):
     assert ex.position() == len(PROMPT) - 1 + n_new
 
 
+def test_extend_in_portions_equals_prefill(setup):
+    """ctox_exec_extend on top of a session: logits of wanted tokens against the oracle, and the same
+    drafts and tokens afterwards as with one prefill (the MTP cache stays exact across portions)."""
+    be, ex, model = setup
+    exp_tokens, exp_logits, _ = model.greedy(PROMPT, 2)
+    ex.reset_session()
+    ex.extend(PROMPT[:4])
+    got = ex.extend(PROMPT[4:], [0, len(PROMPT) - 5])
+    assert rel_l2(got[1], exp_logits[0]) <= 1e-3
+    assert rel_l2(got[0], model.greedy(PROMPT[:5], 1)[1][0]) <= 1e-3
+    assert ex.position() == len(PROMPT) and ex.decode(exp_tokens[0], mtp_enabled=False).token_id == exp_tokens[1]
+    long = PROMPT * 3
+    runs = []
+    for cuts in (None, (3, 8, 9, 20)):
+        if cuts is None:
+            ex.prefill(long)
+        else:
+            ex.reset_session()
+            edges = [0] + list(cuts) + [len(long) - 1]
+            for a, b in zip(edges, edges[1:]):
+                ex.extend(long[a:b])
+        tok, blocks = long[-1], []
+        for _ in range(4):
+            blk = ex.decode(tok, mtp_enabled=True)
+            blocks.append((blk.draft_tokens, blk.emitted))
+            tok = blk.token_id
+        runs.append(blocks)
+    assert runs[0] == runs[1]
+    assert list(ex.generate(PROMPT, 2)) == exp_tokens
+
+
 def test_mtp_greedy_emits_the_same_sequence(setup):
     be, ex, model = setup
     n_new = 24
