@@ -9,6 +9,30 @@
 namespace ctox {
 
 constexpr int kDvThreads = 256, kDvWarps = kDvThreads / 32;
+constexpr uint32_t kBatch = 4;                               // vectors a thread requests at once
+constexpr int kSplitLanes = (kAttnSplitsDense + 31) / 32;  // splits per lane of a merging warp
+
+// Columns c .. c + 3 of p, zero from `end` on.
+__device__ __forceinline__ float4 load4(const float *p, uint32_t c, uint32_t end, bool vec) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c + 4 <= end && vec) return *reinterpret_cast<const float4 *>(p + c);
+    if (c < end) v.x = p[c];
+    if (c + 1 < end) v.y = p[c + 1];
+    if (c + 2 < end) v.z = p[c + 2];
+    if (c + 3 < end) v.w = p[c + 3];
+    return v;
+}
+__device__ __forceinline__ void store4(float *p, uint32_t c, uint32_t end, const float4 &v) {
+    if (c + 4 <= end && ((uintptr_t)p & 15) == 0) {
+        *reinterpret_cast<float4 *>(p + c) = v;
+        return;
+    }
+    if (c < end) p[c] = v.x;
+    if (c + 1 < end) p[c + 1] = v.y;
+    if (c + 2 < end) p[c + 2] = v.z;
+    if (c + 3 < end) p[c + 3] = v.w;
+}
+__device__ __forceinline__ void prefetch_l1(const void *p) { asm volatile("prefetch.global.L1 [%0];" ::"l"(p)); }
 
 // Sum over the kDvThreads / M threads of a position (whole warps); every thread of the CTA calls it.
 template <int M>
@@ -65,7 +89,7 @@ __device__ void latent_append_row(const LatentAppend &a, uint32_t m, uint32_t ti
 // columns as [half][lane][4]. The first weights of every warp are requested before the dependency
 // wait (they are constants), so they arrive while the prologue forms the input.
 template <int M, int R>
-__global__ void __launch_bounds__(kDvThreads, 2)
+__global__ void __launch_bounds__(kDvThreads, M <= 2 ? 3 : 2)
     k_dense_matvec(const __nv_bfloat16 *__restrict__ W, uint32_t ld, uint32_t rows_per_group, uint32_t units_per_group,
                    uint32_t units, uint32_t ks, uint32_t lpr_log2, uint32_t npos, VecIn in, VecOut out,
                    LatentAppend ap, uint32_t append_positions) {
@@ -99,92 +123,156 @@ __global__ void __launch_bounds__(kDvThreads, 2)
                 dst[r] = __ldg(reinterpret_cast<const uint4 *>(base + (size_t)(row0 + r) * ld + c));
         }
     };
-    // ---- the input of `group`, normalised, into xs
+    // ---- the input of `group`, normalised, into xs. Loads are issued in batches of kBatch vectors before
+    // anything is stored, so that a thread waits for one round trip per batch.
+    constexpr uint32_t T = kDvThreads / M;
+    const uint32_t pm = tid / T, pt = tid % T;  // position and thread within it
+    float *xm = xs + pm * ldx;
+    const uint32_t cols = in.cols;
+    auto at = [&](uint32_t c) { return c / span * span + ((c >> 2) & 1) * (lpr * 4) + (c % span) / 8 * 4; };  // c % 4 == 0
+    auto slot4 = [&](uint32_t c) -> float4 & { return *reinterpret_cast<float4 *>(xm + at(c)); };
+    auto each = [&](uint32_t end, auto &&f) {
+        for (uint32_t c = pt * 4; c < end; c += T * 4) f(c);
+    };
     auto stage = [&](uint32_t group) {
-        constexpr uint32_t T = kDvThreads / M;
-        const uint32_t m = tid / T, t = tid % T;
-        const bool live = m < npos;
-        float *xm = xs + m * ldx;
-        auto at = [&](uint32_t c) { return c / span * span + ((c >> 2) & 1) * (lpr * 4) + (c % span) / 8 * 4 + (c & 3); };
-        const uint32_t cols = in.cols;
+        const bool live = pm < npos;
+        const uint32_t end = live ? cols : 0;
         if (in.ws_o) {
-            const size_t row = (size_t)m * in.groups + group;
-            if (live) {
-                float mx = -INFINITY;
-                for (uint32_t s = 0; s < in.splits; ++s) mx = fmaxf(mx, in.ws_ml[((size_t)s * in.ws_rows + row) * 2]);
-                float den = 0.f;
-                for (uint32_t s = 0; s < in.splits; ++s) {
-                    const float *ml = in.ws_ml + ((size_t)s * in.ws_rows + row) * 2;
-                    den += ml[1] * expf(ml[0] - mx);
+            const size_t row = (size_t)pm * in.groups + group;
+            if (live) {  // every warp forms the weights of the splits: lane = split and split + 32
+                float mv[kSplitLanes], sv[kSplitLanes], mx = -INFINITY, den = 0.f;
+#pragma unroll
+                for (int i = 0; i < kSplitLanes; ++i) {
+                    const uint32_t sp = lane + i * 32;
+                    const float2 ml = sp < in.splits ? *reinterpret_cast<const float2 *>(in.ws_ml + ((size_t)sp * in.ws_rows + row) * 2)
+                                                     : make_float2(-INFINITY, 0.f);
+                    mv[i] = ml.x;
+                    sv[i] = ml.y;
+                    mx = fmaxf(mx, ml.x);
                 }
-                for (uint32_t s = t; s < in.splits; s += T)
-                    mw[m][s] = expf(in.ws_ml[((size_t)s * in.ws_rows + row) * 2] - mx) / den;
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+#pragma unroll
+                for (int i = 0; i < kSplitLanes; ++i) {
+                    mv[i] = mv[i] == -INFINITY ? 0.f : expf(mv[i] - mx);
+                    den += sv[i] * mv[i];
+                }
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
+                if (pt < 32)
+#pragma unroll
+                    for (int i = 0; i < kSplitLanes; ++i) mw[pm][lane + i * 32] = mv[i] / den;
             }
             __syncthreads();
-            for (uint32_t c = t; c < ldx; c += T) {
-                float v = 0.f;
-                if (live && c < cols)
-                    for (uint32_t s = 0; s < in.splits; ++s)
-                        v += mw[m][s] * in.ws_o[((size_t)s * in.ws_rows + row) * cols + c];
-                xm[at(c)] = v;
-            }
+            each(ldx, [&](uint32_t c) {
+                float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (c < end)
+                    for (uint32_t s0 = 0; s0 < in.splits; s0 += kBatch * 2) {
+                        float4 o[kBatch * 2];
+#pragma unroll
+                        for (uint32_t i = 0; i < kBatch * 2; ++i)
+                            o[i] = s0 + i < in.splits ? *reinterpret_cast<const float4 *>(in.ws_o + ((size_t)(s0 + i) * in.ws_rows + row) * cols + c)
+                                                      : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+                        for (uint32_t i = 0; i < kBatch * 2; ++i) {
+                            const float w = s0 + i < in.splits ? mw[pm][s0 + i] : 0.f;
+                            v.x = fmaf(w, o[i].x, v.x);
+                            v.y = fmaf(w, o[i].y, v.y);
+                            v.z = fmaf(w, o[i].z, v.z);
+                            v.w = fmaf(w, o[i].w, v.w);
+                        }
+                    }
+                slot4(c) = v;
+            });
             return;
         }
-        const float *x = in.x + (size_t)m * in.x_stride + (size_t)group * in.x_group;
-        if (in.norm == NORM_NONE) {
-            for (uint32_t c = t; c < ldx; c += T) xm[at(c)] = live && c < cols ? x[c] : 0.f;
-            return;
-        }
-        float s = 0.f;
-        if (in.norm == NORM_RMS) {
-            for (uint32_t c = t; c < ldx; c += T) {
-                const float v = live && c < cols ? x[c] : 0.f;
-                xm[at(c)] = v;
-                s += v * v;
-            }
-            const float inv = 1.0f / sqrtf(position_sum<M>(s, red) / (float)cols + in.eps);
-            for (uint32_t c = t; c < cols; c += T) xm[at(c)] *= inv * in.w[c];
-            return;
-        }
-        const float n = (float)cols;
-        float mean = 0.f, inv = 0.f;
-        if (in.y) {
-            const float *y = in.y + (size_t)m * in.y_stride;
-            for (uint32_t c = t; c < cols; c += T) {
-                const float v = live ? y[c] : 0.f;
-                xm[at(c)] = v;
-                s += v;
-            }
-            mean = position_sum<M>(s, red) / n;
-            s = 0.f;
-            for (uint32_t c = t; c < cols; c += T) {
-                const float d = xm[at(c)] - mean;
-                s += d * d;
-            }
-            inv = 1.0f / sqrtf(position_sum<M>(s, red) / n + in.eps);
-        }
-        s = 0.f;
-        for (uint32_t c = t; c < ldx; c += T) {
-            float v = 0.f;
-            if (live && c < cols) {
-                v = x[c];
-                if (in.y) {
-                    v += (xm[at(c)] - mean) * inv * in.wb[c];
-                    if (blockIdx.x == 0) in.x_out[(size_t)m * in.x_stride + c] = v;
+        const float *x = in.x + (size_t)pm * in.x_stride + (size_t)group * in.x_group;
+        // f(c, values of p at c .. c + 3, values of q) for this thread's columns below `until`; zero from `end` on
+        auto stream = [&](const float *p, const float *q, uint32_t until, auto &&f) {
+            const bool vec_p = ((uintptr_t)p & 15) == 0, vec_q = ((uintptr_t)q & 15) == 0;
+            for (uint32_t c0 = pt * 4; c0 < until; c0 += T * 4 * kBatch) {
+                float4 a[kBatch], b[kBatch];
+#pragma unroll
+                for (uint32_t i = 0; i < kBatch; ++i) {
+                    const uint32_t c = c0 + i * T * 4;
+                    a[i] = load4(p, c, end, vec_p);
+                    if (q) b[i] = load4(q, c, end, vec_q);
+                }
+#pragma unroll
+                for (uint32_t i = 0; i < kBatch; ++i) {
+                    const uint32_t c = c0 + i * T * 4;
+                    if (c < until) f(c, a[i], b[i]);
                 }
             }
-            xm[at(c)] = v;
-            s += v;
+        };
+        if (in.norm == NORM_NONE) {
+            stream(x, nullptr, ldx, [&](uint32_t c, const float4 &v, const float4 &) { slot4(c) = v; });
+            return;
         }
+        auto sum4 = [](const float4 &v) { return (v.x + v.y) + (v.z + v.w); };
+        auto sq4 = [](const float4 &v) { return (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); };
+        const float n = (float)cols;
+        float s = 0.f;
+        if (in.norm == NORM_RMS) {
+            stream(x, nullptr, ldx, [&](uint32_t c, const float4 &v, const float4 &) {
+                slot4(c) = v;
+                s += sq4(v);
+            });
+            const float inv = 1.0f / sqrtf(position_sum<M>(s, red) / n + in.eps);
+            stream(in.w, nullptr, end, [&](uint32_t c, const float4 &w, const float4 &) {
+                float4 v = slot4(c);
+                slot4(c) = make_float4(v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w);
+            });
+            return;
+        }
+        // sum of squared deviations of what xs holds (columns past the last one do not count)
+        auto deviations = [&](float mean) {
+            float q = 0.f;
+            each(end, [&](uint32_t c) {
+                float4 v = slot4(c);
+                v = make_float4(v.x - mean, c + 1 < cols ? v.y - mean : 0.f, c + 2 < cols ? v.z - mean : 0.f,
+                                c + 3 < cols ? v.w - mean : 0.f);
+                q += sq4(v);
+            });
+            return q;
+        };
+        float mean = 0.f, inv = 0.f;
+        if (in.y) {
+            stream(in.y + (size_t)pm * in.y_stride, nullptr, end, [&](uint32_t c, const float4 &v, const float4 &) {
+                slot4(c) = v;
+                s += sum4(v);
+            });
+            mean = position_sum<M>(s, red) / n;
+            inv = 1.0f / sqrtf(position_sum<M>(deviations(mean), red) / n + in.eps);
+            s = 0.f;
+        }
+        stream(x, in.y ? in.wb : nullptr, ldx, [&](uint32_t c, const float4 &xv, const float4 &wb) {
+            float4 v = xv;
+            if (in.y && c < end) {
+                const float4 y = slot4(c);
+                v.x += (y.x - mean) * inv * wb.x;
+                v.y += (y.y - mean) * inv * wb.y;  // the weight is zero past the last column
+                v.z += (y.z - mean) * inv * wb.z;
+                v.w += (y.w - mean) * inv * wb.w;
+                if (blockIdx.x == 0) store4(in.x_out + (size_t)pm * in.x_stride, c, cols, v);
+            }
+            slot4(c) = v;
+            s += sum4(v);
+        });
         mean = position_sum<M>(s, red) / n;
-        s = 0.f;
-        for (uint32_t c = t; c < cols; c += T) {
-            const float d = xm[at(c)] - mean;
-            s += d * d;
-        }
-        inv = 1.0f / sqrtf(position_sum<M>(s, red) / n + in.eps);
-        for (uint32_t c = t; c < cols; c += T) xm[at(c)] = (xm[at(c)] - mean) * inv * in.w[c];
+        inv = 1.0f / sqrtf(position_sum<M>(deviations(mean), red) / n + in.eps);
+        stream(in.w, nullptr, end, [&](uint32_t c, const float4 &w, const float4 &) {
+            const float4 v = slot4(c);
+            slot4(c) = make_float4((v.x - mean) * inv * w.x, (v.y - mean) * inv * w.y, (v.z - mean) * inv * w.z,
+                                   (v.w - mean) * inv * w.w);
+        });
     };
+    // norm weights are constants: bring their lines in before the wait
+    if (in.w)
+        each(cols, [&](uint32_t c) {
+            prefetch_l1(in.w + c);
+            if (in.y) prefetch_l1(in.wb + c);
+        });
 
     uint32_t staged = 0xffffffffu;
     for (uint32_t unit = blockIdx.x; unit < units; unit += grid) {
@@ -377,46 +465,76 @@ constexpr int kSnThreads = 256;
 __global__ void __launch_bounds__(kSnThreads) k_stream_norm(StreamNorm a) {
     pdl_launch();
     pdl_wait();
-    extern __shared__ float v_s[];  // [width]
+    extern __shared__ __align__(16) float v_s[];  // [width rounded up to 4]
     __shared__ float red[kDvWarps];
-    const uint32_t row = a.rows ? a.rows[blockIdx.x] : blockIdx.x, tid = threadIdx.x;
-    const float n = (float)a.width;
-    const float *x = a.x + (size_t)row * a.width;
-    float s = 0.f, mean = 0.f, inv = 0.f;
-    if (a.y) {
-        const float *y = a.y + (size_t)row * a.width;
-        for (uint32_t c = tid; c < a.width; c += kSnThreads) {
-            const float v = y[c];
-            v_s[c] = v;
-            s += v;
+    const uint32_t row = a.rows ? a.rows[blockIdx.x] : blockIdx.x, tid = threadIdx.x, W = a.width;
+    const float n = (float)W;
+    const float *x = a.x + (size_t)row * W, *y = a.y ? a.y + (size_t)row * W : nullptr;
+    auto slot4 = [&](uint32_t c) -> float4 & { return *reinterpret_cast<float4 *>(v_s + c); };
+    auto stream = [&](const float *p, const float *q, auto &&f) {  // batches of loads, then the work on them
+        const bool vec_p = ((uintptr_t)p & 15) == 0, vec_q = ((uintptr_t)q & 15) == 0;
+        for (uint32_t c0 = tid * 4; c0 < W; c0 += kSnThreads * 4 * kBatch) {
+            float4 u[kBatch], v[kBatch];
+#pragma unroll
+            for (uint32_t i = 0; i < kBatch; ++i) {
+                u[i] = load4(p, c0 + i * kSnThreads * 4, W, vec_p);
+                if (q) v[i] = load4(q, c0 + i * kSnThreads * 4, W, vec_q);
+            }
+#pragma unroll
+            for (uint32_t i = 0; i < kBatch; ++i)
+                if (c0 + i * kSnThreads * 4 < W) f(c0 + i * kSnThreads * 4, u[i], v[i]);
         }
+    };
+    auto deviations = [&](float mean) {
+        float q = 0.f;
+        for (uint32_t c = tid * 4; c < W; c += kSnThreads * 4) {
+            const float4 v = slot4(c);
+            const float d0 = v.x - mean, d1 = c + 1 < W ? v.y - mean : 0.f, d2 = c + 2 < W ? v.z - mean : 0.f,
+                        d3 = c + 3 < W ? v.w - mean : 0.f;
+            q += (d0 * d0 + d1 * d1) + (d2 * d2 + d3 * d3);
+        }
+        return q;
+    };
+    float s = 0.f, mean = 0.f, inv = 0.f;
+    if (y) {
+        stream(y, nullptr, [&](uint32_t c, const float4 &v, const float4 &) {
+            slot4(c) = v;
+            s += (v.x + v.y) + (v.z + v.w);
+        });
         mean = position_sum<1>(s, red) / n;
+        inv = 1.0f / sqrtf(position_sum<1>(deviations(mean), red) / n + a.eps);
         s = 0.f;
-        for (uint32_t c = tid; c < a.width; c += kSnThreads) s += (v_s[c] - mean) * (v_s[c] - mean);
-        inv = 1.0f / sqrtf(position_sum<1>(s, red) / n + a.eps);
     }
-    s = 0.f;
-    for (uint32_t c = tid; c < a.width; c += kSnThreads) {
-        float v = x[c];
-        if (a.y) v += (v_s[c] - mean) * inv * a.wb[c];
-        if (a.x_out) a.x_out[(size_t)row * a.width + c] = v;
-        v_s[c] = v;
-        s += v;
-    }
+    stream(x, y ? a.wb : nullptr, [&](uint32_t c, const float4 &xv, const float4 &wb) {
+        float4 v = xv;
+        if (y) {
+            const float4 u = slot4(c);
+            v.x += (u.x - mean) * inv * wb.x;
+            v.y += (u.y - mean) * inv * wb.y;  // the weight is zero past the last column
+            v.z += (u.z - mean) * inv * wb.z;
+            v.w += (u.w - mean) * inv * wb.w;
+        }
+        if (a.x_out) store4(a.x_out + (size_t)row * W, c, W, v);
+        slot4(c) = v;
+        s += (v.x + v.y) + (v.z + v.w);
+    });
     if (!a.w) return;
     mean = position_sum<1>(s, red) / n;
-    s = 0.f;
-    for (uint32_t c = tid; c < a.width; c += kSnThreads) s += (v_s[c] - mean) * (v_s[c] - mean);
-    inv = 1.0f / sqrtf(position_sum<1>(s, red) / n + a.eps);
-    for (uint32_t c = tid; c < a.width; c += kSnThreads) {
-        const float v = (v_s[c] - mean) * inv * a.w[c];
-        if (a.f32_out) a.f32_out[(size_t)blockIdx.x * a.width + c] = v;
-        if (a.bf16_out) a.bf16_out[(size_t)blockIdx.x * a.bf16_ld + c] = __float2bfloat16_rn(v);
-    }
+    inv = 1.0f / sqrtf(position_sum<1>(deviations(mean), red) / n + a.eps);
+    stream(a.w, nullptr, [&](uint32_t c, const float4 &w, const float4 &) {
+        const float4 u = slot4(c);
+        const float4 v = make_float4((u.x - mean) * inv * w.x, (u.y - mean) * inv * w.y, (u.z - mean) * inv * w.z,
+                                     (u.w - mean) * inv * w.w);
+        if (a.f32_out) store4(a.f32_out + (size_t)blockIdx.x * W, c, W, v);
+        if (a.bf16_out) {  // rows are padded to whole vectors of eight
+            const __nv_bfloat162 h[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
+            *reinterpret_cast<uint2 *>(a.bf16_out + (size_t)blockIdx.x * a.bf16_ld + c) = *reinterpret_cast<const uint2 *>(h);
+        }
+    });
 }
 
 ctox_status launch_stream_norm(ctox_ctx *ctx, const StreamNorm &a, uint32_t m) {
-    const size_t smem = (size_t)a.width * 4;
+    const size_t smem = ((size_t)a.width + 3) / 4 * 16;
     if (smem + 1024 > (size_t)ctx->max_smem_optin)
         return fail(ctx, CTOX_MEMORY_BUDGET, "stream norm: width %u does not fit shared memory", a.width);
     if (smem > 40 * 1024)

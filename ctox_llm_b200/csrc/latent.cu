@@ -191,15 +191,31 @@ __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAt
     };
     if (t_beg < t_end) load_tile(t_beg, 0);
     const float qscale = a.scale * 1.4426950408889634f;  // scores in units of log 2
-    for (uint32_t i = tid; i < kLaRowsMma * D; i += kLaThreads) {
-        const uint32_t r = i / D, c = i % D, row = row0 + r;
-        float v = 0.f;
-        if (row < rows)
-            v = (c < a.kv_pad ? a.q_abs[(size_t)row * a.kv_pad + c] : a.q_rot[(size_t)row * a.q_stride + c - a.kv_pad]) * qscale;
-        __nv_bfloat16 hi, lo;
-        split_bf16(v, hi, lo);
-        q_s[r * ld + c] = hi;
-        q_s[(kLaRowsMma + r) * ld + c] = lo;
+    // two rows per warp; a lane requests kQ vectors of a row before it stores any
+    constexpr uint32_t kQ = 5;
+    for (uint32_t r = warp; r < kLaRowsMma; r += kLaWarps) {
+        const uint32_t row = row0 + r;
+        const float *qa = a.q_abs + (size_t)row * a.kv_pad, *qr = a.q_rot + (size_t)row * a.q_stride;
+        for (uint32_t c0 = lane * 4; c0 < D; c0 += 128 * kQ) {
+            float4 v[kQ];
+#pragma unroll
+            for (uint32_t i = 0; i < kQ; ++i) {
+                const uint32_t c = c0 + i * 128;
+                v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (row < rows && c < D) v[i] = *reinterpret_cast<const float4 *>(c < a.kv_pad ? qa + c : qr + (c - a.kv_pad));
+            }
+#pragma unroll
+            for (uint32_t i = 0; i < kQ; ++i) {
+                const uint32_t c = c0 + i * 128;
+                if (c >= D) break;
+                const float f[4] = {v[i].x * qscale, v[i].y * qscale, v[i].z * qscale, v[i].w * qscale};
+                __nv_bfloat16 hi[4], lo[4];
+#pragma unroll
+                for (int j = 0; j < 4; ++j) split_bf16(f[j], hi[j], lo[j]);
+                *reinterpret_cast<uint2 *>(q_s + r * ld + c) = *reinterpret_cast<uint2 *>(hi);
+                *reinterpret_cast<uint2 *>(q_s + (kLaRowsMma + r) * ld + c) = *reinterpret_cast<uint2 *>(lo);
+            }
+        }
     }
     float o[NT][4];
 #pragma unroll

@@ -2,10 +2,10 @@
 //
 // Scores and the weighted sum run on tcgen05.mma with operands staged by TMA; scores (double-buffered) and
 // the output accumulate in tensor memory. One warp loads, one issues the products, four hold one query
-// row per thread for the softmax: they read the scores from tensor memory, write the weights to shared
-// memory as the next product's operand, and rescale the output only when a row's maximum has grown by more
-// than 2^8 since its last reference (the final division is exact either way). Two CTAs share an SM when
-// their buffers fit, so one's softmax overlaps the other's products.
+// row per thread for the softmax: they read the scores from tensor memory, write the weights over them as
+// the next product's operand, and rescale the output only when a row's maximum has grown by more than 2^8
+// since its last reference (the final division makes up for it). Two CTAs share an SM when their buffers
+// fit, so one's softmax overlaps the other's products.
 #include "latent.cuh"
 #include "umma.cuh"
 
@@ -33,7 +33,7 @@ __device__ __forceinline__ float ex2(float x) {
 __global__ void __launch_bounds__(kLpThreads)
     k_latent_prefill(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_qr,
                      const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_kr,
-                     const __grid_constant__ CUtensorMap map_v, LatentPrefill a, uint32_t stages, uint32_t tmem_cols,
+                     const __grid_constant__ CUtensorMap map_v, LatentPrefill a, uint32_t k_stages, uint32_t v_stages, uint32_t tmem_cols,
                      int32_t *error_word) {
     using namespace umma;
     pdl_launch();
@@ -46,7 +46,7 @@ __global__ void __launch_bounds__(kLpThreads)
     const LpBox bd = lp_box(a.dim_pad), br = lp_box(a.rot_pad);
     const uint32_t q_bytes = kLpQ * D * 2, k_bytes = kLpK * D * 2, v_bytes = a.vdim_pad * kLpK * 2;
     const uint32_t base = (smem_addr(raw) + 1023) & ~1023u;
-    const uint32_t q_s = base, p_s = q_s + q_bytes, k_s = p_s + kLpQ * kLpK * 2, v_s = k_s + stages * k_bytes;
+    const uint32_t q_s = base, k_s = q_s + q_bytes, v_s = k_s + k_stages * k_bytes;
     const uint32_t b0 = smem_addr(bars), q_full = b0, k_full = b0 + 8, k_empty = b0 + 24, v_full = b0 + 40,
                    v_empty = b0 + 56, s_full = b0 + 72, p_full = b0 + 88, o_done = b0 + 96, drained = b0 + 104;
     if (tid == 0) {
@@ -86,7 +86,8 @@ __global__ void __launch_bounds__(kLpThreads)
             uint32_t k_issued = 0, v_issued = 0;
             bool ok = true;
             for (uint32_t j = 0; j < n; ++j) {
-                const uint32_t s = j % stages, round = j / stages, row = (t_lo + j) * kLpK;
+                const uint32_t row = (t_lo + j) * kLpK, s = j % k_stages, round = j / k_stages, vs = j % v_stages,
+                               v_round = j / v_stages;
                 if (round > 0 && !(ok = bar_wait(k_empty + s * 8, (round - 1) & 1, &dead))) break;
                 const uint32_t pos = a.row0 + row;
                 const int slot = (int)(a.page_table[pos / a.page_tokens] * a.page_tokens + pos % a.page_tokens);
@@ -98,23 +99,23 @@ __global__ void __launch_bounds__(kLpThreads)
                     tma_load(kd + kLpK * a.dim_pad * 2 + i * kLpK * br.width * 2, &map_kr, k_full + s * 8,
                              (int)(a.kv_pad + i * br.width), slot);
                 ++k_issued;
-                if (round > 0 && !(ok = bar_wait(v_empty + s * 8, (round - 1) & 1, &dead))) break;
-                bar_expect(v_full + s * 8, v_bytes);
-                tma_load(v_s + s * v_bytes, &map_v, v_full + s * 8, (int)row, (int)(head * a.vdim_pad));
+                if (v_round > 0 && !(ok = bar_wait(v_empty + vs * 8, (v_round - 1) & 1, &dead))) break;
+                bar_expect(v_full + vs * 8, v_bytes);
+                tma_load(v_s + vs * v_bytes, &map_v, v_full + vs * 8, (int)row, (int)(head * a.vdim_pad));
                 ++v_issued;
             }
             if (!ok) {  // leave no copy in flight behind
                 bar_drain(q_full, 0);
-                for (uint32_t s = 0; s < stages && s < k_issued; ++s) bar_drain(k_full + s * 8, ((k_issued - 1 - s) / stages) & 1);
-                for (uint32_t s = 0; s < stages && s < v_issued; ++s) bar_drain(v_full + s * 8, ((v_issued - 1 - s) / stages) & 1);
+                for (uint32_t s = 0; s < k_stages && s < k_issued; ++s) bar_drain(k_full + s * 8, ((k_issued - 1 - s) / k_stages) & 1);
+                for (uint32_t s = 0; s < v_stages && s < v_issued; ++s) bar_drain(v_full + s * 8, ((v_issued - 1 - s) / v_stages) & 1);
             }
         }
     } else if (warp == 1) {
         if (lane == 0) {
             const uint32_t idesc_s = idesc_bf16(kLpQ, kLpK), idesc_o = idesc_bf16(kLpQ, a.vdim_pad);
             auto scores = [&](uint32_t j) -> bool {
-                const uint32_t s = j % stages;
-                if (!bar_wait(k_full + s * 8, (j / stages) & 1, &dead)) return false;
+                const uint32_t s = j % k_stages;
+                if (!bar_wait(k_full + s * 8, (j / k_stages) & 1, &dead)) return false;
                 fence_after();
                 const uint32_t d = tmem + (j & 1) * kLpK, kd = k_s + s * k_bytes;
                 bool acc = false;
@@ -134,12 +135,13 @@ __global__ void __launch_bounds__(kLpThreads)
             bool ok = bar_wait(q_full, 0, &dead) && scores(0);
             for (uint32_t j = 0; j < n && ok; ++j) {
                 if (j + 1 < n && !(ok = scores(j + 1))) break;
-                const uint32_t s = j % stages;
-                if (!(ok = bar_wait(p_full, j & 1, &dead) && bar_wait(v_full + s * 8, (j / stages) & 1, &dead))) break;
+                const uint32_t s = j % v_stages;
+                if (!(ok = bar_wait(p_full, j & 1, &dead) && bar_wait(v_full + s * 8, (j / v_stages) & 1, &dead))) break;
                 fence_after();
-                const uint64_t dp = smem_desc(p_s, 128), dv = smem_desc(v_s + s * v_bytes, 128);
+                const uint32_t p = tmem + (j & 1) * kLpK;  // the weights, where the scores were
+                const uint64_t dv = smem_desc(v_s + s * v_bytes, 128);
 #pragma unroll
-                for (uint32_t k = 0; k < kLpK / 16; ++k) mma_f16(tmem_o, dp + k * 2, dv + k * 2, idesc_o, j > 0 || k > 0);
+                for (uint32_t k = 0; k < kLpK / 16; ++k) mma_f16_ts(tmem_o, p + k * 8, dv + k * 2, idesc_o, j > 0 || k > 0);
                 commit(v_empty + s * 8);
                 commit(o_done);
             }
@@ -153,7 +155,7 @@ __global__ void __launch_bounds__(kLpThreads)
         const uint32_t lanes = (quarter * 32) << 16;
         const uint32_t pos = a.pos0 + i0 + row;
         const float c = a.scale * 1.4426950408889634f;
-        float ref = -INFINITY, sum = 0.f;
+        float ref = -INFINITY, sum[4] = {0.f, 0.f, 0.f, 0.f};
         bool ok = true;
         for (uint32_t j = 0; j < n; ++j) {
             if (!(ok = __all_sync(0xffffffffu, bar_wait(s_full + (j & 1) * 8, (j >> 1) & 1, &dead)))) break;
@@ -171,23 +173,21 @@ __global__ void __launch_bounds__(kLpThreads)
                     if (t > pos || (a.window && pos - t >= a.window)) s[k] = -INFINITY;
                 }
             }
-            float mx = s[0];
+            float m4[4] = {s[0], s[1], s[2], s[3]};
 #pragma unroll
-            for (uint32_t k = 1; k < kLpK; ++k) mx = fmaxf(mx, s[k]);
-            mx *= c;
-            // P and O belong to the product of the tile before until it has finished
-            if (j > 0) {
-                if (!(ok = __all_sync(0xffffffffu, bar_wait(o_done, (j - 1) & 1, &dead)))) break;
-                fence_after();
-            }
+            for (uint32_t k = 4; k < kLpK; ++k) m4[k & 3] = fmaxf(m4[k & 3], s[k]);
+            const float mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])) * c;
             const bool grow = mx > ref + 8.f || (ref == -INFINITY && mx > ref);
             if (__any_sync(0xffffffffu, grow)) {
                 const float f = grow ? ex2(ref - mx) : 1.f;  // ref = -inf: 0, and nothing but zeros was added
                 if (grow) {
                     ref = mx;
-                    sum *= f;
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) sum[i] *= f;
                 }
-                if (j > 0) {
+                if (j > 0) {  // the output belongs to the product of the tile before until that has finished
+                    if (!(ok = __all_sync(0xffffffffu, bar_wait(o_done, (j - 1) & 1, &dead)))) break;
+                    fence_after();
                     for (uint32_t d = 0; d < a.vdim_pad; d += 16) {
                         float o[16];
                         tmem_ld16(tmem_o + d + lanes, o);
@@ -196,37 +196,30 @@ __global__ void __launch_bounds__(kLpThreads)
                         for (int i = 0; i < 16; ++i) o[i] *= f;
                         tmem_st16(tmem_o + d + lanes, o);
                     }
-                    tmem_st_wait();
                 }
             }
             const float r = ref == -INFINITY ? 0.f : ref;
-            const uint32_t dst = p_s + row * 128;
+            uint32_t p[kLpK / 2];
 #pragma unroll
-            for (uint32_t k = 0; k < kLpK; k += 8) {
-                float p[8];
-#pragma unroll
-                for (int i = 0; i < 8; ++i) {
-                    p[i] = ex2(fmaf(s[k + i], c, -r));
-                    sum += p[i];
-                }
-                uint32_t h[4];
-#pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    const __nv_bfloat162 b = __floats2bfloat162_rn(p[2 * i], p[2 * i + 1]);
-                    h[i] = *reinterpret_cast<const uint32_t *>(&b);
-                }
-                asm volatile("st.shared.v4.b32 [%0], {%1,%2,%3,%4};" ::"r"(dst + (((k >> 3) ^ (row & 7)) << 4)), "r"(h[0]),
-                             "r"(h[1]), "r"(h[2]), "r"(h[3])
-                             : "memory");
+            for (uint32_t k = 0; k < kLpK; k += 2) {
+                const float a0 = ex2(fmaf(s[k], c, -r)), a1 = ex2(fmaf(s[k + 1], c, -r));
+                sum[k & 2] += a0;
+                sum[(k & 2) + 1] += a1;
+                const __nv_bfloat162 b = __floats2bfloat162_rn(a0, a1);
+                p[k / 2] = *reinterpret_cast<const uint32_t *>(&b);
             }
-            fence_smem_async();
+            tmem_st32(tmem + (j & 1) * kLpK + lanes, p);
+            tmem_st_wait();
             fence_before();
             __syncwarp();
             if (lane == 0) bar_arrive(p_full);
         }
+        // A wait tells a phase from its neighbours only. Having seen the scores of tile j, the products up to
+        // tile j - 2 are known to be complete: the last two are waited for in turn.
+        if (ok && n > 1) ok = __all_sync(0xffffffffu, bar_wait(o_done, (n - 2) & 1, &dead));
         if (ok && (ok = __all_sync(0xffffffffu, bar_wait(o_done, (n - 1) & 1, &dead)))) {
             fence_after();
-            const float inv = 1.0f / sum;
+            const float inv = 1.0f / ((sum[0] + sum[1]) + (sum[2] + sum[3]));
             __nv_bfloat16 *out = a.out + ((size_t)(i0 + row) * a.heads + head) * a.vdim_pad;
             for (uint32_t d = 0; d < a.vdim_pad; d += 16) {
                 float o[16];
@@ -257,27 +250,33 @@ __global__ void __launch_bounds__(kLpThreads)
 
 namespace {
 
-size_t lp_smem(uint32_t dim_pad, uint32_t rot_pad, uint32_t vdim_pad, uint32_t stages) {
+size_t lp_smem(uint32_t dim_pad, uint32_t rot_pad, uint32_t vdim_pad, uint32_t k_stages, uint32_t v_stages) {
     const size_t D = dim_pad + rot_pad;
-    return 1024 + kLpQ * D * 2 + kLpQ * kLpK * 2 + stages * (kLpK * D * 2 + (size_t)vdim_pad * kLpK * 2);
+    return 1024 + kLpQ * D * 2 + k_stages * kLpK * D * 2 + (size_t)v_stages * vdim_pad * kLpK * 2;
 }
 
 }  // namespace
 
 bool latent_prefill_fits(const ctox_ctx *ctx, uint32_t dim_pad, uint32_t rot_pad, uint32_t vdim_pad) {
-    return vdim_pad <= 256 && lp_smem(dim_pad, rot_pad, vdim_pad, 1) + 1024 <= (size_t)ctx->max_smem_optin;
+    return vdim_pad <= 256 && lp_smem(dim_pad, rot_pad, vdim_pad, 1, 1) + 1024 <= (size_t)ctx->max_smem_optin;
 }
 
 ctox_status launch_latent_prefill(ctox_ctx *ctx, const LatentPrefill &a) {
     if (!latent_prefill_fits(ctx, a.dim_pad, a.rot_pad, a.vdim_pad) || a.page_tokens % kLpQ || a.row0 % kLpQ || a.vt_ld % 8)
         return fail(ctx, CTOX_SHAPE, "latent prefill: unsupported sizes");
     const size_t half = ((size_t)ctx->max_smem_optin - 2048) / 2 - 1024;  // two CTAs on an SM
-    uint32_t stages = 2;
-    size_t smem = lp_smem(a.dim_pad, a.rot_pad, a.vdim_pad, 2);
-    if (smem > half && (lp_smem(a.dim_pad, a.rot_pad, a.vdim_pad, 1) <= half || smem + 1024 > (size_t)ctx->max_smem_optin)) {
-        stages = 1;
-        smem = lp_smem(a.dim_pad, a.rot_pad, a.vdim_pad, 1);
+    // the deepest buffering that lets two CTAs share an SM; else the deepest that fits one
+    uint32_t ks = 0, vs = 0;
+    for (size_t limit : {half, (size_t)ctx->max_smem_optin - 1024}) {
+        for (uint32_t i = 0; i < 4 && !ks; ++i) {
+            const uint32_t k = i < 2 ? 2 : 1, v = i == 0 || i == 2 ? 2 : 1;
+            if (lp_smem(a.dim_pad, a.rot_pad, a.vdim_pad, k, v) <= limit) {
+                ks = k;
+                vs = v;
+            }
+        }
     }
+    const size_t smem = lp_smem(a.dim_pad, a.rot_pad, a.vdim_pad, ks, vs);
     uint32_t cols = 256;  // scores 2 x 64 and the output
     if (2 * kLpK + a.vdim_pad > 256) cols = 512;
     const LpBox bd = lp_box(a.dim_pad), br = a.rot_pad ? lp_box(a.rot_pad) : LpBox{16, 0};
@@ -293,7 +292,7 @@ ctox_status launch_latent_prefill(ctox_ctx *ctx, const LatentPrefill &a) {
     const uint32_t grid = (a.m + kLpQ - 1) / kLpQ * a.heads;
     timing_begin(ctx);
     CTOX_CUDA(ctx, launch_pdl(k_latent_prefill, dim3(grid), dim3(kLpThreads), smem, ctx->stream, mq, mqr, mk, mkr, mv, a,
-                              stages, cols, ctx->dev_error));
+                              ks, vs, cols, ctx->dev_error));
     double pairs = 0;  // visible (query, key) pairs
     if (ctx->timing)
         for (uint32_t i = 0; i < a.m; ++i) {

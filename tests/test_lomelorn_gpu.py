@@ -103,6 +103,22 @@ def test_whole_prompt_portions_and_single_tokens(opened, name, dtype):
     assert close(single, want[:60], dtype)
 
 
+def test_portions_of_a_tile_again_and_again(opened):
+    """Few key tiles per pass and many passes: the last products of a tile row are the ones just issued."""
+    config, t = model([layer(heads=10, dim=32, rot_dim=16, vdim=80, window=100), layer(heads=6, dim=64, rot_dim=32, vdim=48, window=60)],
+                      seed=8)
+    tokens = tokens_of(700, config["vocab"], 4)
+    want, _ = oracle.forward(config, t, tokens)
+    ex = opened(config, t, "bfloat16")
+    first = None
+    for size in (64, 63, 37, 130) * 5:
+        got = run(ex, tokens, range(size, 700, size))
+        assert close(got, want, "bfloat16"), size
+        if size == 64:
+            first = got if first is None else first
+            assert np.array_equal(got, first)
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_passes_of_every_short_length(opened, dtype):
     config, t = MODELS["mixed"]()
