@@ -821,6 +821,9 @@ LATENT_SIZES = {
                kv_rank=512, window=4096, hybrid_heads=(24, 4)),
     "7k": dict(width=7168, layers=4, vocab=32768, ff=18432, heads=128, dim=128, rot_dim=64, vdim=128, q_rank=1536,
                kv_rank=512, window=4096, hybrid_heads=(32, 8)),
+    # a window as wide as the context: what latent attention reads is then of the hybrid cache's order
+    "5k-wide": dict(width=5120, layers=4, vocab=32768, ff=17408, heads=40, dim=128, rot_dim=64, vdim=128, q_rank=1536,
+                    kv_rank=512, window=32768, context=32768, hybrid_heads=(24, 4)),
 }
 
 
@@ -828,7 +831,7 @@ def run_latent(args):
     """The layer-stack model (Lomelorn: latent attention, window 4096, bf16 weights) beside the closest
     existing model, the hybrid with full attention in every layer, at the same width, depth, feed-forward
     and vocabulary: decode at a context of 8192 tokens and prefill of one 4096-token prompt, through the
-    executor's own calls, random weights. Per kernel family: device time with an event pair around every
+    executor's own calls, random weights ("5k-wide": window and context 32768). Per kernel family: device time with an event pair around every
     launch (serialised), and the fraction of its roofline (the larger of bytes / measured copy bandwidth and
     flops / measured bf16 product)."""
     import torch
@@ -845,7 +848,7 @@ def run_latent(args):
     if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")):
         with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
             tflops = float(json.load(f)["bf16_tflops"])
-    context, prompt_n = 8192, 4096
+    prompt_n = 4096
     prompt = [int(t) for t in np.random.default_rng(0).integers(0, 32768, prompt_n)]
 
     def stack(z):
@@ -854,13 +857,14 @@ def run_latent(args):
                      score_scale=(z["dim"] + z["rot_dim"]) ** -0.5, mlp=N.MLP_RELU2, ff=z["ff"])
         return ctox.StackConfig(vocab_size=z["vocab"], hidden_size=z["width"], norm_eps=1e-6, logit_softcap=30.0,
                                 layers=[N.LayerConfig(**layer) for _ in range(z["layers"])],
-                                max_context_tokens=context + 1024, pass_tokens=args.pass_tokens)
+                                max_context_tokens=z.get("context", 8192) + 1024, pass_tokens=args.pass_tokens)
 
     def hybrid(z):
         return ctox.qwen38_27b_config(
             vocab_size=z["vocab"], hidden_size=z["width"], intermediate_size=z["ff"], num_hidden_layers=z["layers"],
             num_attention_heads=z["hybrid_heads"][0], num_key_value_heads=z["hybrid_heads"][1], full_attention_interval=1,
-            mtp_num_hidden_layers=0, draft_vocab=0, max_draft_tokens=0, max_context_tokens=context + 1024)
+            mtp_num_hidden_layers=0, draft_vocab=0, max_draft_tokens=0,
+            max_context_tokens=z.get("context", 8192) + 1024)
 
     def families(work):
         be.kernel_timing(True)
@@ -874,7 +878,7 @@ def run_latent(args):
                 k["roofline_frac"] = ideal / k["ms"]
         return out
 
-    def measure(config):
+    def measure(config, context):
         ex = ctox.B200Executor(be, config)
         ex.fill_synthetic(seed=0)
         ex.warmup()
@@ -923,15 +927,15 @@ def run_latent(args):
     with torch.cuda.stream(stream):
         for name in args.sizes.split(","):
             z = LATENT_SIZES[name]
-            sweep[name] = {"shape": z, "lomelorn": measure(stack(z))}
+            sweep[name] = {"shape": z, "lomelorn": measure(stack(z), z.get("context", 8192))}
             if not args.quick:
-                sweep[name]["hybrid"] = measure(hybrid(z))
+                sweep[name]["hybrid"] = measure(hybrid(z), z.get("context", 8192))
     last = sweep[args.sizes.split(",")[-1] if "5k" not in sweep else "5k"]["lomelorn"]
     line = {"metric": "latent_decode_tokens_per_s", "value": last["decode"]["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
             "steps": args.steps, "warmup": max(args.warmup, 3), "ms_per_step": last["decode"]["ms"], "higher_is_better": True,
             "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
             "config": {"workload": "layer stack (latent attention) beside the hybrid model with full attention at equal width, "
-                                   f"depth, feed-forward and vocabulary; decode at context {context}, prefill of {prompt_n} tokens",
+                                   f"depth, feed-forward and vocabulary; decode at context 8192 (5k-wide: 32768), prefill of {prompt_n} tokens",
                        "l2": "a pass streams more weights than twice the L2"},
             "e2e": {"value": last["decode"]["e2e_tokens_per_s"], "unit": "tokens/s", "h2d_bytes_per_step": 4,
                     "d2h_bytes_per_step": 300},
@@ -957,7 +961,7 @@ def main():
     ap.add_argument("--replicas", type=int, default=0,
                     help="matvec: weight replicas to rotate (default: enough to exceed twice the L2; 1 = weights "
                          "stay in L2, a diagnostic that separates the instruction cost from the HBM stream)")
-    ap.add_argument("--sizes", default="2k,5k,7k", help="latent: sizes to run")
+    ap.add_argument("--sizes", default="2k,5k,7k,5k-wide", help="latent: sizes to run")
     ap.add_argument("--pass-tokens", type=int, default=0, help="latent: prompt tokens per pass (0: the default)")
     ap.add_argument("--context", type=int, default=32768)
     ap.add_argument("--drafts", type=int, default=3,

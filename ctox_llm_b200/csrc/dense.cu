@@ -9,6 +9,7 @@
 namespace ctox {
 
 constexpr int kDvThreads = 256, kDvWarps = kDvThreads / 32;
+constexpr uint64_t kUnitCost = 8000;                         // of a unit of rows, in columns
 constexpr uint32_t kBatch = 4;                               // vectors a thread requests at once
 constexpr int kSplitLanes = (kAttnSplitsDense + 31) / 32;  // splits per lane of a merging warp
 
@@ -89,7 +90,7 @@ __device__ void latent_append_row(const LatentAppend &a, uint32_t m, uint32_t ti
 // columns as [half][lane][4]. The first weights of every warp are requested before the dependency
 // wait (they are constants), so they arrive while the prologue forms the input.
 template <int M, int R>
-__global__ void __launch_bounds__(kDvThreads, M <= 2 ? 3 : 2)
+__global__ void __launch_bounds__(kDvThreads, 2)
     k_dense_matvec(const __nv_bfloat16 *__restrict__ W, uint32_t ld, uint32_t rows_per_group, uint32_t units_per_group,
                    uint32_t units, uint32_t ks, uint32_t lpr_log2, uint32_t npos, VecIn in, VecOut out,
                    LatentAppend ap, uint32_t append_positions) {
@@ -436,11 +437,22 @@ ctox_status launch_dense_matvec(ctox_ctx *ctx, const DenseMat &w, uint32_t group
         }
         o.y += (size_t)p * o.y_stride;
         o.pos0 += p;
-        // enough warps to cover the machine: fewer rows per warp, then several warps per row
-        const uint32_t want = (uint32_t)ctx->sm_count * 16, nsub = 32u >> lpr_log2;
-        const uint32_t R = M <= 2 && w.rows / (4 * nsub) >= want ? 4 : 2;
-        uint32_t ks = 1;
-        while (ks < kDvWarps && w.rows / (R * nsub) * ks < want && nsteps / (2 * ks) >= 2) ks *= 2;
+        // Rows per warp (R) and warps per row (ks): the least work of the busiest CTA with two CTAs per SM,
+        // a unit's fixed cost counted as some columns.
+        const uint32_t rows = w.rows / groups, nsub = 32u >> lpr_log2, fit = 2 * (uint32_t)ctx->sm_count;
+        uint32_t R = 2, ks = 1;
+        uint64_t best = ~0ull;
+        for (uint32_t r = 2; r <= (M <= 2 ? 4u : 2u); r *= 2)
+            for (uint32_t k = 1; k <= kDvWarps && k <= nsteps; k *= 2) {
+                const uint32_t unit = kDvWarps / k * nsub * r, units = (rows + unit - 1) / unit * groups;
+                const uint64_t cols = (uint64_t)((nsteps + k - 1) / k) * k * span;
+                const uint64_t cost = (uint64_t)((units + fit - 1) / fit) * (unit * cols + kUnitCost);
+                if (cost < best) {
+                    best = cost;
+                    R = r;
+                    ks = k;
+                }
+            }
         const uint32_t na = append && p == 0 ? m : 0;
         const size_t smem = M * row_bytes;
         ctox_status rc;

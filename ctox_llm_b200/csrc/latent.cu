@@ -190,6 +190,7 @@ __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAt
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     if (t_beg < t_end) load_tile(t_beg, 0);
+    if (stages == 2 && t_beg + 1 < t_end) load_tile(t_beg + 1, 1);
     const float qscale = a.scale * 1.4426950408889634f;  // scores in units of log 2
     // two rows per warp; a lane requests kQ vectors of a row before it stores any
     constexpr uint32_t kQ = 5;
@@ -226,9 +227,7 @@ __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAt
     const uint32_t p_addr = smem_u32(p_s + (lane & 15) * kLdP + (lane >> 4) * 8);
     for (uint32_t tile = t_beg; tile < t_end; ++tile) {
         const uint32_t st = stages == 2 ? (tile - t_beg) & 1 : 0;
-        const bool ahead = stages == 2 && tile + 1 < t_end;
-        if (ahead) load_tile(tile + 1, st ^ 1);
-        if (ahead)
+        if (stages == 2 && tile + 1 < t_end)  // the next tile may still be on its way
             asm volatile("cp.async.wait_group 1;" ::: "memory");
         else
             asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -239,6 +238,7 @@ __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAt
 #pragma unroll
         for (int i = 0; i < 4; ++i) s4[i][0] = s4[i][1] = s4[i][2] = s4[i][3] = 0.f;
         const uint32_t k_addr = smem_u32(kt + (warp * 8 + (lane & 7)) * ld + ((lane >> 3) & 1) * 8);
+#pragma unroll 4
         for (uint32_t k = 0; k < D; k += 16) {
             uint32_t ah[4], al[4], b[2];
             ldsm_x4(ah, q_addr + k * 2);
@@ -322,7 +322,7 @@ __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAt
             }
         }
         __syncthreads();
-        if (stages == 1 && tile + 1 < t_end) load_tile(tile + 1, 0);
+        if (tile + stages < t_end) load_tile(tile + stages, st);  // into the buffer just read
     }
 #pragma unroll
     for (int i = 0; i < 2; ++i) {

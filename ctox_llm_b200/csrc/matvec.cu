@@ -962,7 +962,7 @@ ctox_status matvec_stream_prepared(ctox_matvec *mv, size_t part_index, uint32_t 
         launch_stream<1>(cfg, grid, smem, ctx->stream, sp);
     else
         launch_stream<0>(cfg, grid, smem, ctx->stream, sp);
-    timing_end(ctx);
+    timing_end(ctx, KC_STREAM_MATVEC, (double)p.prep_bytes, 2.0 * (double)p.rows * (double)mv->columns * npos);
     CTOX_CUDA(ctx, cudaGetLastError());
     return CTOX_OK;
 }
