@@ -9,7 +9,7 @@
 namespace ctox {
 
 constexpr int kDvThreads = 256, kDvWarps = kDvThreads / 32;
-constexpr uint64_t kUnitCost = 8000;                         // of a unit of rows, in columns
+constexpr uint64_t kUnitCost = 20000;                        // of a unit of rows, in columns
 constexpr uint32_t kBatch = 4;                               // vectors a thread requests at once
 constexpr int kSplitLanes = (kAttnSplitsDense + 31) / 32;  // splits per lane of a merging warp
 

@@ -15,7 +15,7 @@
 namespace ctox {
 
 constexpr uint32_t kDensePass = 8;       // positions per pass of the matrix-vector form
-constexpr uint32_t kAttnSplitsDense = 32;  // most context splits a merge prologue takes
+constexpr uint32_t kAttnSplitsDense = 64;  // most context splits a merge prologue takes
 
 // Row-major [rows][ld] bf16, ld = columns rounded up to 8 (16-byte rows), padding zero.
 struct DenseMat {

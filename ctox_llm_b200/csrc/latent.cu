@@ -134,9 +134,6 @@ __device__ __forceinline__ void ldsm_x4(uint32_t *r, uint32_t addr) {
                  : "r"(addr)
                  : "memory");
 }
-__device__ __forceinline__ void ldsm_x2(uint32_t *r, uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr) : "memory");
-}
 __device__ __forceinline__ void ldsm_x4_t(uint32_t *r, uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
@@ -153,20 +150,25 @@ __device__ __forceinline__ void split_bf16(float v, __nv_bfloat16 &hi, __nv_bflo
     lo = __float2bfloat16_rn(v - __bfloat162float(hi));
 }
 
-// Sixteen query rows against 64-token tiles of cache rows. Scores: each warp eight tokens over the whole
-// row; weighted sum: each warp every eighth group of eight latent columns, the same tile read as the
+// Sixteen query rows against 64-token tiles of cache rows. The row dimension is dealt to the warps in steps
+// of 16 values, so a warp keeps its part of the queries in registers and reads its part of a tile once;
+// the partial scores meet in shared memory, where sixteen threads hold a query row for the softmax.
+// Weighted sum: each warp every eighth group of eight latent columns, the same tile read as the
 // transposed operand. Queries and weights are split into two bf16 parts (about 16 bits), so the only bf16
-// rounding is the cache's. NT: groups of eight columns per warp.
+// rounding is the cache's. NT: groups of eight latent columns per warp.
+__host__ __device__ constexpr int la_steps(int nt) { return nt <= 2 ? 2 : nt / 2 + 1; }  // 16-value steps of a row per warp
+constexpr uint32_t kLaLdP = kLaTileMma + 8, kLaLdS = kLaTileMma + 4;
+
 template <int NT>
 __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAttn a, uint32_t splits, uint32_t stages) {
+    constexpr int NK = la_steps(NT);
     pdl_launch();
     extern __shared__ __align__(16) uint8_t smraw[];
-    constexpr uint32_t kLdP = kLaTileMma + 8;
     const uint32_t D = a.kv_pad + a.rot_pad, ld = D + 8, rows = a.m * a.heads;
-    __nv_bfloat16 *k_s = reinterpret_cast<__nv_bfloat16 *>(smraw);                // [stages][64][ld]
-    __nv_bfloat16 *q_s = k_s + (size_t)stages * kLaTileMma * ld;                   // [hi, lo][16][ld]
-    __nv_bfloat16 *p_s = q_s + 2 * kLaRowsMma * ld;                                // [hi, lo][16][kLdP]
-    float *red = reinterpret_cast<float *>(p_s + 2 * kLaRowsMma * kLdP);           // [8][16]
+    __nv_bfloat16 *k_s = reinterpret_cast<__nv_bfloat16 *>(smraw);           // [stages][64][ld]
+    float *s_s = reinterpret_cast<float *>(k_s + (size_t)stages * kLaTileMma * ld);  // [8 warps][16][kLaLdS]
+    __nv_bfloat16 *p_s = reinterpret_cast<__nv_bfloat16 *>(s_s + kLaWarps * kLaRowsMma * kLaLdS);  // [hi, lo][16][kLaLdP]
+    float *al_s = reinterpret_cast<float *>(p_s + 2 * kLaRowsMma * kLaLdP);  // [16]
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
     const uint32_t row0 = blockIdx.x * kLaRowsMma, sp = blockIdx.y;
     const KeyRange kr = key_range(a.pos0, a.m, a.window);
@@ -191,40 +193,39 @@ __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAt
     };
     if (t_beg < t_end) load_tile(t_beg, 0);
     if (stages == 2 && t_beg + 1 < t_end) load_tile(t_beg + 1, 1);
+    // ---- this warp's part of the queries: steps warp, warp + 8, ... as operand fragments
     const float qscale = a.scale * 1.4426950408889634f;  // scores in units of log 2
-    // two rows per warp; a lane requests kQ vectors of a row before it stores any
-    constexpr uint32_t kQ = 5;
-    for (uint32_t r = warp; r < kLaRowsMma; r += kLaWarps) {
-        const uint32_t row = row0 + r;
-        const float *qa = a.q_abs + (size_t)row * a.kv_pad, *qr = a.q_rot + (size_t)row * a.q_stride;
-        for (uint32_t c0 = lane * 4; c0 < D; c0 += 128 * kQ) {
-            float4 v[kQ];
+    uint32_t qh[NK][4], ql[NK][4];
+    {
+        float2 v[NK][4];
 #pragma unroll
-            for (uint32_t i = 0; i < kQ; ++i) {
-                const uint32_t c = c0 + i * 128;
-                v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-                if (row < rows && c < D) v[i] = *reinterpret_cast<const float4 *>(c < a.kv_pad ? qa + c : qr + (c - a.kv_pad));
+        for (int i = 0; i < NK; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {  // rows g, g + 8; values 2 t4 and 2 t4 + 8
+                const uint32_t row = row0 + g + (j & 1) * 8, c = (warp + i * kLaWarps) * 16 + t4 * 2 + (j >> 1) * 8;
+                v[i][j] = make_float2(0.f, 0.f);
+                if (row < rows && c < D)
+                    v[i][j] = *reinterpret_cast<const float2 *>(c < a.kv_pad ? a.q_abs + (size_t)row * a.kv_pad + c
+                                                                             : a.q_rot + (size_t)row * a.q_stride + (c - a.kv_pad));
             }
 #pragma unroll
-            for (uint32_t i = 0; i < kQ; ++i) {
-                const uint32_t c = c0 + i * 128;
-                if (c >= D) break;
-                const float f[4] = {v[i].x * qscale, v[i].y * qscale, v[i].z * qscale, v[i].w * qscale};
-                __nv_bfloat16 hi[4], lo[4];
+        for (int i = 0; i < NK; ++i)
 #pragma unroll
-                for (int j = 0; j < 4; ++j) split_bf16(f[j], hi[j], lo[j]);
-                *reinterpret_cast<uint2 *>(q_s + r * ld + c) = *reinterpret_cast<uint2 *>(hi);
-                *reinterpret_cast<uint2 *>(q_s + (kLaRowsMma + r) * ld + c) = *reinterpret_cast<uint2 *>(lo);
+            for (int j = 0; j < 4; ++j) {
+                __nv_bfloat162 hi, lo;
+                split_bf16(v[i][j].x * qscale, hi.x, lo.x);
+                split_bf16(v[i][j].y * qscale, hi.y, lo.y);
+                qh[i][j] = *reinterpret_cast<uint32_t *>(&hi);
+                ql[i][j] = *reinterpret_cast<uint32_t *>(&lo);
             }
-        }
     }
     float o[NT][4];
 #pragma unroll
     for (int j = 0; j < NT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-    float mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.f, 0.f};  // rows g, g + 8
-    const uint32_t pos_a = a.pos0 + (row0 + g) / a.heads, pos_b = a.pos0 + (row0 + g + 8) / a.heads;
-    const uint32_t q_addr = smem_u32(q_s + (lane & 15) * ld + (lane >> 4) * 8);
-    const uint32_t p_addr = smem_u32(p_s + (lane & 15) * kLdP + (lane >> 4) * 8);
+    // softmax: thread = (query row, four tokens of a tile)
+    const uint32_t srow = tid >> 4, stok = (tid & 15) * 4, qrow = row0 + srow, qpos = a.pos0 + qrow / a.heads;
+    float mx = -INFINITY, sum = 0.f;
+    const uint32_t p_addr = smem_u32(p_s + (lane & 15) * kLaLdP + (lane >> 4) * 8);
     for (uint32_t tile = t_beg; tile < t_end; ++tile) {
         const uint32_t st = stages == 2 ? (tile - t_beg) & 1 : 0;
         if (stages == 2 && tile + 1 < t_end)  // the next tile may still be on its way
@@ -233,71 +234,75 @@ __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAt
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         const __nv_bfloat16 *kt = k_s + (size_t)st * kLaTileMma * ld;
-        // ---- scores of tokens warp * 8 .. + 8
-        float s4[4][4];
+        // ---- partial scores over this warp's steps
+        float s[8][4];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) s4[i][0] = s4[i][1] = s4[i][2] = s4[i][3] = 0.f;
-        const uint32_t k_addr = smem_u32(kt + (warp * 8 + (lane & 7)) * ld + ((lane >> 3) & 1) * 8);
-#pragma unroll 4
-        for (uint32_t k = 0; k < D; k += 16) {
-            uint32_t ah[4], al[4], b[2];
-            ldsm_x4(ah, q_addr + k * 2);
-            ldsm_x4(al, q_addr + kLaRowsMma * ld * 2 + k * 2);
-            ldsm_x2(b, k_addr + k * 2);
-            if ((k >> 4) & 1) {
-                mma_bf16(s4[2], ah, b);
-                mma_bf16(s4[3], al, b);
-            } else {
-                mma_bf16(s4[0], ah, b);
-                mma_bf16(s4[1], al, b);
+        for (int n = 0; n < 8; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+        const uint32_t k_addr = smem_u32(kt + ((lane & 7) + (lane >> 4) * 8) * ld + ((lane >> 3) & 1) * 8);
+#pragma unroll
+        for (int i = 0; i < NK; ++i) {
+            const uint32_t c = (warp + i * kLaWarps) * 16;
+            if (c < D) {
+#pragma unroll
+                for (int n = 0; n < 8; n += 2) {  // two groups of eight tokens per load
+                    uint32_t b[4];
+                    ldsm_x4(b, k_addr + (n * 8 * ld + c) * 2);
+                    mma_bf16(s[n], qh[i], b);
+                    mma_bf16(s[n + 1], qh[i], b + 2);
+                    mma_bf16(s[n], ql[i], b);
+                    mma_bf16(s[n + 1], ql[i], b + 2);
+                }
             }
         }
-        float s[4];
+        float *sw = s_s + warp * kLaRowsMma * kLaLdS;
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            s[i] = (s4[0][i] + s4[2][i]) + (s4[1][i] + s4[3][i]);
-            const uint32_t t = kr.lo + tile * kLaTileMma + warp * 8 + t4 * 2 + (i & 1);
-            const uint32_t row = row0 + g + (i >= 2 ? 8 : 0);
-            if (row >= rows || t >= kr.hi || !key_visible(t, i >= 2 ? pos_b : pos_a, a.window)) s[i] = -INFINITY;
-        }
-        float tm[2] = {fmaxf(s[0], s[1]), fmaxf(s[2], s[3])};
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            tm[i] = fmaxf(tm[i], __shfl_xor_sync(0xffffffffu, tm[i], 1));
-            tm[i] = fmaxf(tm[i], __shfl_xor_sync(0xffffffffu, tm[i], 2));
-        }
-        if (t4 == 0) {
-            red[warp * kLaRowsMma + g] = tm[0];
-            red[warp * kLaRowsMma + g + 8] = tm[1];
+        for (int n = 0; n < 8; ++n) {
+            *reinterpret_cast<float2 *>(sw + g * kLaLdS + n * 8 + t4 * 2) = make_float2(s[n][0], s[n][1]);
+            *reinterpret_cast<float2 *>(sw + (g + 8) * kLaLdS + n * 8 + t4 * 2) = make_float2(s[n][2], s[n][3]);
         }
         __syncthreads();
-        float alpha[2];
+        // ---- scores of one row's four tokens, softmax
+        float v[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            float nm = mx[i];
-#pragma unroll
-            for (int w = 0; w < kLaWarps; ++w) nm = fmaxf(nm, red[w * kLaRowsMma + g + i * 8]);
-            alpha[i] = nm == -INFINITY ? 1.f : exp2f(mx[i] - nm);
-            mx[i] = nm;
-            float p[2];
-#pragma unroll
-            for (int j = 0; j < 2; ++j) p[j] = s[i * 2 + j] == -INFINITY ? 0.f : exp2f(s[i * 2 + j] - nm);
-            sum[i] = sum[i] * alpha[i] + p[0] + p[1];
-            __nv_bfloat162 hi, lo;
-            split_bf16(p[0], hi.x, lo.x);
-            split_bf16(p[1], hi.y, lo.y);
-            __nv_bfloat16 *dst = p_s + (g + i * 8) * kLdP + warp * 8 + t4 * 2;
-            *reinterpret_cast<__nv_bfloat162 *>(dst) = hi;
-            *reinterpret_cast<__nv_bfloat162 *>(dst + kLaRowsMma * kLdP) = lo;
+        for (int w = 0; w < kLaWarps; ++w) {
+            const float4 q = *reinterpret_cast<const float4 *>(s_s + (w * kLaRowsMma + srow) * kLaLdS + stok);
+            v[0] += q.x;
+            v[1] += q.y;
+            v[2] += q.z;
+            v[3] += q.w;
         }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const uint32_t t = kr.lo + tile * kLaTileMma + stok + j;
+            if (qrow >= rows || t >= kr.hi || !key_visible(t, qpos, a.window)) v[j] = -INFINITY;
+        }
+        float nm = fmaxf(fmaxf(v[0], v[1]), fmaxf(v[2], v[3]));
+#pragma unroll
+        for (int off = 8; off > 0; off >>= 1) nm = fmaxf(nm, __shfl_xor_sync(0xffffffffu, nm, off));
+        nm = fmaxf(nm, mx);
+        const float alpha = nm == -INFINITY ? 1.f : exp2f(mx - nm);
+        mx = nm;
+        __nv_bfloat16 hi[4], lo[4];
+        float ps = 0.f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const float p = v[j] == -INFINITY ? 0.f : exp2f(v[j] - nm);
+            ps += p;
+            split_bf16(p, hi[j], lo[j]);
+        }
+        sum = sum * alpha + ps;  // this thread's tokens; the row is added up at the end
+        *reinterpret_cast<uint2 *>(p_s + srow * kLaLdP + stok) = *reinterpret_cast<uint2 *>(hi);
+        *reinterpret_cast<uint2 *>(p_s + (kLaRowsMma + srow) * kLaLdP + stok) = *reinterpret_cast<uint2 *>(lo);
+        if ((tid & 15) == 0) al_s[srow] = alpha;
         __syncthreads();
         // ---- weighted sum of the cache rows
+        const float al0 = al_s[g], al1 = al_s[g + 8];
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
-            o[j][0] *= alpha[0];
-            o[j][1] *= alpha[0];
-            o[j][2] *= alpha[1];
-            o[j][3] *= alpha[1];
+            o[j][0] *= al0;
+            o[j][1] *= al0;
+            o[j][2] *= al1;
+            o[j][3] *= al1;
         }
 #pragma unroll
         for (uint32_t k = 0; k < kLaTileMma; k += 32) {
@@ -305,7 +310,7 @@ __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAt
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
                 ldsm_x4(ph[i], p_addr + (k + i * 16) * 2);
-                ldsm_x4(pl[i], p_addr + kLaRowsMma * kLdP * 2 + (k + i * 16) * 2);
+                ldsm_x4(pl[i], p_addr + kLaRowsMma * kLaLdP * 2 + (k + i * 16) * 2);
             }
             const uint32_t v_addr = smem_u32(kt + (k + lane) * ld);
 #pragma unroll
@@ -325,26 +330,10 @@ __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAt
         if (tile + stages < t_end) load_tile(tile + stages, st);  // into the buffer just read
     }
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-        sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 1);
-        sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 2);
-    }
-    __syncthreads();
-    if (t4 == 0) {
-        red[warp * kLaRowsMma + g] = sum[0];
-        red[warp * kLaRowsMma + g + 8] = sum[1];
-    }
-    __syncthreads();
-    if (warp == 0 && t4 == 0) {
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const uint32_t row = row0 + g + i * 8;
-            if (row >= rows) continue;
-            float total = 0.f;
-            for (int w = 0; w < kLaWarps; ++w) total += red[w * kLaRowsMma + g + i * 8];
-            a.ws_ml[((size_t)sp * rows + row) * 2] = mx[i] * 0.6931471805599453f;
-            a.ws_ml[((size_t)sp * rows + row) * 2 + 1] = total;
-        }
+    for (int off = 8; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
+    if ((tid & 15) == 0 && qrow < rows) {
+        a.ws_ml[((size_t)sp * rows + qrow) * 2] = mx * 0.6931471805599453f;
+        a.ws_ml[((size_t)sp * rows + qrow) * 2 + 1] = sum;
     }
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
@@ -363,12 +352,18 @@ __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAt
 namespace {
 
 size_t mma_smem(const LatentAttn &a, uint32_t stages) {
-    const size_t ld = a.kv_pad + a.rot_pad + 8;
-    return (stages * kLaTileMma + 2 * kLaRowsMma) * ld * 2 + 2 * kLaRowsMma * (kLaTileMma + 8) * 2 + kLaWarps * kLaRowsMma * 4;
+    return (size_t)stages * kLaTileMma * (a.kv_pad + a.rot_pad + 8) * 2 + kLaWarps * kLaRowsMma * kLaLdS * 4 +
+           2 * kLaRowsMma * kLaLdP * 2 + kLaRowsMma * 4;
+}
+// Smallest form (NT) of the tensor-core kernel that takes these rows; 0: none does.
+int mma_form(const LatentAttn &a) {
+    for (int nt : {1, 2, 4, 8, 16})
+        if (a.kv_pad <= 64u * nt && a.kv_pad + a.rot_pad <= 128u * la_steps(nt)) return nt;
+    return 0;
 }
 // Tile stages of the tensor-core form (0: it does not apply).
 uint32_t mma_stages(const ctox_ctx *ctx, const LatentAttn &a) {
-    if (!a.bf16 || a.kv_pad > 1024) return 0;
+    if (!a.bf16 || !mma_form(a)) return 0;
     for (uint32_t st = 2; st > 0; --st)
         if (mma_smem(a, st) <= (size_t)ctx->max_smem_optin) return st;
     return 0;
@@ -401,7 +396,9 @@ uint32_t latent_attn_splits(const ctox_ctx *ctx, const LatentAttn &a) {
     const KeyRange kr = key_range(a.pos0, a.m, a.window);
     const uint32_t tiles = (kr.hi - kr.lo + tile - 1) / tile;
     uint32_t s = (uint32_t)ctx->sm_count / row_tiles;
-    if (s > kAttnSplitsDense) s = kAttnSplitsDense;
+    // every product that merges the splits reads them all: many only where they shorten a long chain of tiles
+    const uint32_t most = tiles >= 256 ? kAttnSplitsDense : kAttnSplitsDense / 2;
+    if (s > most) s = most;
     if (s > tiles) s = tiles;
     return s ? s : 1;
 }
@@ -409,13 +406,15 @@ uint32_t latent_attn_splits(const ctox_ctx *ctx, const LatentAttn &a) {
 static ctox_status latent_attention_any(ctox_ctx *ctx, const LatentAttn &a, uint32_t splits) {
     const uint32_t rows = a.m * a.heads, stages = mma_stages(ctx, a);
     if (stages) {
-        const uint32_t row_tiles = (rows + kLaRowsMma - 1) / kLaRowsMma, nt = (a.kv_pad + 63) / 64;
+        const uint32_t row_tiles = (rows + kLaRowsMma - 1) / kLaRowsMma;
         const size_t smem = mma_smem(a, stages);
-        if (nt <= 1) return mma_launch<1>(ctx, a, splits, row_tiles, smem, stages);
-        if (nt <= 2) return mma_launch<2>(ctx, a, splits, row_tiles, smem, stages);
-        if (nt <= 4) return mma_launch<4>(ctx, a, splits, row_tiles, smem, stages);
-        if (nt <= 8) return mma_launch<8>(ctx, a, splits, row_tiles, smem, stages);
-        return mma_launch<16>(ctx, a, splits, row_tiles, smem, stages);
+        switch (mma_form(a)) {
+            case 1: return mma_launch<1>(ctx, a, splits, row_tiles, smem, stages);
+            case 2: return mma_launch<2>(ctx, a, splits, row_tiles, smem, stages);
+            case 4: return mma_launch<4>(ctx, a, splits, row_tiles, smem, stages);
+            case 8: return mma_launch<8>(ctx, a, splits, row_tiles, smem, stages);
+            default: return mma_launch<16>(ctx, a, splits, row_tiles, smem, stages);
+        }
     }
     const size_t smem = fma_smem(a);
     const uint32_t row_tiles = (rows + kLaRowsFma - 1) / kLaRowsFma, j = (a.kv_pad + kLaThreads - 1) / kLaThreads;
