@@ -161,7 +161,7 @@ constexpr uint32_t kLaLdP = kLaTileMma + 8, kLaLdS = kLaTileMma + 4;
 
 template <int NT>
 __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAttn a, uint32_t splits, uint32_t stages) {
-    constexpr int NK = la_steps(NT);
+    constexpr int NK = la_steps(NT), JG = NT < 4 ? NT : 4;
     pdl_launch();
     extern __shared__ __align__(16) uint8_t smraw[];
     const uint32_t D = a.kv_pad + a.rot_pad, ld = D + 8, rows = a.m * a.heads;
@@ -177,12 +177,14 @@ __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAt
     const uint32_t chunks = D / 8;
     pdl_wait();
     auto load_tile = [&](uint32_t tile, uint32_t stage) {
-        const uint32_t t0 = kr.lo + tile * kLaTileMma;
-        for (uint32_t r = warp; r < kLaTileMma; r += kLaWarps) {
-            const uint32_t t = t0 + r;
-            const bool in = t < kr.hi;
-            const __nv_bfloat16 *src =
-                (const __nv_bfloat16 *)a.cache + (in ? paged_slot(a.page_table, a.page_tokens, t) * D : 0);
+        // lane i < 8 looks the slot of this warp's row i up, for all lanes
+        const uint32_t mine = kr.lo + tile * kLaTileMma + warp + (lane & 7) * kLaWarps;
+        const uint32_t slot = mine < kr.hi ? (uint32_t)paged_slot(a.page_table, a.page_tokens, mine) : 0xffffffffu;
+#pragma unroll
+        for (uint32_t i = 0; i < kLaTileMma / kLaWarps; ++i) {
+            const uint32_t r = warp + i * kLaWarps, from = __shfl_sync(0xffffffffu, slot, i);
+            const bool in = from != 0xffffffffu;
+            const __nv_bfloat16 *src = (const __nv_bfloat16 *)a.cache + (in ? (size_t)from * D : 0);
             __nv_bfloat16 *dst = k_s + ((size_t)stage * kLaTileMma + r) * ld;
             for (uint32_t c = lane; c < chunks; c += 32)
                 asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + c * 8)), "l"(src + c * 8),
@@ -244,13 +246,14 @@ __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAt
             const uint32_t c = (warp + i * kLaWarps) * 16;
             if (c < D) {
 #pragma unroll
-                for (int n = 0; n < 8; n += 2) {  // two groups of eight tokens per load
-                    uint32_t b[4];
+                for (int n = 0; n < 8; n += 4) {  // two groups of eight tokens per load
+                    uint32_t b[8];
                     ldsm_x4(b, k_addr + (n * 8 * ld + c) * 2);
-                    mma_bf16(s[n], qh[i], b);
-                    mma_bf16(s[n + 1], qh[i], b + 2);
-                    mma_bf16(s[n], ql[i], b);
-                    mma_bf16(s[n + 1], ql[i], b + 2);
+                    ldsm_x4(b + 4, k_addr + ((n + 2) * 8 * ld + c) * 2);
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) mma_bf16(s[n + k], qh[i], b + 2 * k);
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) mma_bf16(s[n + k], ql[i], b + 2 * k);
                 }
             }
         }
@@ -314,16 +317,21 @@ __global__ void __launch_bounds__(kLaThreads, 1) k_latent_attention_mma(LatentAt
             }
             const uint32_t v_addr = smem_u32(kt + (k + lane) * ld);
 #pragma unroll
-            for (int j = 0; j < NT; ++j) {
-                const uint32_t n = (warp + j * kLaWarps) * 8;
-                if (n < a.kv_pad) {
-                    uint32_t b[4];
-                    ldsm_x4_t(b, v_addr + n * 2);
-                    mma_bf16(o[j], ph[0], b);
-                    mma_bf16(o[j], pl[0], b);
-                    mma_bf16(o[j], ph[1], b + 2);
-                    mma_bf16(o[j], pl[1], b + 2);
+            for (int j0 = 0; j0 < NT; j0 += JG) {  // JG independent accumulators between dependent products
+                uint32_t b[JG][4];
+#pragma unroll
+                for (int j = 0; j < JG; ++j) {  // groups past the latent repeat the first (never stored)
+                    const uint32_t n = (warp + (j0 + j) * kLaWarps) * 8;
+                    ldsm_x4_t(b[j], v_addr + (n < a.kv_pad ? n : 0) * 2);
                 }
+#pragma unroll
+                for (int j = 0; j < JG; ++j) mma_bf16(o[j0 + j], ph[0], b[j]);
+#pragma unroll
+                for (int j = 0; j < JG; ++j) mma_bf16(o[j0 + j], pl[0], b[j]);
+#pragma unroll
+                for (int j = 0; j < JG; ++j) mma_bf16(o[j0 + j], ph[1], b[j] + 2);
+#pragma unroll
+                for (int j = 0; j < JG; ++j) mma_bf16(o[j0 + j], pl[1], b[j] + 2);
             }
         }
         __syncthreads();
