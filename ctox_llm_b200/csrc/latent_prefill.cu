@@ -38,7 +38,7 @@ __global__ void __launch_bounds__(kLpThreads)
     using namespace umma;
     pdl_launch();
     extern __shared__ uint8_t raw[];
-    __shared__ __align__(8) uint64_t bars[14];
+    __shared__ __align__(8) uint64_t bars[15];
     __shared__ uint32_t tmem_slot;
     __shared__ volatile int dead;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -48,7 +48,7 @@ __global__ void __launch_bounds__(kLpThreads)
     const uint32_t base = (smem_addr(raw) + 1023) & ~1023u;
     const uint32_t q_s = base, k_s = q_s + q_bytes, v_s = k_s + k_stages * k_bytes;
     const uint32_t b0 = smem_addr(bars), q_full = b0, k_full = b0 + 8, k_empty = b0 + 24, v_full = b0 + 40,
-                   v_empty = b0 + 56, s_full = b0 + 72, p_full = b0 + 88, o_done = b0 + 96, drained = b0 + 104;
+                   v_empty = b0 + 56, s_full = b0 + 72, p_full = b0 + 88, o_done = b0 + 96, drained = b0 + 112;
     if (tid == 0) {
         dead = 0;
         bar_init(q_full, 1);
@@ -58,9 +58,9 @@ __global__ void __launch_bounds__(kLpThreads)
             bar_init(v_full + i * 8, 1);
             bar_init(v_empty + i * 8, 1);
             bar_init(s_full + i * 8, 1);
+            bar_init(o_done + i * 8, 1);
         }
         bar_init(p_full, 4);
-        bar_init(o_done, 1);
         bar_init(drained, 1);
         bar_init_fence();
     }
@@ -143,7 +143,7 @@ __global__ void __launch_bounds__(kLpThreads)
 #pragma unroll
                 for (uint32_t k = 0; k < kLpK / 16; ++k) mma_f16_ts(tmem_o, p + k * 8, dv + k * 2, idesc_o, j > 0 || k > 0);
                 commit(v_empty + s * 8);
-                commit(o_done);
+                commit(o_done + (j & 1) * 8);
             }
             if (!ok) {
                 commit(drained);
@@ -186,7 +186,7 @@ __global__ void __launch_bounds__(kLpThreads)
                     for (int i = 0; i < 4; ++i) sum[i] *= f;
                 }
                 if (j > 0) {  // the output belongs to the product of the tile before until that has finished
-                    if (!(ok = __all_sync(0xffffffffu, bar_wait(o_done, (j - 1) & 1, &dead)))) break;
+                    if (!(ok = __all_sync(0xffffffffu, bar_wait(o_done + ((j - 1) & 1) * 8, ((j - 1) >> 1) & 1, &dead)))) break;
                     fence_after();
                     for (uint32_t d = 0; d < a.vdim_pad; d += 16) {
                         float o[16];
@@ -214,10 +214,11 @@ __global__ void __launch_bounds__(kLpThreads)
             __syncwarp();
             if (lane == 0) bar_arrive(p_full);
         }
-        // A wait tells a phase from its neighbours only. Having seen the scores of tile j, the products up to
-        // tile j - 2 are known to be complete: the last two are waited for in turn.
-        if (ok && n > 1) ok = __all_sync(0xffffffffu, bar_wait(o_done, (n - 2) & 1, &dead));
-        if (ok && (ok = __all_sync(0xffffffffu, bar_wait(o_done, (n - 1) & 1, &dead)))) {
+        // Most tiles skip the wait for the product before them, and a wait tells a phase from its neighbours
+        // only. Hence one barrier for even and one for odd tiles: having seen the scores of tile j, the
+        // products up to j - 2 are complete and the one of tile j + 1 cannot be, so either wait (here and at a
+        // rescale) meets its barrier in the phase it asks for or the one right before.
+        if (ok && (ok = __all_sync(0xffffffffu, bar_wait(o_done + ((n - 1) & 1) * 8, ((n - 1) >> 1) & 1, &dead)))) {
             fence_after();
             const float inv = 1.0f / ((sum[0] + sum[1]) + (sum[2] + sum[3]));
             __nv_bfloat16 *out = a.out + ((size_t)(i0 + row) * a.heads + head) * a.vdim_pad;
