@@ -38,7 +38,7 @@ __global__ void __launch_bounds__(kLpThreads)
     using namespace umma;
     pdl_launch();
     extern __shared__ uint8_t raw[];
-    __shared__ __align__(8) uint64_t bars[15];
+    __shared__ __align__(8) uint64_t bars[16];
     __shared__ uint32_t tmem_slot;
     __shared__ volatile int dead;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -48,7 +48,7 @@ __global__ void __launch_bounds__(kLpThreads)
     const uint32_t base = (smem_addr(raw) + 1023) & ~1023u;
     const uint32_t q_s = base, k_s = q_s + q_bytes, v_s = k_s + k_stages * k_bytes;
     const uint32_t b0 = smem_addr(bars), q_full = b0, k_full = b0 + 8, k_empty = b0 + 24, v_full = b0 + 40,
-                   v_empty = b0 + 56, s_full = b0 + 72, p_full = b0 + 88, o_done = b0 + 96, drained = b0 + 112;
+                   v_empty = b0 + 56, s_full = b0 + 72, p_full = b0 + 88, o_done = b0 + 104, drained = b0 + 120;
     if (tid == 0) {
         dead = 0;
         bar_init(q_full, 1);
@@ -58,9 +58,9 @@ __global__ void __launch_bounds__(kLpThreads)
             bar_init(v_full + i * 8, 1);
             bar_init(v_empty + i * 8, 1);
             bar_init(s_full + i * 8, 1);
+            bar_init(p_full + i * 8, 4);
             bar_init(o_done + i * 8, 1);
         }
-        bar_init(p_full, 4);
         bar_init(drained, 1);
         bar_init_fence();
     }
@@ -136,7 +136,7 @@ __global__ void __launch_bounds__(kLpThreads)
             for (uint32_t j = 0; j < n && ok; ++j) {
                 if (j + 1 < n && !(ok = scores(j + 1))) break;
                 const uint32_t s = j % v_stages;
-                if (!(ok = bar_wait(p_full, j & 1, &dead) && bar_wait(v_full + s * 8, (j / v_stages) & 1, &dead))) break;
+                if (!(ok = bar_wait(p_full + (j & 1) * 8, (j >> 1) & 1, &dead) && bar_wait(v_full + s * 8, (j / v_stages) & 1, &dead))) break;
                 fence_after();
                 const uint32_t p = tmem + (j & 1) * kLpK;  // the weights, where the scores were
                 const uint64_t dv = smem_desc(v_s + s * v_bytes, 128);
@@ -212,7 +212,9 @@ __global__ void __launch_bounds__(kLpThreads)
             tmem_st_wait();
             fence_before();
             __syncwarp();
-            if (lane == 0) bar_arrive(p_full);
+            // A warp may be one tile ahead of another (the next scores are already there), but not two: those
+            // are issued once all four have arrived here. Hence a barrier each for even and odd tiles.
+            if (lane == 0) bar_arrive(p_full + (j & 1) * 8);
         }
         // Most tiles skip the wait for the product before them, and a wait tells a phase from its neighbours
         // only. Hence one barrier for even and one for odd tiles: having seen the scores of tile j, the

@@ -119,6 +119,26 @@ def test_portions_of_a_tile_again_and_again(opened):
             assert np.array_equal(got, first)
 
 
+@pytest.mark.parametrize("heads,dim,rot_dim,vdim,window,size", [(16, 128, 64, 128, 4096, 1000), (8, 32, 32, 80, 90, 1000),
+                                                                (8, 32, 32, 80, 90, 70), (10, 64, 32, 48, 300, 500)])
+def test_many_prompts_give_the_same_bits(be, heads, dim, rot_dim, vdim, window, size):
+    spec = dict(rope_base=1e4, mixer=N.MIXER_LATENT_ATTENTION, heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, q_rank=256,
+                kv_rank=128, window=window, kv_from=-1, score_scale=3 * (dim + rot_dim) ** -0.5, mlp=N.MLP_RELU2, ff=512)
+    ex = ctox.B200Executor(be, ctox.StackConfig(vocab_size=1000, hidden_size=512, norm_eps=1e-6, logit_softcap=30.0,
+                                                layers=[N.LayerConfig(**spec) for _ in range(3)], max_context_tokens=3100))
+    ex.fill_synthetic(0)
+    ex.warmup()
+    tokens, first = tokens_of(3000, 1000, 1), None
+    for _ in range(40):
+        ex.reset_session()
+        for a in range(0, 3000, size):
+            ex.extend(tokens[a:a + size])
+        hidden = ex.last_hidden()
+        first = hidden if first is None else first
+        assert np.array_equal(hidden, first)
+    ex.unload()
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_passes_of_every_short_length(opened, dtype):
     config, t = MODELS["mixed"]()
