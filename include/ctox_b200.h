@@ -435,7 +435,7 @@ typedef struct {
     double rope_base;
     uint32_t mixer;  /* CTOX_MIXER_* */
     uint32_t heads, dim, rot_dim, vdim, q_rank, kv_rank;
-    uint32_t window; /* a token sees itself and window - 1 tokens before it; 0: all of them */
+    uint32_t window; /* keys at a distance below it are visible; 0: every earlier key */
     int32_t kv_from; /* -1: own cache */
     float score_scale;
     uint32_t mlp; /* CTOX_MLP_* */
