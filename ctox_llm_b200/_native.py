@@ -77,7 +77,8 @@ class ModelConfig(C.Structure):
             "max_draft_tokens", "draft_vocab")]
 
 
-KERNEL_CLASSES = ("stream_matvec", "attention", "dense_matvec", "latent_attention", "gemm", "latent_prefill", "norm", "other")
+KERNEL_CLASSES = ("stream_matvec", "attention", "dense_matvec", "stack_attention", "gemm", "stack_prefill", "norm",
+                  "query_key_value", "matrix_memory", "matrix_memory_prefill", "linear_attention")
 
 
 class KernelClass(C.Structure):
@@ -86,8 +87,10 @@ class KernelClass(C.Structure):
     _fields_ = [("ms", C.c_double), ("launches", C.c_uint64), ("bytes", C.c_double), ("flops", C.c_double)]
 
 
-MIXER_LATENT_ATTENTION = 1
-MLP_NONE, MLP_RELU2 = 0, 1
+MIXER_LATENT_ATTENTION, MIXER_GROUPED_ATTENTION, MIXER_MATRIX_MEMORY = 1, 2, 3
+MLP_NONE, MLP_RELU2, MLP_CLAMPED_GLU = 0, 1, 2
+NORM_LAYER, NORM_RMS = 0, 1
+ATTN_BIAS, ATTN_QK_NORM, ATTN_SINK, ATTN_V_MIX = 1, 2, 4, 8
 
 
 class LayerConfig(C.Structure):
@@ -95,7 +98,9 @@ class LayerConfig(C.Structure):
 
     _fields_ = [("rope_base", C.c_double)] + [(n, C.c_uint32) for n in (
         "mixer", "heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "window")] + [
-        ("kv_from", C.c_int32), ("score_scale", C.c_float), ("mlp", C.c_uint32), ("ff", C.c_uint32)]
+        ("kv_from", C.c_int32), ("score_scale", C.c_float), ("mlp", C.c_uint32), ("ff", C.c_uint32),
+        ("kv_heads", C.c_uint32), ("attn", C.c_uint32), ("gate_cap", C.c_float), ("mlp_limit", C.c_float),
+        ("mlp_slope", C.c_float)]
 
 
 class StackConfigC(C.Structure):
@@ -103,7 +108,8 @@ class StackConfigC(C.Structure):
 
     _fields_ = [("vocab_size", C.c_uint32), ("hidden_size", C.c_uint32), ("num_layers", C.c_uint32),
                 ("norm_eps", C.c_float), ("logit_softcap", C.c_float)] + [(n, C.c_uint32) for n in (
-                    "max_context_tokens", "kv_page_tokens", "kv_dtype", "pass_tokens")]
+                    "max_context_tokens", "kv_page_tokens", "kv_dtype", "pass_tokens", "norm", "out_norms",
+                    "tied_head")] + [("embed_scale", C.c_float)]
 
 
 class ExecStep(C.Structure):
@@ -123,7 +129,9 @@ class ExecStep(C.Structure):
 (T_EMBED, T_LM_HEAD, T_FINAL_NORM, T_INPUT_NORM, T_POST_NORM, T_ATTN_QKV, T_ATTN_O, T_Q_NORM, T_K_NORM,
  T_LIN_IN, T_LIN_OUT, T_CONV_W, T_A_LOG, T_DT_BIAS, T_LIN_NORM, T_MLP_GATE_UP, T_MLP_DOWN, T_MTP_FC,
  T_MTP_NORM_E, T_MTP_NORM_H, T_MTP_NORM, T_DRAFT_IDS, T_Q_DOWN, T_Q_DOWN_NORM, T_Q_UP, T_KV_DOWN, T_KV_DOWN_NORM,
- T_K_UP, T_V_UP, T_MIX_OUT_NORM, T_MLP_UP, T_MLP_OUT_NORM) = range(32)
+ T_K_UP, T_V_UP, T_MIX_OUT_NORM, T_MLP_UP, T_MLP_OUT_NORM, T_MIX_Q, T_MIX_K, T_MIX_V, T_MIX_Q_BIAS, T_MIX_K_BIAS,
+ T_MIX_V_BIAS, T_MIX_O_BIAS, T_ATTN_SINK, T_V_MIX, T_MIX_GATE, T_MIX_HEAD_NORM, T_MEM_IN, T_MEM_IN_BIAS, T_MEM_FORGET,
+ T_MEM_FORGET_BIAS, T_MLP_GATE) = range(48)
 LAYER_GLOBAL = 0xFFFFFFFF
 
 

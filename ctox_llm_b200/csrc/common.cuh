@@ -20,11 +20,15 @@ enum KernelClass : int {
     KC_STREAM_MATVEC = 0,   // packed weights
     KC_ATTENTION = 1,       // hybrid model's attention with its merge
     KC_DENSE_MATVEC = 2,    // bf16 weights, short passes
-    KC_LATENT_ATTENTION = 3,  // latent cache, short passes
+    KC_STACK_ATTENTION = 3, // layer stacks, short passes
     KC_GEMM = 4,            // tensor-core product, long passes
-    KC_LATENT_PREFILL = 5,  // tensor-core attention, long passes
+    KC_STACK_PREFILL = 5,   // tensor-core attention, long passes
     KC_NORM = 6,            // norms of long passes
-    KC_COUNT = 8
+    KC_QKV = 7,             // between the projection of queries, keys, values and attention
+    KC_MEMORY = 8,          // matrix memory, short passes
+    KC_MEMORY_PREFILL = 9,  // matrix memory, long passes
+    KC_LINEAR_ATTENTION = 10,  // hybrid model
+    KC_COUNT = CTOX_KERNEL_CLASSES
 };
 struct TimedLaunch {
     cudaEvent_t begin, end;

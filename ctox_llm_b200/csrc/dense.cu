@@ -215,7 +215,12 @@ __global__ void __launch_bounds__(kDvThreads, 2)
         const float n = (float)cols;
         float s = 0.f;
         if (in.norm == NORM_RMS) {
-            stream(x, nullptr, ldx, [&](uint32_t c, const float4 &v, const float4 &) {
+            stream(x, in.y ? in.y + (size_t)pm * in.y_stride : nullptr, ldx, [&](uint32_t c, const float4 &xv, const float4 &yv) {
+                float4 v = xv;
+                if (in.y) {
+                    v = make_float4(v.x + yv.x, v.y + yv.y, v.z + yv.z, v.w + yv.w);
+                    if (blockIdx.x == 0 && c < end) store4(in.x_out + (size_t)pm * in.x_stride, c, cols, v);
+                }
                 slot4(c) = v;
                 s += sq4(v);
             });
@@ -238,7 +243,10 @@ __global__ void __launch_bounds__(kDvThreads, 2)
             return q;
         };
         float mean = 0.f, inv = 0.f;
-        if (in.y) {
+        const bool post = in.y && in.wb;
+        if (in.y && !in.wb) {
+            stream(in.y + (size_t)pm * in.y_stride, nullptr, end, [&](uint32_t c, const float4 &v, const float4 &) { slot4(c) = v; });
+        } else if (in.y) {
             stream(in.y + (size_t)pm * in.y_stride, nullptr, end, [&](uint32_t c, const float4 &v, const float4 &) {
                 slot4(c) = v;
                 s += sum4(v);
@@ -247,14 +255,14 @@ __global__ void __launch_bounds__(kDvThreads, 2)
             inv = 1.0f / sqrtf(position_sum<M>(deviations(mean), red) / n + in.eps);
             s = 0.f;
         }
-        stream(x, in.y ? in.wb : nullptr, ldx, [&](uint32_t c, const float4 &xv, const float4 &wb) {
+        stream(x, post ? in.wb : nullptr, ldx, [&](uint32_t c, const float4 &xv, const float4 &wb) {
             float4 v = xv;
             if (in.y && c < end) {
                 const float4 y = slot4(c);
-                v.x += (y.x - mean) * inv * wb.x;
-                v.y += (y.y - mean) * inv * wb.y;  // the weight is zero past the last column
-                v.z += (y.z - mean) * inv * wb.z;
-                v.w += (y.w - mean) * inv * wb.w;
+                v.x += post ? (y.x - mean) * inv * wb.x : y.x;
+                v.y += post ? (y.y - mean) * inv * wb.y : y.y;  // the weight is zero past the last column
+                v.z += post ? (y.z - mean) * inv * wb.z : y.z;
+                v.w += post ? (y.w - mean) * inv * wb.w : y.w;
                 if (blockIdx.x == 0) store4(in.x_out + (size_t)pm * in.x_stride, c, cols, v);
             }
             slot4(c) = v;
@@ -272,7 +280,7 @@ __global__ void __launch_bounds__(kDvThreads, 2)
     if (in.w)
         each(cols, [&](uint32_t c) {
             prefetch_l1(in.w + c);
-            if (in.y) prefetch_l1(in.wb + c);
+            if (in.y && in.wb) prefetch_l1(in.wb + c);
         });
 
     uint32_t staged = 0xffffffffu;
@@ -358,6 +366,14 @@ __global__ void __launch_bounds__(kDvThreads, 2)
                     }
                 const uint32_t m = k / R, row = row0 + k % R;
                 if (m >= npos || row >= rows_per_group) continue;
+                if (out.bias) {
+                    v += out.bias[(size_t)group * rows_per_group + row];
+                    if ((row ^ 1u) < rows_per_group) pair += out.bias[(size_t)group * rows_per_group + (row ^ 1u)];
+                }
+                if (out.kind == OUT_CLAMPED_GLU) {
+                    if (!(row & 1)) out.y[(size_t)m * out.y_stride + (row >> 1)] = clamped_glu(v, pair, out.cap, out.slope);
+                    continue;
+                }
                 if (out.kind == OUT_RELU2) {
                     v = v > 0.f ? v * v : 0.f;
                 } else if (out.kind == OUT_SOFTCAP) {
@@ -508,7 +524,8 @@ __global__ void __launch_bounds__(kSnThreads) k_stream_norm(StreamNorm a) {
         return q;
     };
     float s = 0.f, mean = 0.f, inv = 0.f;
-    if (y) {
+    const bool post = y && a.wb, rms = a.norm == NORM_RMS;
+    if (post) {
         stream(y, nullptr, [&](uint32_t c, const float4 &v, const float4 &) {
             slot4(c) = v;
             s += (v.x + v.y) + (v.z + v.w);
@@ -517,9 +534,11 @@ __global__ void __launch_bounds__(kSnThreads) k_stream_norm(StreamNorm a) {
         inv = 1.0f / sqrtf(position_sum<1>(deviations(mean), red) / n + a.eps);
         s = 0.f;
     }
-    stream(x, y ? a.wb : nullptr, [&](uint32_t c, const float4 &xv, const float4 &wb) {
+    stream(x, post ? a.wb : y, [&](uint32_t c, const float4 &xv, const float4 &wb) {
         float4 v = xv;
-        if (y) {
+        if (y && !post) {
+            v = make_float4(v.x + wb.x, v.y + wb.y, v.z + wb.z, v.w + wb.w);
+        } else if (y) {
             const float4 u = slot4(c);
             v.x += (u.x - mean) * inv * wb.x;
             v.y += (u.y - mean) * inv * wb.y;  // the weight is zero past the last column
@@ -528,11 +547,12 @@ __global__ void __launch_bounds__(kSnThreads) k_stream_norm(StreamNorm a) {
         }
         if (a.x_out) store4(a.x_out + (size_t)row * W, c, W, v);
         slot4(c) = v;
-        s += (v.x + v.y) + (v.z + v.w);
+        s += rms ? (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w) : (v.x + v.y) + (v.z + v.w);
     });
     if (!a.w) return;
-    mean = position_sum<1>(s, red) / n;
-    inv = 1.0f / sqrtf(position_sum<1>(deviations(mean), red) / n + a.eps);
+    s = position_sum<1>(s, red) / n;
+    mean = rms ? 0.f : s;
+    inv = 1.0f / sqrtf((rms ? s : position_sum<1>(deviations(mean), red) / n) + a.eps);
     stream(a.w, nullptr, [&](uint32_t c, const float4 &w, const float4 &) {
         const float4 u = slot4(c);
         const float4 v = make_float4((u.x - mean) * inv * w.x, (u.y - mean) * inv * w.y, (u.z - mean) * inv * w.z,
@@ -587,16 +607,16 @@ ctox_status launch_latent_split(ctox_ctx *ctx, const float *fan, uint32_t fan_st
 // ------------------------------------------------------------------ embedding rows, weight layout
 __global__ void __launch_bounds__(256) k_embed_dense(const __nv_bfloat16 *__restrict__ embed, uint32_t ld,
                                                      const uint32_t *__restrict__ tokens, uint32_t width,
-                                                     float *__restrict__ x) {
+                                                     float scale, float *__restrict__ x) {
     pdl_launch();
     pdl_wait();
     const __nv_bfloat16 *row = embed + (size_t)tokens[blockIdx.x] * ld;
-    for (uint32_t c = threadIdx.x; c < width; c += 256) x[(size_t)blockIdx.x * width + c] = __bfloat162float(row[c]);
+    for (uint32_t c = threadIdx.x; c < width; c += 256) x[(size_t)blockIdx.x * width + c] = __bfloat162float(row[c]) * scale;
 }
 
 ctox_status launch_embed_dense(ctox_ctx *ctx, const __nv_bfloat16 *embed, uint32_t ld, const uint32_t *tokens,
-                               uint32_t width, uint32_t m, float *x) {
-    CTOX_CUDA(ctx, launch_pdl(k_embed_dense, dim3(m), dim3(256), 0, ctx->stream, embed, ld, tokens, width, x));
+                               uint32_t width, uint32_t m, float scale, float *x) {
+    CTOX_CUDA(ctx, launch_pdl(k_embed_dense, dim3(m), dim3(256), 0, ctx->stream, embed, ld, tokens, width, scale, x));
     return CTOX_OK;
 }
 
@@ -627,7 +647,8 @@ ctox_status launch_relayout(ctox_ctx *ctx, const __nv_bfloat16 *src, uint32_t ro
     return CTOX_OK;
 }
 
-__global__ void k_fill_normal_bf16(__nv_bfloat16 *__restrict__ out, uint64_t n, float std, uint64_t seed) {
+template <typename T>
+__global__ void k_fill_normal_dense(T *__restrict__ out, uint64_t n, float std, uint64_t seed) {
     const uint64_t i = (uint64_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n) return;
     uint64_t x = seed + (i + 1) * 0x9E3779B97F4A7C15ull;  // splitmix64
@@ -636,11 +657,16 @@ __global__ void k_fill_normal_bf16(__nv_bfloat16 *__restrict__ out, uint64_t n, 
     x ^= x >> 31;
     const float u1 = ((float)(x >> 40) + 0.5f) * (1.0f / 16777216.0f);
     const float u2 = (float)((x >> 16) & 0xffffff) * (1.0f / 16777216.0f);
-    out[i] = __float2bfloat16_rn(std * sqrtf(-2.0f * logf(u1)) * cosf(6.28318530718f * u2));
+    out[i] = (T)(std * sqrtf(-2.0f * logf(u1)) * cosf(6.28318530718f * u2));
 }
 
 ctox_status launch_fill_normal_bf16(ctox_ctx *ctx, __nv_bfloat16 *out, uint64_t n, float std, uint64_t seed) {
-    k_fill_normal_bf16<<<(unsigned)((n + 255) / 256), 256, 0, ctx->stream>>>(out, n, std, seed);
+    k_fill_normal_dense<<<(unsigned)((n + 255) / 256), 256, 0, ctx->stream>>>(out, n, std, seed);
+    CTOX_CUDA(ctx, cudaGetLastError());
+    return CTOX_OK;
+}
+ctox_status launch_fill_normal_f32(ctox_ctx *ctx, float *out, uint64_t n, float std, uint64_t seed) {
+    k_fill_normal_dense<<<(unsigned)((n + 255) / 256), 256, 0, ctx->stream>>>(out, n, std, seed);
     CTOX_CUDA(ctx, cudaGetLastError());
     return CTOX_OK;
 }

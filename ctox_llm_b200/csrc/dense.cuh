@@ -26,8 +26,8 @@ struct DenseMat {
 enum NormKind : int { NORM_NONE = 0, NORM_LAYER = 1, NORM_RMS = 2 };
 
 // Input vector of a matrix-vector product, [position][x_stride] (a grouped product adds
-// group * x_group). With a norm, `cols` values are normalised and weighted by w. With y set (layer
-// norm only) the input is first x + layer_norm(y; wb), which the first CTA stores to x_out. With
+// group * x_group). With a norm, `cols` values are normalised and weighted by w. With y set the input is
+// first x + y (layer norm with wb set: x + layer_norm(y; wb)), which the first CTA stores to x_out. With
 // ws_o set the input is the merge of `splits` partial attention results of row position * groups +
 // group instead.
 struct VecIn {
@@ -44,15 +44,17 @@ struct VecIn {
     uint32_t splits, ws_rows, groups;
 };
 
-enum OutKind : int { OUT_PLAIN = 0, OUT_RELU2 = 1, OUT_SOFTCAP = 2, OUT_ROPE = 3 };
+enum OutKind : int { OUT_PLAIN = 0, OUT_RELU2 = 1, OUT_SOFTCAP = 2, OUT_ROPE = 3, OUT_CLAMPED_GLU = 4 };
 
-// Output vector [position][y_stride]. OUT_ROPE: rows come in heads of head_width, of which the rows
-// rope0 .. rope0 + rope_dims are turned in interleaved pairs by (pos0 + position) * freq[pair].
+// Output vector [position][y_stride], the row's bias (may be null) added first. OUT_ROPE: rows come in heads
+// of head_width, of which the rows rope0 .. rope0 + rope_dims are turned in interleaved pairs by (pos0 +
+// position) * freq[pair]. OUT_CLAMPED_GLU: rows 2i and 2i + 1 are gate and up of output i (cap: the limit).
 struct VecOut {
     float *y;
     uint32_t y_stride;
     int kind;
-    float cap;
+    const float *bias;
+    float cap, slope;
     uint32_t head_width, rope0, rope_dims, pos0;
     const float *freq;
 };
@@ -76,9 +78,10 @@ struct LatentAppend {
 ctox_status launch_dense_matvec(ctox_ctx *ctx, const DenseMat &w, uint32_t groups, uint32_t m, const VecIn &in,
                                 const VecOut &out, const LatentAppend *append);
 
-// x <- x + layer_norm(y; wb) (y may be null; x_out may equal x), then layer_norm(.; w) of the result
-// as fp32 and / or bf16. One CTA per row; `rows` (device, may be null) picks input rows.
+// x <- x + layer_norm(y; wb), or x + y without wb (y may be null; x_out may equal x), then the norm (w) of
+// the result as fp32 and / or bf16. One CTA per row; `rows` (device, may be null) picks input rows.
 struct StreamNorm {
+    int norm;  // NORM_LAYER or NORM_RMS
     const float *x;
     const float *y, *wb, *w;
     float eps;
@@ -97,7 +100,7 @@ ctox_status launch_latent_split(ctox_ctx *ctx, const float *fan, uint32_t fan_st
                                 const LatentAppend *append, uint32_t m);
 
 ctox_status launch_embed_dense(ctox_ctx *ctx, const __nv_bfloat16 *embed, uint32_t ld, const uint32_t *tokens,
-                               uint32_t width, uint32_t m, float *x);
+                               uint32_t width, uint32_t m, float scale, float *x);
 
 // Index map of one axis when a matrix is laid out anew: groups of `group` indices become groups of
 // group_pad, the indices of a group from `split` on start at split_pad.
@@ -111,6 +114,7 @@ ctox_status launch_relayout(ctox_ctx *ctx, const __nv_bfloat16 *src, uint32_t ro
                             uint32_t transpose_cols);
 
 ctox_status launch_fill_normal_bf16(ctox_ctx *ctx, __nv_bfloat16 *out, uint64_t n, float std, uint64_t seed);
+ctox_status launch_fill_normal_f32(ctox_ctx *ctx, float *out, uint64_t n, float std, uint64_t seed);
 
 }  // namespace ctox
 
@@ -122,6 +126,11 @@ __device__ __forceinline__ void rope_pair(float &u, float &v, float angle) {
     const float a = u * c - v * s, b = v * c + u * s;
     u = a;
     v = b;
+}
+// Gated feed-forward with clamped inputs: g = min(gate, limit), u = clamp(up, +-limit); g sigmoid(slope g) (u + 1).
+__device__ __forceinline__ float clamped_glu(float gate, float up, float limit, float slope) {
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+    return g / (1.0f + expf(-slope * g)) * (u + 1.0f);
 }
 // Cache slot of position t.
 __device__ __forceinline__ size_t paged_slot(const uint32_t *page_table, uint32_t page_tokens, uint32_t t) {

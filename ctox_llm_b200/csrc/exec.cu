@@ -286,23 +286,22 @@ ctox_status ctox_exec_load_vector(ctox_exec *e, uint32_t layer, uint32_t tensor,
         e->warmed = false;
         return CTOX_OK;
     }
-    float **slot = nullptr;
-    uint64_t expect = 0, *loaded = nullptr;
-    if (e->stack ? !stack_vector_slot(e, layer, tensor, &slot, &expect, &loaded)
-                 : !vector_slot(e, layer, tensor, &slot, &expect))
+    VectorSlot slot;
+    if (e->stack ? !stack_vector_slot(e, layer, tensor, &slot) : !vector_slot(e, layer, tensor, &slot.base, &slot.n))
         return fail(ctx, CTOX_INVALID_ARTIFACT, "tensor %u is not a vector of layer %u", tensor, layer);
-    if (n != expect)
+    if (!slot.total) slot.total = slot.n;
+    if (n != slot.n)
         return fail(ctx, CTOX_SHAPE, "tensor %u of layer %u has %llu values, expected %llu", tensor, layer,
-                    (unsigned long long)n, (unsigned long long)expect);
+                    (unsigned long long)n, (unsigned long long)slot.n);
     for (uint64_t i = 0; i < n; ++i)
         if (!std::isfinite(values[i])) return fail(ctx, CTOX_INVALID_ARTIFACT, "tensor %u has a non-finite value", tensor);
-    if (!*slot) {
-        ctox_status rc = xalloc(e, (void **)slot, n * sizeof(float), false);
+    if (!*slot.base) {
+        ctox_status rc = xalloc(e, (void **)slot.base, slot.total * sizeof(float), false);
         if (rc) return rc;
     }
-    CTOX_CUDA(ctx, cudaMemcpyAsync(*slot, values, n * sizeof(float), cudaMemcpyHostToDevice, ctx->stream));
+    CTOX_CUDA(ctx, cudaMemcpyAsync(*slot.base + slot.offset, values, n * sizeof(float), cudaMemcpyHostToDevice, ctx->stream));
     CTOX_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
-    if (loaded) *loaded |= 1ull << tensor;
+    if (slot.loaded) *slot.loaded |= 1ull << tensor;
     e->warmed = false;
     return CTOX_OK;
 }
@@ -769,6 +768,7 @@ ctox_status ctox_exec_reset_session(ctox_exec *e) {
     ctox_ctx *ctx = e->ctx;
     if (!e->h && !(e->stack && e->warmed)) return fail(ctx, CTOX_INVALID_STATE, "reset: executor is not warm");
     const ctox_model_config &c = e->cfg;
+    if (e->stack) EX(stack_reset(e));
     for (uint32_t l = 0; l < e->w.size(); ++l) {
         LayerS &ls = e->s[l];
         if (e->w[l].full) continue;  // cache slots are rewritten before they are read
@@ -935,7 +935,10 @@ ctox_status layer_body(ctox_exec *e, uint32_t l, float *h, uint32_t m, uint64_t 
                           c.linear_conv_kernel_dim, ls.conv_state, lw.conv_w, lw.a_log, lw.dt_bias, lw.lin_norm,
                           c.rms_norm_epsilon, ls.delta[ls.cur], ls.delta[ls.cur ^ 1], ls.conv_in, ls.q, ls.k, ls.v,
                           ls.g, ls.beta, out_in};
+        timing_begin(ctx);
         launch_linear_attention(st, la, m);
+        timing_end(ctx, KC_LINEAR_ATTENTION, 2.0 * 4.0 * 128 * 128 * c.linear_num_value_heads,
+                   8.0 * 128 * 128 * c.linear_num_value_heads * m);
     } else {
         const AttnGeom g = attn_geom(e);
         launch_attn_pre(st, fan, g, lw.q_norm, lw.k_norm, rope_pos0, slot0, m, e->aq, e->agate, ls.k_cache,
@@ -981,7 +984,7 @@ ctox_status target_pass(ctox_exec *e, uint32_t m, uint64_t pos0) {
 ctox_status commit_positions(ctox_exec *e, uint32_t m, uint32_t n) {
     ctox_ctx *ctx = e->ctx;
     const ctox_model_config &c = e->cfg;
-    if (e->stack) {  // the cache only advances; the pass left the last position's hidden state in place
+    if (e->stack) {  // the pass appended to the caches, moved the states on and left the last position's hidden state in place
         e->hist_n = 1;
         e->have_hidden = true;
         e->position += n;

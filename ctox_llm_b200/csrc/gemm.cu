@@ -49,6 +49,28 @@ __device__ __forceinline__ int operand_row(const GemmPages &p, uint32_t row) {
 
 // 32 columns n0 .. n0 + 32 of one output row.
 __device__ __forceinline__ void gemm_store(const GemmOut &o, float *v, uint32_t m, uint32_t n0, uint32_t N) {
+    if (o.bias) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j)
+            if (n0 + j < N) v[j] += __ldg(o.bias + n0 + j);
+    }
+    if (o.kind == OUT_CLAMPED_GLU) {
+        __nv_bfloat16 *d = (__nv_bfloat16 *)o.d + (size_t)m * o.ld + n0 / 2;
+        __nv_bfloat162 h[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+            h[j] = __floats2bfloat162_rn(clamped_glu(v[4 * j], v[4 * j + 1], o.cap, o.slope),
+                                         clamped_glu(v[4 * j + 2], v[4 * j + 3], o.cap, o.slope));
+        if (n0 + 32 <= N && o.ld % 8 == 0) {
+            *reinterpret_cast<uint4 *>(d) = *reinterpret_cast<uint4 *>(h);
+            *reinterpret_cast<uint4 *>(d + 8) = *reinterpret_cast<uint4 *>(h + 4);
+        } else {
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+                if (n0 + 2 * j < N) d[j] = j & 1 ? h[j / 2].y : h[j / 2].x;
+        }
+        return;
+    }
     if (o.kind == OUT_RELU2) {
 #pragma unroll
         for (int j = 0; j < 32; ++j) v[j] = v[j] > 0.f ? v[j] * v[j] : 0.f;
@@ -70,7 +92,12 @@ __device__ __forceinline__ void gemm_store(const GemmOut &o, float *v, uint32_t 
         }
     }
     const bool full = n0 + 32 <= N;
-    if (o.bf16) {
+    if (o.split && n0 >= o.split) {
+        float *d = o.d2 + (size_t)m * o.ld2 + (n0 - o.split);
+#pragma unroll
+        for (int j = 0; j < 32; ++j)
+            if (n0 + j < N) d[j] = v[j];
+    } else if (o.bf16) {
         __nv_bfloat16 *d = (__nv_bfloat16 *)o.d + (size_t)m * o.ld + n0;
         if (full && o.ld % 8 == 0) {
 #pragma unroll
@@ -105,7 +132,6 @@ __global__ void __launch_bounds__(kGmThreads, 1)
     using namespace umma;
     constexpr uint32_t kABytes = kGmM * kGmK * 2, kBBytes = BN * kGmK * 2, kBBox = BN < 128 ? BN : 128;
     constexpr uint32_t kCols = 2 * BN < 32 ? 32 : 2 * BN;
-    pdl_launch();
     extern __shared__ uint8_t raw[];
     __shared__ __align__(8) uint64_t bars[2 * kGmStageMax + 5];
     __shared__ uint32_t tmem_slot;
@@ -133,6 +159,7 @@ __global__ void __launch_bounds__(kGmThreads, 1)
     fence_before();
     __syncthreads();
     fence_after();
+    pdl_launch();  // a later kernel's allocation must not come before this one's (see umma.cuh)
     const uint32_t tmem = tmem_slot;
     const uint32_t tiles_m = (M + kGmM - 1) / kGmM, tiles_n = (N + BN - 1) / BN, tiles = tiles_m * tiles_n;
     const uint32_t ksteps = (K + kGmK - 1) / kGmK;

@@ -5,7 +5,7 @@
 
 namespace ctox {
 
-// Rows of `ld` bf16 values, `cols` of them live. With a page table, rows live in the latent cache: row
+// Rows of `ld` bf16 values, `cols` of them live. With a page table, rows live in a paged cache: row
 // r of the operand is the cache row of position row0 + r (row0 a multiple of the 128-row tile, pages a
 // multiple of 128 tokens).
 struct GemmOperand {
@@ -20,7 +20,12 @@ struct GemmOut {
     uint32_t ld;
     int bf16;
     int kind;  // OutKind
-    float cap;
+    const float *bias;  // per column, may be null
+    float cap, slope;   // OUT_CLAMPED_GLU: columns 2i and 2i + 1 are gate and up of output column i
+    // columns from `split` (a multiple of 32; 0: none) on go to d2 as fp32, counted from there
+    uint32_t split;
+    float *d2;
+    uint32_t ld2;
     // OUT_ROPE: columns come in heads of head_width; columns rope0 .. rope0 + rope_dims of a head are turned in
     // pairs by table[row][pair] = (cos, sin)
     uint32_t head_width, rope0, rope_dims;

@@ -14,19 +14,29 @@ struct StackLayer {
     ctox_layer_config c{};
     uint32_t owner = 0;  // the layer whose cache this one reads (itself, or its kv_from)
     uint32_t dim_pad = 0, rot_pad = 0, vdim_pad = 0, kv_pad = 0, head_w = 0;  // head sizes rounded up to 16
-    DenseMat fan;        // [query down | key/value down] x hidden
+    // What the mixer projects from the stream, x hidden. Latent attention: [query down | key/value down]; grouped
+    // attention: [q | k | v]; matrix memory: [q | k | v | output gate] with padded heads, then from gate_row on the
+    // gates' rows [input | forget].
+    DenseMat fan;
+    uint32_t gate_row = 0;
     DenseMat q_up;       // heads x [dim_pad | rot_pad] rows
     DenseMat k_up;       // heads x dim_pad rows, columns kv_pad (long passes)
     DenseMat k_up_t;     // heads x kv_pad rows, columns dim_pad (short passes)
     DenseMat v_up;       // heads x vdim_pad rows, columns kv_pad
     DenseMat o;          // columns heads x vdim_pad
-    DenseMat up, down;
+    DenseMat up, down;   // up of a gated feed-forward: rows 2i and 2i + 1 are gate and up of unit i
     float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr, *q_norm = nullptr,
           *kv_norm = nullptr;
+    float *k_norm = nullptr, *fan_bias = nullptr, *o_bias = nullptr, *sink = nullptr, *v_mix = nullptr;  // grouped attention
+    float *in_bias = nullptr, *forget_bias = nullptr, *head_norm = nullptr;  // matrix memory
+    bool mixes_values = false;  // v_mix is applied: not in the first layer that has it
+    float *state = nullptr, *top = nullptr;  // matrix memory of the session (parts of StackModel::memory)
     float *freq = nullptr;     // [rot_dim / 2]
     float2 *table = nullptr;   // [position of the pass][rot_dim / 2] (cos, sin), shared by layers that rotate alike
     uint64_t loaded = 0;    // bit per tensor id
-    // cache of an owner: ring of pages through the page table, rows [kv_pad | rot_pad]
+    // cache of an owner: ring of pages through the page table. Rows of slot_cols values: latent attention [kv_pad |
+    // rot_pad], grouped attention kv_heads x [dim_pad | vdim_pad]
+    uint32_t slot_cols = 0;
     void *cache = nullptr;
     uint32_t *page_table = nullptr;
     uint32_t slots = 0;
@@ -49,8 +59,15 @@ struct StackModel {
     float *head_in = nullptr;
     uint32_t *rows_dev = nullptr;
     uint32_t head_rows = 0;  // rows of e->logits
-    // the stream at the end of the last pass: x[cur] + layer_norm(y; y_norm) when y_norm is set
+    float *v_first = nullptr;     // values of the first layer that mixes them, of the pass
+    uint32_t *arrived = nullptr;  // counters of the split merge
+    float *memory = nullptr;      // states of all matrix memories, cleared with the session
+    uint64_t memory_floats = 0;
+    __nv_bfloat16 *fan_b = nullptr, *mem_start = nullptr;
+    float *gates = nullptr, *mem_scan = nullptr, *mem_delta = nullptr, *mem_raw = nullptr;
+    // the stream at the end of the last pass: x[cur], plus y when it is pending (its norm y_norm applied, if any)
     int cur = 0;
+    bool pending = false;
     const float *y_norm = nullptr;
     float *streams = nullptr;  // [layer][max_context_tokens][hidden] when kept (evidence)
 };
@@ -58,7 +75,15 @@ struct StackModel {
 ctox_status stack_create(ctox_ctx *ctx, const ctox_stack_config *c, const ctox_layer_config *layers, ctox_exec **out);
 void stack_destroy(ctox_exec *e);
 ctox_status stack_load_matrix(ctox_exec *e, uint32_t layer, uint32_t tensor, const ctox_fused_matvec_op *op);
-bool stack_vector_slot(ctox_exec *e, uint32_t layer, uint32_t tensor, float ***slot, uint64_t *n, uint64_t **loaded);
+// Where a vector goes: `n` values from `offset` on of an array of `total` (allocated with its first part).
+struct VectorSlot {
+    float **base = nullptr;
+    uint64_t n = 0, total = 0, offset = 0;
+    uint64_t *loaded = nullptr;
+};
+bool stack_vector_slot(ctox_exec *e, uint32_t layer, uint32_t tensor, VectorSlot *slot);
+// A new session: recurrent states start at zero.
+ctox_status stack_reset(ctox_exec *e);
 ctox_status stack_fill_synthetic(ctox_exec *e, uint64_t seed);
 ctox_status stack_warmup(ctox_exec *e);
 ctox_status stack_prefill_synthetic(ctox_exec *e, uint64_t n, uint64_t seed);

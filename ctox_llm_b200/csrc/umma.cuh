@@ -15,8 +15,23 @@ namespace ctox {
 ctox_status tensor_map_bf16(ctox_ctx *ctx, CUtensorMap *map, const void *base, uint64_t rows, uint64_t cols, uint64_t ld,
                             uint32_t box_rows, uint32_t box_cols);
 
+// A segment of a head's dimensions (a multiple of 16), cut into boxes one swizzle atom wide.
+struct HeadBox {
+    uint32_t width, n;
+};
+__host__ __device__ inline HeadBox head_box(uint32_t dims) {
+    const uint32_t w = dims % 64 == 0 ? 64 : dims % 32 == 0 ? 32 : 16;
+    return HeadBox{w, dims / w};
+}
+
 #ifdef __CUDACC__
 namespace umma {
+
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 
 __device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void bar_init(uint32_t bar, uint32_t count) {
@@ -70,6 +85,9 @@ __device__ __forceinline__ void tma_load(uint32_t dst, const CUtensorMap *map, u
 __device__ __forceinline__ void tma_prefetch_map(const CUtensorMap *map) {
     asm volatile("prefetch.tensormap [%0];" ::"l"(map) : "memory");
 }
+// An allocation waits until the SM has the columns. A kernel that is launched early (pdl_launch) holds what it
+// allocates until the kernels before it have finished, so those must have allocated by then: a kernel calls
+// pdl_launch after its allocation, on every CTA.
 __device__ __forceinline__ void tmem_alloc(uint32_t smem_result, uint32_t cols) {  // one warp
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_result), "r"(cols) : "memory");
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
@@ -108,6 +126,17 @@ __device__ __forceinline__ uint64_t smem_desc(uint32_t addr, uint32_t row_bytes)
     const uint64_t swizzle = row_bytes == 128 ? 2 : row_bytes == 64 ? 4 : 6;
     return (uint64_t)((addr & 0x3ffff) >> 4) | (1ull << 16) | ((uint64_t)(row_bytes * 8 >> 4) << 32) | (1ull << 46) |
            (swizzle << 61);
+}
+// The same for an operand whose rows run along k (MN-major): rows of one swizzle atom of m or n values, all k
+// rows of an atom in a row, `atom_stride` bytes from one atom to the next. Sixteen values of k are 16 *
+// row_bytes apart. The instruction descriptor names such operands (a_mn, b_mn).
+__device__ __forceinline__ uint64_t smem_desc_mn(uint32_t addr, uint32_t row_bytes, uint32_t atom_stride) {
+    const uint64_t swizzle = row_bytes == 128 ? 2 : row_bytes == 64 ? 4 : 6;
+    return (uint64_t)((addr & 0x3ffff) >> 4) | ((uint64_t)(atom_stride >> 4) << 16) | ((uint64_t)(row_bytes * 8 >> 4) << 32) |
+           (1ull << 46) | (swizzle << 61);
+}
+__host__ __device__ constexpr uint32_t idesc_bf16_mn(uint32_t m, uint32_t n, bool a_mn, bool b_mn) {
+    return idesc_bf16(m, n) | ((uint32_t)a_mn << 15) | ((uint32_t)b_mn << 16);
 }
 // 32 lanes x 32 columns of tensor memory, one register per column.
 __device__ __forceinline__ void tmem_ld32(uint32_t tmem, float *v) {

@@ -67,11 +67,16 @@ class StackConfig:
     kv_page_tokens: int = 128
     kv_dtype: int = N.BF16
     pass_tokens: int = 0
+    norm: int = N.NORM_LAYER
+    out_norms: bool = True
+    tied_head: bool = False
+    embed_scale: float = 1.0
     mtp_num_hidden_layers: int = 0  # such a model has no MTP layer
 
     def create(self, backend: B200Backend, handle) -> int:
         c = N.StackConfigC(self.vocab_size, self.hidden_size, len(self.layers), self.norm_eps, self.logit_softcap,
-                           self.max_context_tokens, self.kv_page_tokens, self.kv_dtype, self.pass_tokens)
+                           self.max_context_tokens, self.kv_page_tokens, self.kv_dtype, self.pass_tokens, self.norm,
+                           int(self.out_norms), int(self.tied_head), self.embed_scale)
         layers = (N.LayerConfig * len(self.layers))(*self.layers)
         return backend._lib.ctox_exec_create_stack(backend._ctx, C.byref(c), layers, C.byref(handle))
 

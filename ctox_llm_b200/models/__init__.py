@@ -54,4 +54,4 @@ def open_model(folder: str, backend: Optional[B200Backend] = None, dtype: str = 
     return executor
 
 
-from . import lomelorn, qwen38  # noqa: E402,F401  (they register themselves)
+from . import lomelorn, qwen38, vasanex  # noqa: E402,F401  (they register themselves)

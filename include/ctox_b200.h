@@ -160,9 +160,11 @@ ctox_status ctox_ctx_kernel_timing(ctox_ctx *ctx, int32_t enable);
 ctox_status ctox_ctx_kernel_timing_read(ctox_ctx *ctx, double *total_ms, uint64_t *launches);
 /* The same for every kernel family that is bracketed (the read above reports class 0 alone); both reads
  * clear. Classes: 0 packed streaming matvec, 1 attention of the hybrid model (with its merge), 2 dense
- * matvec, 3 latent attention of short passes, 4 tensor-core product, 5 latent attention of long passes,
- * 6 norms of long passes. bytes / flops: algorithmic work (0 where not counted). */
-#define CTOX_KERNEL_CLASSES 8
+ * matvec, 3 attention of layer stacks in short passes, 4 tensor-core product, 5 attention of layer stacks in
+ * long passes, 6 norms of long passes, 7 queries / keys / values between their projection and attention,
+ * 8 matrix memory in short passes, 9 matrix memory in long passes, 10 linear attention of the hybrid model.
+ * bytes / flops: algorithmic work (0 where not counted). */
+#define CTOX_KERNEL_CLASSES 11
 typedef struct {
     double ms;
     uint64_t launches;
@@ -415,22 +417,58 @@ enum {
     CTOX_T_V_UP = 28,          /* layer, matrix heads*vdim x kv_rank */
     CTOX_T_MIX_OUT_NORM = 29,  /* layer, vector hidden (after the mixer) */
     CTOX_T_MLP_UP = 30,        /* layer, matrix ff x hidden */
-    CTOX_T_MLP_OUT_NORM = 31   /* layer, vector hidden (after the feed-forward) */
+    CTOX_T_MLP_OUT_NORM = 31,  /* layer, vector hidden (after the feed-forward) */
+    CTOX_T_MIX_Q = 32,         /* layer, matrix heads*dim x hidden */
+    CTOX_T_MIX_K = 33,         /* layer, matrix kv_heads*dim x hidden (matrix memory: heads*dim) */
+    CTOX_T_MIX_V = 34,         /* layer, matrix kv_heads*vdim x hidden (matrix memory: heads*vdim) */
+    CTOX_T_MIX_Q_BIAS = 35,    /* layer, vector, rows of the projection; likewise K, V and O */
+    CTOX_T_MIX_K_BIAS = 36,
+    CTOX_T_MIX_V_BIAS = 37,
+    CTOX_T_MIX_O_BIAS = 38,
+    CTOX_T_ATTN_SINK = 39,     /* layer, vector heads */
+    CTOX_T_V_MIX = 40,         /* layer, vector 1 (may be left out in the first layer that mixes) */
+    CTOX_T_MIX_GATE = 41,      /* layer, matrix heads*vdim x hidden (output gate) */
+    CTOX_T_MIX_HEAD_NORM = 42, /* layer, vector heads*vdim */
+    CTOX_T_MEM_IN = 43,        /* layer, matrix heads x hidden (log input gate) */
+    CTOX_T_MEM_IN_BIAS = 44,   /* layer, vector heads */
+    CTOX_T_MEM_FORGET = 45,    /* layer, matrix heads x hidden (log forget gate) */
+    CTOX_T_MEM_FORGET_BIAS = 46, /* layer, vector heads */
+    CTOX_T_MLP_GATE = 47       /* layer, matrix ff x hidden */
 };
 #define CTOX_LAYER_GLOBAL 0xffffffffu
 /* layer index of the MTP decoder layer = num_hidden_layers */
 
 /* ---- models described layer by layer (no counterpart in the reference) ----
- * Every layer is x += norm(mixer(norm(x))), then, with a feed-forward, x += norm(ff(norm(x))); the
- * norms are layer norms with a weight. They run through the same executor calls as the hybrid model:
- * prefill, extend, decode, select_target, evidence. One GPU, no MTP layer. */
-enum { CTOX_MIXER_LATENT_ATTENTION = 1 };
-enum { CTOX_MLP_NONE = 0, CTOX_MLP_RELU2 = 1 /* down(relu(up x)^2) */ };
+ * Every layer is x += mixer(norm(x)), then, with a feed-forward, x += ff(norm(x)); with out_norms the
+ * result of each sublayer is normalised before it is added. The norms are layer or RMS norms with a
+ * weight. They run through the same executor calls as the hybrid model: prefill, extend, decode,
+ * select_target, evidence. One GPU, no MTP layer. */
+enum { CTOX_MIXER_LATENT_ATTENTION = 1, CTOX_MIXER_GROUPED_ATTENTION = 2, CTOX_MIXER_MATRIX_MEMORY = 3 };
+enum {
+    CTOX_MLP_NONE = 0,
+    CTOX_MLP_RELU2 = 1,      /* down(relu(up x)^2) */
+    CTOX_MLP_CLAMPED_GLU = 2 /* g = min(gate x, limit), u = clamp(up x, +-limit): down(g sigmoid(slope g) (u + 1)) */
+};
+enum { CTOX_NORM_LAYER = 0, CTOX_NORM_RMS = 1 };
+/* options of grouped attention */
+enum {
+    CTOX_ATTN_BIAS = 1,    /* the four projections have biases */
+    CTOX_ATTN_QK_NORM = 2, /* RMS norm over the whole query and the whole key projection, before the rotation */
+    CTOX_ATTN_SINK = 4,    /* every head's softmax has one more term exp(sink) in its denominator */
+    CTOX_ATTN_V_MIX = 8    /* values <- (1 - a) values + a (values of the first such layer, same token) */
+};
 
 /* Latent attention: queries through a q_rank latent with an RMS norm; keys and values of all heads are
  * made from one cached row per token, an RMS-normed latent of kv_rank values and a rotated key part of
  * rot_dim values (interleaved pairs, base rope_base). kv_from >= 0 reads the cache of that earlier layer
- * (same kv_rank, rot_dim and rope_base) instead of writing its own. */
+ * (same kv_rank, rot_dim and rope_base) instead of writing its own.
+ *
+ * Grouped attention: query head h reads key/value head h / (heads / kv_heads); the first rot_dim dimensions
+ * of a head are rotated, i paired with i + rot_dim / 2 (rot_dim 0: no rotation).
+ *
+ * Matrix memory: per head a dim x vdim state with exponential input and forget gates (logs capped by
+ * gate_cap), a normaliser and a running maximum; queries are scaled by dim^-1/2; the heads' outputs are
+ * RMS-normed one by one, weighted (MIX_HEAD_NORM) and gated by sigmoid(MIX_GATE x). */
 typedef struct {
     double rope_base;
     uint32_t mixer;  /* CTOX_MIXER_* */
@@ -440,6 +478,10 @@ typedef struct {
     float score_scale;
     uint32_t mlp; /* CTOX_MLP_* */
     uint32_t ff;
+    uint32_t kv_heads;
+    uint32_t attn; /* CTOX_ATTN_* */
+    float gate_cap;
+    float mlp_limit, mlp_slope;
 } ctox_layer_config;
 
 typedef struct {
@@ -451,6 +493,10 @@ typedef struct {
     uint32_t kv_dtype;    /* CTOX_BF16: 16-bit products; CTOX_F32: everything in 32-bit, passes of 8 tokens */
     uint32_t pass_tokens; /* most prompt tokens of one pass (0: a default); cached pages cover the widest
                              window and one pass */
+    uint32_t norm;        /* CTOX_NORM_* of the residual stream */
+    uint32_t out_norms;   /* sublayer outputs are normalised (MIX_OUT_NORM, MLP_OUT_NORM); layer norms only */
+    uint32_t tied_head;   /* logits come from the embedding table; no LM_HEAD tensor */
+    float embed_scale;    /* of the embedding rows (not of a tied head) */
 } ctox_stack_config;
 
 /* One speculative block (engine.rs:110-116 ResolvedGreedyMtpVerification). */

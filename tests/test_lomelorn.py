@@ -123,7 +123,7 @@ def test_unknown_parts_are_refused(change):
 
 
 def test_registry_knows_the_architectures(tmp_path):
-    assert models.architectures() == ["Lomelorn", "Qwen38"]
+    assert models.architectures() == ["Lomelorn", "Qwen38", "Vasanex"]
     (tmp_path / "config.json").write_text(json.dumps({"architecture": "Other"}))
     with pytest.raises(ctox.CtoxError) as e:
         models.read_config(str(tmp_path))
@@ -142,8 +142,8 @@ def test_struct_layouts_match_the_header(tmp_path):
         for f in s._fields_:
             src.append(f'printf("%zu\\n", offsetof({name}, {f[0]}));')
             want.append(getattr(s, f[0]).offset)
-    src.append(f'printf("%d\\n", (int)CTOX_T_MLP_OUT_NORM); return 0;}}')
-    want.append(N.T_MLP_OUT_NORM)
+    src.append(f'printf("%d\\n", (int)CTOX_T_MLP_GATE); return 0;}}')
+    want.append(N.T_MLP_GATE)
     c, exe = tmp_path / "l.c", tmp_path / "l"
     c.write_text("\n".join(src))
     subprocess.check_call(["gcc", "-I", os.path.join(ROOT, "include"), str(c), "-o", str(exe)])
@@ -185,4 +185,4 @@ def test_trace_replay_writes_wanted_rows_and_resets_between_requests(tmp_path, m
 
 def test_command_line_lists_the_models():
     out = subprocess.run([sys.executable, "-m", "ctox_llm_b200", "models"], cwd=ROOT, capture_output=True, text=True)
-    assert out.returncode == 0 and out.stdout.split() == ["Lomelorn", "Qwen38"]
+    assert out.returncode == 0 and out.stdout.split() == ["Lomelorn", "Qwen38", "Vasanex"]
