@@ -827,11 +827,24 @@ LATENT_SIZES = {
 }
 
 
-def run_latent(args):
-    """The layer-stack model (Lomelorn: latent attention, window 4096, bf16 weights) beside the closest
-    existing model, the hybrid with full attention in every layer, at the same width, depth, feed-forward
-    and vocabulary: decode at a context of 8192 tokens and prefill of one 4096-token prompt, through the
-    executor's own calls, random weights ("5k-wide": window and context 32768). Per kernel family: device time with an event pair around every
+# Vasanex: attention and matrix memory in turn, a feed-forward in every layer. heads, kv_heads (of 128), window |
+# matrix memory: heads of 256 x 512 | the hybrid model (full and linear attention in turn) | Lomelorn's mixer
+VASANEX_SIZES = {
+    "2k": dict(width=2048, layers=8, vocab=32768, ff=8192, heads=16, kv_heads=4, window=4096, memory_heads=4,
+               hybrid_heads=(8, 2), linear_heads=(16, 16), latent=LATENT_SIZES["2k"]),
+    "5k": dict(width=5120, layers=8, vocab=32768, ff=17408, heads=40, kv_heads=8, window=4096, memory_heads=10,
+               hybrid_heads=(24, 4), linear_heads=(16, 48), latent=LATENT_SIZES["5k"]),
+    "5k-wide": dict(width=5120, layers=4, vocab=32768, ff=17408, heads=40, kv_heads=8, window=32768, context=32768,
+                    memory_heads=10, hybrid_heads=(24, 4), linear_heads=(16, 48), latent=LATENT_SIZES["5k-wide"]),
+}
+
+
+def run_stack(args):
+    """A layer-stack model beside the closest existing ones at the same width, depth, feed-forward and vocabulary:
+    decode at a context of 8192 tokens and prefill of one 4096-token prompt, through the executor's own calls,
+    random weights (the "-wide" sizes: window and context 32768). `latent`: Lomelorn (latent attention, bf16 weights)
+    beside the hybrid model with full attention in every layer. `vasanex`: Vasanex beside the hybrid model with full
+    and linear attention in turn, and Lomelorn. Per kernel family: device time with an event pair around every
     launch (serialised), and the fraction of its roofline (the larger of bytes / measured copy bandwidth and
     flops / measured bf16 product)."""
     import torch
@@ -859,10 +872,22 @@ def run_latent(args):
                                 layers=[N.LayerConfig(**layer) for _ in range(z["layers"])],
                                 max_context_tokens=z.get("context", 8192) + 1024, pass_tokens=args.pass_tokens)
 
+    def vasanex(z):
+        mlp = dict(kv_from=-1, mlp=N.MLP_CLAMPED_GLU, ff=z["ff"], mlp_limit=7.0, mlp_slope=1.702)
+        grouped = dict(mlp, mixer=N.MIXER_GROUPED_ATTENTION, heads=z["heads"], kv_heads=z["kv_heads"], dim=128, vdim=128, rot_dim=64,
+                       rope_base=10000.0, window=z["window"], score_scale=128 ** -0.5, attn=15)
+        memory = dict(mlp, mixer=N.MIXER_MATRIX_MEMORY, heads=z["memory_heads"], dim=256, vdim=512, gate_cap=15.0)
+        return ctox.StackConfig(vocab_size=z["vocab"], hidden_size=z["width"], norm_eps=1e-6, logit_softcap=0.0,
+                                layers=[N.LayerConfig(**(memory if i % 2 else grouped)) for i in range(z["layers"])],
+                                max_context_tokens=z.get("context", 8192) + 1024, pass_tokens=args.pass_tokens,
+                                norm=N.NORM_RMS, out_norms=False, tied_head=True)
+
     def hybrid(z):
+        keys, values = z.get("linear_heads", (16, 48))
         return ctox.qwen38_27b_config(
             vocab_size=z["vocab"], hidden_size=z["width"], intermediate_size=z["ff"], num_hidden_layers=z["layers"],
-            num_attention_heads=z["hybrid_heads"][0], num_key_value_heads=z["hybrid_heads"][1], full_attention_interval=1,
+            num_attention_heads=z["hybrid_heads"][0], num_key_value_heads=z["hybrid_heads"][1],
+            full_attention_interval=2 if "linear_heads" in z else 1, linear_num_key_heads=keys, linear_num_value_heads=values,
             mtp_num_hidden_layers=0, draft_vocab=0, max_draft_tokens=0,
             max_context_tokens=z.get("context", 8192) + 1024)
 
@@ -923,18 +948,26 @@ def run_latent(args):
     sampler = ClockSampler(local)
     sampler.start()
     sweep = {}
+    sizes = (args.sizes or ("2k,5k,7k,5k-wide" if args.workload == "latent" else "2k,5k,5k-wide")).split(",")
     launches0 = be.kernel_launches()
     with torch.cuda.stream(stream):
-        for name in args.sizes.split(","):
-            z = LATENT_SIZES[name]
-            sweep[name] = {"shape": z, "lomelorn": measure(stack(z), z.get("context", 8192))}
+        for name in sizes:
+            z = (LATENT_SIZES if args.workload == "latent" else VASANEX_SIZES)[name]
+            context = z.get("context", 8192)
+            sweep[name] = {"shape": z}
+            if args.workload == "vasanex":
+                sweep[name]["vasanex"] = measure(vasanex(z), context)
+            if args.workload == "latent" or not args.quick:
+                sweep[name]["lomelorn"] = measure(stack(z.get("latent", z)), context)
             if not args.quick:
-                sweep[name]["hybrid"] = measure(hybrid(z), z.get("context", 8192))
-    last = sweep[args.sizes.split(",")[-1] if "5k" not in sweep else "5k"]["lomelorn"]
-    line = {"metric": "latent_decode_tokens_per_s", "value": last["decode"]["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
+                sweep[name]["hybrid"] = measure(hybrid(z), context)
+    last = sweep[sizes[-1] if "5k" not in sweep else "5k"]["lomelorn" if args.workload == "latent" else "vasanex"]
+    mixers = ("latent attention) beside the hybrid model with full attention" if args.workload == "latent" else
+              "grouped attention and matrix memory) beside the hybrid model with full and linear attention and the latent one")
+    line = {"metric": f"{args.workload}_decode_tokens_per_s", "value": last["decode"]["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
             "steps": args.steps, "warmup": max(args.warmup, 3), "ms_per_step": last["decode"]["ms"], "higher_is_better": True,
             "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-            "config": {"workload": "layer stack (latent attention) beside the hybrid model with full attention at equal width, "
+            "config": {"workload": f"layer stack ({mixers} at equal width, "
                                    f"depth, feed-forward and vocabulary; decode at context 8192 (5k-wide: 32768), prefill of {prompt_n} tokens",
                        "l2": "a pass streams more weights than twice the L2"},
             "e2e": {"value": last["decode"]["e2e_tokens_per_s"], "unit": "tokens/s", "h2d_bytes_per_step": 4,
@@ -952,7 +985,7 @@ def main():
     ap.add_argument("--warmup", type=int, default=None)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--workload", default="decode",
-                    choices=["decode", "q4_matvec", "q2_matvec", "matvec", "verify_layer", "gated_delta", "kv_pack", "latent"])
+                    choices=["decode", "q4_matvec", "q2_matvec", "matvec", "verify_layer", "gated_delta", "kv_pack", "latent", "vasanex"])
     ap.add_argument("--dtype", default="q4", choices=["q4", "q2"], help="matvec: code format")
     ap.add_argument("--rows", type=int, default=17408)
     ap.add_argument("--cols", type=int, default=5120)
@@ -961,8 +994,8 @@ def main():
     ap.add_argument("--replicas", type=int, default=0,
                     help="matvec: weight replicas to rotate (default: enough to exceed twice the L2; 1 = weights "
                          "stay in L2, a diagnostic that separates the instruction cost from the HBM stream)")
-    ap.add_argument("--sizes", default="2k,5k,7k,5k-wide", help="latent: sizes to run")
-    ap.add_argument("--pass-tokens", type=int, default=0, help="latent: prompt tokens per pass (0: the default)")
+    ap.add_argument("--sizes", default="", help="latent, vasanex: sizes to run (default: all)")
+    ap.add_argument("--pass-tokens", type=int, default=0, help="latent, vasanex: prompt tokens per pass (0: the default)")
     ap.add_argument("--context", type=int, default=32768)
     ap.add_argument("--drafts", type=int, default=3,
                     help="decode: chained MTP drafts per block (3 = 4 verify positions, BASELINE config 2; "
@@ -973,15 +1006,15 @@ def main():
                     help="decode: only the timed region and one kernel-timing block (for launch lists)")
     args = ap.parse_args()
     if args.steps is None:
-        args.steps = {"decode": 256, "verify_layer": 400, "gated_delta": 50, "kv_pack": 50, "latent": 64}.get(args.workload, 2000)
+        args.steps = {"decode": 256, "verify_layer": 400, "gated_delta": 50, "kv_pack": 50, "latent": 64, "vasanex": 64}.get(args.workload, 2000)
     if args.warmup is None:
-        args.warmup = {"decode": 4, "gated_delta": 5, "kv_pack": 5, "latent": 4}.get(args.workload, 50)
+        args.warmup = {"decode": 4, "gated_delta": 5, "kv_pack": 5, "latent": 4, "vasanex": 4}.get(args.workload, 50)
     if args.impl == "reference":
         run_reference(args)
     elif args.workload == "decode":
         run_decode(args)
-    elif args.workload == "latent":
-        run_latent(args)
+    elif args.workload in ("latent", "vasanex"):
+        run_stack(args)
     elif args.workload == "q4_matvec":
         run_b200(args)
     else:
