@@ -129,7 +129,7 @@ __global__ void __launch_bounds__(kMdThreads) k_memory_delta(const __grid_consta
     __shared__ __align__(8) uint64_t bars[2];
     __shared__ uint32_t tmem_slot;
     __shared__ volatile int dead;
-    __shared__ float w_s[kMemChunk];
+    __shared__ float w_s[kMemChunk], norm_s[kMdThreads / 32][256];
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const uint32_t v0 = blockIdx.x * kMdRows, chunk = blockIdx.y, head = blockIdx.z;
     const HeadBox bd = head_box(a.dim_pad);
@@ -166,6 +166,7 @@ __global__ void __launch_bounds__(kMdThreads) k_memory_delta(const __grid_consta
     const bool ok = bar_wait(loaded, 0, &dead);
     if (!ok) bar_drain(loaded, 0);
     // the weights into the values, in two parts (a 16-byte piece keeps its place, whatever the swizzle)
+#pragma unroll 4
     for (uint32_t u = tid; u < 2 * kBox / 16; u += kMdThreads) {
         const float w = w_s[u * 16 % kBox / 128];
         uint4 *hp = reinterpret_cast<uint4 *>(base_p + u * 16);
@@ -198,36 +199,49 @@ __global__ void __launch_bounds__(kMdThreads) k_memory_delta(const __grid_consta
         commit(done);
     }
     float *dst = delta + ((size_t)chunk * a.heads + head) * (a.vdim_pad + kMemRows) * a.dim_pad;
-    if (blockIdx.x == 0) {  // the normaliser: the weighted sum of the keys
+    if (blockIdx.x == 0) {  // the normaliser: the weighted sum of the keys; a warp takes every fourth token
         const uint32_t mask = bd.width / 8 - 1, shift = bd.width == 64 ? 0 : bd.width == 32 ? 1 : 2;
-        for (uint32_t d = tid; d < a.dim_pad; d += kMdThreads) {
-            const uint32_t c = d % bd.width;
+        for (uint32_t d = lane * 8; d < a.dim_pad; d += 256) {
             const uint8_t *box = base_p + k_off + d / bd.width * k_box;
-            float s = 0.f;
-            for (uint32_t t = 0; t < kMemChunk; ++t) {
-                const uint32_t piece = (c / 8) ^ ((t >> shift) & mask);
-                s = fmaf(w_s[t], __bfloat162float(*reinterpret_cast<const __nv_bfloat16 *>(box + t * bd.width * 2 + piece * 16 + c % 8 * 2)), s);
+            float n[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+            for (uint32_t t = warp; t < kMemChunk; t += kMdThreads / 32) {
+                const uint4 k = *reinterpret_cast<const uint4 *>(box + t * bd.width * 2 + ((d % bd.width / 8) ^ ((t >> shift) & mask)) * 16);
+                const uint32_t x[4] = {k.x, k.y, k.z, k.w};
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    n[2 * j] = fmaf(w_s[t], __uint_as_float(x[j] << 16), n[2 * j]);
+                    n[2 * j + 1] = fmaf(w_s[t], __uint_as_float(x[j] & 0xffff0000u), n[2 * j + 1]);
+                }
             }
-            dst[(size_t)a.vdim_pad * a.dim_pad + d] = s;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) norm_s[warp][d + j] = n[j];
         }
+        __syncthreads();
+        for (uint32_t d = tid; d < a.dim_pad; d += kMdThreads)
+            dst[(size_t)a.vdim_pad * a.dim_pad + d] = (norm_s[0][d] + norm_s[1][d]) + (norm_s[2][d] + norm_s[3][d]);
     }
-    __syncwarp();
-    if (__all_sync(0xffffffffu, bar_wait(done, 0, &dead))) {
-        fence_after();
-        const uint32_t v = v0 + warp * 32 + lane;
+    const bool finished = bar_wait(done, 0, &dead);
+    if (!finished) bar_drain(done, 0);
+    __syncthreads();  // the operands' buffers are free
+    fence_after();
+    {   // a thread's row of the product goes to its own padded line, and from there as one copy
+        const uint32_t v = v0 + tid, line = tid * (a.dim_pad * 4 + 16);
         for (uint32_t d = 0; d < a.dim_pad; d += 16) {
             float x[16];
             tmem_ld16(tmem + d + ((warp * 32) << 16), x);
             tmem_ld_wait();
-            if (v < a.vdim_pad) {
-                float4 *p = reinterpret_cast<float4 *>(dst + (size_t)v * a.dim_pad + d);
 #pragma unroll
-                for (int j = 0; j < 4; ++j) p[j] = make_float4(x[4 * j], x[4 * j + 1], x[4 * j + 2], x[4 * j + 3]);
-            }
+            for (int j = 0; j < 4; ++j)
+                *reinterpret_cast<float4 *>(base_p + line + d * 4 + j * 16) = make_float4(x[4 * j], x[4 * j + 1], x[4 * j + 2], x[4 * j + 3]);
         }
         fence_before();
-    } else if (tid == 0) {
-        bar_drain(done, 0);
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+        if (v < a.vdim_pad)
+            asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(dst + (size_t)v * a.dim_pad), "r"(base + line),
+                         "r"(a.dim_pad * 4)
+                         : "memory");
+        asm volatile("cp.async.bulk.commit_group;\n\tcp.async.bulk.wait_group 0;" ::: "memory");
     }
     __syncthreads();
     if (warp == 0) {
@@ -281,29 +295,41 @@ __global__ void __launch_bounds__(kMcThreads) k_memory_scan(MatrixMemory a, floa
 // ------------------------------------------------------------------ outputs
 constexpr int kMoThreads = 192;      // warp 0: TMA, warp 1: MMA, warps 2-5: a token per thread
 constexpr uint32_t kMoSlice = 64;    // value columns at once
+constexpr uint32_t kMoBatch = 4;     // rows whose loads are in flight together
 
 // Tensor memory: scores (then their weighted bf16 form), two buffers each of the state's share and of the
 // chunk's own, n . q.
 constexpr uint32_t kMoState = 128, kMoOwn = 256, kMoNorm = 384, kMoCols = 512;
 
+// One whole 32-byte sector.
+__device__ __forceinline__ void store8(float *p, const float *v) {
+    asm volatile("st.global.v8.f32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};" ::"l"(p), "f"(v[0]), "f"(v[1]), "f"(v[2]), "f"(v[3]), "f"(v[4]),
+                 "f"(v[5]), "f"(v[6]), "f"(v[7])
+                 : "memory");
+}
+
 __global__ void __launch_bounds__(kMoThreads) k_memory_output(const __grid_constant__ CUtensorMap map_qk,
                                                               const __grid_constant__ CUtensorMap map_v,
                                                               const __grid_constant__ CUtensorMap map_s,
                                                               const __grid_constant__ CUtensorMap map_n, MatrixMemory a, MemoryLong w,
-                                                              uint32_t m, uint32_t chunks, uint32_t stages, int32_t *error_word) {
+                                                              uint32_t m, uint32_t chunks, int32_t *error_word) {
     using namespace umma;
     extern __shared__ uint8_t raw[];
     __shared__ __align__(8) uint64_t bars[14];
     __shared__ uint32_t tmem_slot;
     __shared__ volatile int dead;
-    __shared__ float a_s[kMemChunk];
+    __shared__ float a_s[kMemChunk], r_s[kMemChunk];
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const uint32_t chunk = blockIdx.x % chunks, head = blockIdx.x / chunks;
     const HeadBox bd = head_box(a.dim_pad);
+    // Two stages of a slice: state [hi | lo] and values. The second one's state takes the place of the keys and its values
+    // that of the normaliser, once those have been used.
     const uint32_t qk_bytes = kMemChunk * a.dim_pad * 2, s_bytes = kMoSlice * a.dim_pad * 2, v_bytes = kMemChunk * kMoSlice * 2,
-                   n_bytes = kMemRows * a.dim_pad * 2, stage_bytes = 2 * s_bytes + v_bytes;
+                   n_bytes = kMemRows * a.dim_pad * 2;
+    static_assert(2 * kMoSlice == kMemChunk && 2 * kMemRows * 256 <= kMemChunk * kMoSlice, "what the second stage replaces");
     const uint32_t base = (smem_addr(raw) + 1023) & ~1023u;
-    const uint32_t q_s = base, k_s = q_s + qk_bytes, st_s = k_s + qk_bytes, n_s = st_s + stages * stage_bytes;
+    const uint32_t q_s = base, k_s = q_s + qk_bytes, v_s = k_s + 2 * qk_bytes, n_s = v_s + v_bytes;
+    auto state_of = [&](uint32_t s) { return s ? k_s : k_s + qk_bytes; };
     const uint32_t b0 = smem_addr(bars), qk_full = b0, n_full = b0 + 8, s_full = b0 + 16, p_full = b0 + 24, nq_full = b0 + 32,
                    st_full = b0 + 40, st_empty = b0 + 56, o_full = b0 + 72, o_empty = b0 + 88, drained = b0 + 104;
     if (tid == 0) {
@@ -342,20 +368,21 @@ __global__ void __launch_bounds__(kMoThreads) k_memory_output(const __grid_const
             uint32_t issued = 0;
             bool ok = true;
             for (uint32_t j = 0; j < slices; ++j) {
-                const uint32_t s = j % stages, round = j / stages, dst = st_s + s * stage_bytes, bar = st_full + s * 8;
-                if (round > 0 && !(ok = bar_wait(st_empty + s * 8, (round - 1) & 1, &dead))) break;
-                bar_expect(bar, stage_bytes);
+                const uint32_t s = j & 1, dst = state_of(s), bar = st_full + s * 8;
+                if (j == 1 && !(ok = bar_wait(nq_full, 0, &dead))) break;
+                if (j >= 2 && !(ok = bar_wait(st_empty + s * 8, ((j >> 1) - 1) & 1, &dead))) break;
+                bar_expect(bar, 2 * s_bytes + v_bytes);
                 for (uint32_t h = 0; h < 2; ++h)
                     for (uint32_t i = 0; i < bd.n; ++i)
                         tma_load(dst + h * s_bytes + i * kMoSlice * bd.width * 2, &map_s, bar, (int)(i * bd.width),
                                  (int)(row0 + j * kMoSlice + h * lo_rows));
-                tma_load(dst + 2 * s_bytes, &map_v, bar, (int)(2 * a.heads * a.dim_pad + head * a.vdim_pad + j * kMoSlice), tok);
+                tma_load(v_s + s * v_bytes, &map_v, bar, (int)(2 * a.heads * a.dim_pad + head * a.vdim_pad + j * kMoSlice), tok);
                 ++issued;
             }
             if (!ok) {  // leave no copy in flight behind
                 bar_drain(qk_full, 0);
                 bar_drain(n_full, 0);
-                for (uint32_t s = 0; s < stages && s < issued; ++s) bar_drain(st_full + s * 8, ((issued - 1 - s) / stages) & 1);
+                for (uint32_t s = 0; s < 2 && s < issued; ++s) bar_drain(st_full + s * 8, ((issued - 1 - s) >> 1) & 1);
             }
         }
     } else if (warp == 1) {
@@ -382,8 +409,8 @@ __global__ void __launch_bounds__(kMoThreads) k_memory_output(const __grid_const
             }
             const uint32_t idesc_v = idesc_bf16_mn(kMemChunk, kMoSlice, false, true);
             for (uint32_t j = 0; j < slices && ok; ++j) {
-                const uint32_t s = j % stages, src = st_s + s * stage_bytes, o = j & 1;
-                if (!(ok = bar_wait(st_full + s * 8, (j / stages) & 1, &dead))) break;
+                const uint32_t o = j & 1, src = state_of(o);  // the slice's stage, and its buffers in tensor memory
+                if (!(ok = bar_wait(st_full + o * 8, (j >> 1) & 1, &dead))) break;
                 if (j >= 2 && !(ok = bar_wait(o_empty + o * 8, ((j >> 1) - 1) & 1, &dead))) break;
                 fence_after();
                 over_dims(tmem + kMoState + o * kMoSlice, src, kMoSlice, kMoSlice, false);
@@ -392,11 +419,11 @@ __global__ void __launch_bounds__(kMoThreads) k_memory_output(const __grid_const
                     if (!(ok = bar_wait(p_full, 0, &dead))) break;
                     fence_after();
                 }
-                const uint64_t dv = smem_desc_mn(src + 2 * s_bytes, 128, v_bytes);
+                const uint64_t dv = smem_desc_mn(v_s + o * v_bytes, 128, v_bytes);
 #pragma unroll
                 for (uint32_t k = 0; k < kMemChunk / 16; ++k)
                     mma_f16_ts(tmem + kMoOwn + o * kMoSlice, tmem + k * 8, dv + k * (16 * 128 / 16), idesc_v, k > 0);
-                commit(st_empty + s * 8);
+                commit(st_empty + o * 8);
                 commit(o_full + o * 8);
             }
             if (!ok) {
@@ -466,31 +493,53 @@ __global__ void __launch_bounds__(kMoThreads) k_memory_output(const __grid_const
                 for (int i = 0; i < 32; i += 16)
                     if (v + i < a.vdim_pad && tok < m)
 #pragma unroll
-                        for (int k = 0; k < 16; k += 4) {
-                            sq += (x[i + k] * x[i + k] + x[i + k + 1] * x[i + k + 1]) + (x[i + k + 2] * x[i + k + 2] + x[i + k + 3] * x[i + k + 3]);
-                            *reinterpret_cast<float4 *>(raw_row + v + i + k) = make_float4(x[i + k], x[i + k + 1], x[i + k + 2], x[i + k + 3]);
+                        for (int k = 0; k < 16; k += 8) {
+#pragma unroll
+                            for (int e = 0; e < 8; e += 2) sq += x[i + k + e] * x[i + k + e] + x[i + k + e + 1] * x[i + k + e + 1];
+                            store8(raw_row + v + i + k, x + i + k);
                         }
             }
             fence_before();
             __syncwarp();
             if (lane == 0) bar_arrive(o_empty + o * 8);
         }
-        if (ok && tok < m) {
-            const float r = 1.0f / sqrtf(sq / (float)a.vdim + a.eps);
-            const __nv_bfloat16 *gate = w.fan + (size_t)tok * w.fan_ld + a.heads * (2 * a.dim_pad + a.vdim_pad) + head * a.vdim_pad;
-            __nv_bfloat16 *out = w.out + ((size_t)tok * a.heads + head) * a.vdim_pad;
-            for (uint32_t v = 0; v < a.vdim_pad; v += 8) {
-                const uint4 g = *reinterpret_cast<const uint4 *>(gate + v);
-                const __nv_bfloat16 *gp = reinterpret_cast<const __nv_bfloat16 *>(&g);
-                float x[8];
-                *reinterpret_cast<float4 *>(x) = *reinterpret_cast<const float4 *>(raw_row + v);
-                *reinterpret_cast<float4 *>(x + 4) = *reinterpret_cast<const float4 *>(raw_row + v + 4);
-                __nv_bfloat162 h[4];
+        if (ok) {  // norm and output gate: the warp goes through its rows, a lane holds eight values
+            r_s[row] = 1.0f / sqrtf(sq / (float)a.vdim + a.eps);
+            __syncwarp();
+            const uint32_t t0 = chunk * kMemChunk + quarter * 32, n = t0 < m ? min(32u, m - t0) : 0;
+            const size_t ld = (size_t)a.heads * a.vdim_pad;
+            for (uint32_t v = lane * 8; v < a.vdim_pad; v += 256) {
+                float nw[8];
 #pragma unroll
-                for (int i = 0; i < 8; ++i) x[i] = v + i < a.vdim ? x[i] * r * a.norm_w[head * a.vdim + v + i] * sigmoid(__bfloat162float(gp[i])) : 0.f;
+                for (int i = 0; i < 8; ++i) nw[i] = v + i < a.vdim ? a.norm_w[head * a.vdim + v + i] : 0.f;
+                const float *rp = w.raw + t0 * ld + head * a.vdim_pad + v;
+                const __nv_bfloat16 *gp = w.fan + (size_t)t0 * w.fan_ld + a.heads * (2 * a.dim_pad + a.vdim_pad) + head * a.vdim_pad + v;
+                __nv_bfloat16 *op = w.out + t0 * ld + head * a.vdim_pad + v;
+                for (uint32_t k0 = 0; k0 < n; k0 += kMoBatch) {
+                    float x[kMoBatch][8];
+                    uint4 g[kMoBatch];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(x[2 * i], x[2 * i + 1]);
-                *reinterpret_cast<uint4 *>(out + v) = *reinterpret_cast<const uint4 *>(h);
+                    for (uint32_t k = 0; k < kMoBatch; ++k)
+                        if (k0 + k < n) {
+                            *reinterpret_cast<float4 *>(x[k]) = *reinterpret_cast<const float4 *>(rp + (k0 + k) * ld);
+                            *reinterpret_cast<float4 *>(x[k] + 4) = *reinterpret_cast<const float4 *>(rp + (k0 + k) * ld + 4);
+                            g[k] = *reinterpret_cast<const uint4 *>(gp + (size_t)(k0 + k) * w.fan_ld);
+                        }
+#pragma unroll
+                    for (uint32_t k = 0; k < kMoBatch; ++k)
+                        if (k0 + k < n) {
+                            const uint32_t gw[4] = {g[k].x, g[k].y, g[k].z, g[k].w};
+                            const float r = r_s[quarter * 32 + k0 + k];
+                            __nv_bfloat162 h[4];
+#pragma unroll
+                            for (int i = 0; i < 4; ++i) {
+                                const float g0 = __uint_as_float(gw[i] << 16), g1 = __uint_as_float(gw[i] & 0xffff0000u);
+                                h[i] = __floats2bfloat162_rn(__fdividef(x[k][2 * i] * r * nw[2 * i], 1.0f + __expf(-g0)),
+                                                             __fdividef(x[k][2 * i + 1] * r * nw[2 * i + 1], 1.0f + __expf(-g1)));
+                            }
+                            *reinterpret_cast<uint4 *>(op + (k0 + k) * ld) = *reinterpret_cast<const uint4 *>(h);
+                        }
+                }
             }
         }
     }
@@ -505,11 +554,10 @@ __global__ void __launch_bounds__(kMoThreads) k_memory_output(const __grid_const
 
 namespace {
 
-size_t output_smem(const MatrixMemory &a, uint32_t stages) {
-    return 1024 + 2 * (size_t)kMemChunk * a.dim_pad * 2 + stages * (2 * (size_t)kMoSlice * a.dim_pad * 2 + kMemChunk * kMoSlice * 2) +
-           2 * (size_t)kMemRows * a.dim_pad * 2;
+size_t output_smem(const MatrixMemory &a) { return 1024 + 3 * (size_t)kMemChunk * a.dim_pad * 2 + 2 * (size_t)kMemChunk * kMoSlice * 2; }
+size_t delta_smem(const MatrixMemory &a) {
+    return 1024 + std::max(4 * (size_t)kMemChunk * 128 + (size_t)kMemChunk * a.dim_pad * 2, (size_t)kMdRows * (a.dim_pad * 4 + 16));
 }
-size_t delta_smem(const MatrixMemory &a) { return 1024 + 4 * (size_t)kMemChunk * 128 + (size_t)kMemChunk * a.dim_pad * 2; }
 
 }  // namespace
 
@@ -520,7 +568,7 @@ MemoryLongSizes memory_long_sizes(const MatrixMemory &a, uint32_t pass_tokens) {
 }
 
 bool memory_long_fits(const ctox_ctx *ctx, const MatrixMemory &a) {
-    return a.dim_pad <= 256 && output_smem(a, 1) + 1024 <= (size_t)ctx->max_smem_optin;
+    return a.dim_pad <= 256 && std::max(output_smem(a), delta_smem(a) + 4096) + 2048 <= (size_t)ctx->max_smem_optin;
 }
 
 ctox_status launch_matrix_memory_long(ctox_ctx *ctx, const MatrixMemory &a, const MemoryLong &w, uint32_t m) {
@@ -533,9 +581,8 @@ ctox_status launch_matrix_memory_long(ctox_ctx *ctx, const MatrixMemory &a, cons
     EX(tensor_map_bf16(ctx, &v, w.fan, m, fan_cols, w.fan_ld, kMemChunk, 64));
     EX(tensor_map_bf16(ctx, &s, w.start, 2ull * chunks * a.heads * rows, a.dim_pad, a.dim_pad, kMoSlice, bd.width));
     EX(tensor_map_bf16(ctx, &n, w.start, 2ull * chunks * a.heads * rows, a.dim_pad, a.dim_pad, kMemRows, bd.width));
-    const uint32_t stages = output_smem(a, 2) + 1024 <= (size_t)ctx->max_smem_optin ? 2 : 1;
     CTOX_CUDA(ctx, cudaFuncSetAttribute(k_memory_delta, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)delta_smem(a)));
-    CTOX_CUDA(ctx, cudaFuncSetAttribute(k_memory_output, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)output_smem(a, stages)));
+    CTOX_CUDA(ctx, cudaFuncSetAttribute(k_memory_output, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)output_smem(a)));
     timing_begin(ctx);
     CTOX_CUDA(ctx, launch_pdl(k_memory_gates, dim3(a.heads), dim3(kMgThreads), 0, ctx->stream, a, w.gates, m, chunks, w.scan));
     CTOX_CUDA(ctx, launch_pdl(k_memory_delta, dim3((a.vdim_pad + kMdRows - 1) / kMdRows, chunks, a.heads), dim3(kMdThreads),
@@ -543,8 +590,8 @@ ctox_status launch_matrix_memory_long(ctox_ctx *ctx, const MatrixMemory &a, cons
     const uint32_t items = (a.vdim_pad + 1) * a.dim_pad / 4;
     CTOX_CUDA(ctx, launch_pdl(k_memory_scan, dim3((items + kMcThreads - 1) / kMcThreads, a.heads), dim3(kMcThreads), 0, ctx->stream, a,
                               w.scan, (const float *)w.delta, w.start, chunks));
-    CTOX_CUDA(ctx, launch_pdl(k_memory_output, dim3(chunks * a.heads), dim3(kMoThreads), output_smem(a, stages), ctx->stream, qk, v, s, n,
-                              a, w, m, chunks, stages, ctx->dev_error));
+    CTOX_CUDA(ctx, launch_pdl(k_memory_output, dim3(chunks * a.heads), dim3(kMoThreads), output_smem(a), ctx->stream, qk, v, s, n,
+                              a, w, m, chunks, ctx->dev_error));
     // algorithmic work: projections in, result out, the state once each way; per token the chunk's triangle and the state's share
     timing_end(ctx, KC_MEMORY_PREFILL, m * (fan_cols * 2.0 + a.heads * a.vdim_pad * 2.0) + 8.0 * a.heads * a.vdim * a.dim,
                2.0 * m * a.heads * ((a.dim + a.vdim) * (kMemChunk / 2.0) + 2.0 * a.dim * a.vdim));
