@@ -112,7 +112,7 @@ __global__ void __launch_bounds__(kMgThreads) k_memory_gates(MatrixMemory a, con
 }
 
 // ------------------------------------------------------------------ what a chunk adds
-constexpr int kMdThreads = 128;
+constexpr int kMdThreads = 256;
 constexpr uint32_t kMdRows = 128;  // value rows per CTA
 
 __host__ __device__ constexpr uint32_t tmem_width(uint32_t cols) {
@@ -161,7 +161,7 @@ __global__ void __launch_bounds__(kMdThreads) k_memory_delta(const __grid_consta
             tma_load(base + k_off + i * k_box, &map_k, loaded, (int)((a.heads + head) * a.dim_pad + i * bd.width), row);
     }
     const MemScan sc = mem_scan(scan, a.heads, chunks, head);
-    w_s[tid] = expf(sc.a[chunk * kMemChunk + tid] - sc.chunk[chunk * 2 + 1]);
+    if (tid < kMemChunk) w_s[tid] = expf(sc.a[chunk * kMemChunk + tid] - sc.chunk[chunk * 2 + 1]);
     __syncthreads();
     const bool ok = bar_wait(loaded, 0, &dead);
     if (!ok) bar_drain(loaded, 0);
@@ -199,7 +199,7 @@ __global__ void __launch_bounds__(kMdThreads) k_memory_delta(const __grid_consta
         commit(done);
     }
     float *dst = delta + ((size_t)chunk * a.heads + head) * (a.vdim_pad + kMemRows) * a.dim_pad;
-    if (blockIdx.x == 0) {  // the normaliser: the weighted sum of the keys; a warp takes every fourth token
+    if (blockIdx.x == 0) {  // the normaliser: the weighted sum of the keys; a warp takes every eighth token
         const uint32_t mask = bd.width / 8 - 1, shift = bd.width == 64 ? 0 : bd.width == 32 ? 1 : 2;
         for (uint32_t d = lane * 8; d < a.dim_pad; d += 256) {
             const uint8_t *box = base_p + k_off + d / bd.width * k_box;
@@ -219,17 +219,18 @@ __global__ void __launch_bounds__(kMdThreads) k_memory_delta(const __grid_consta
         }
         __syncthreads();
         for (uint32_t d = tid; d < a.dim_pad; d += kMdThreads)
-            dst[(size_t)a.vdim_pad * a.dim_pad + d] = (norm_s[0][d] + norm_s[1][d]) + (norm_s[2][d] + norm_s[3][d]);
+            dst[(size_t)a.vdim_pad * a.dim_pad + d] = ((norm_s[0][d] + norm_s[1][d]) + (norm_s[2][d] + norm_s[3][d])) +
+                                                      ((norm_s[4][d] + norm_s[5][d]) + (norm_s[6][d] + norm_s[7][d]));
     }
     const bool finished = bar_wait(done, 0, &dead);
     if (!finished) bar_drain(done, 0);
     __syncthreads();  // the operands' buffers are free
     fence_after();
-    {   // a thread's row of the product goes to its own padded line, and from there as one copy
-        const uint32_t v = v0 + tid, line = tid * (a.dim_pad * 4 + 16);
-        for (uint32_t d = 0; d < a.dim_pad; d += 16) {
+    {   // a row of the product goes to its own padded line (two warps share the columns), and from there as one copy
+        const uint32_t quarter = warp & 3, row_bytes = a.dim_pad * 4 + 16, line = (quarter * 32 + lane) * row_bytes;
+        for (uint32_t d = (warp >> 2) * 16; d < a.dim_pad; d += 32) {
             float x[16];
-            tmem_ld16(tmem + d + ((warp * 32) << 16), x);
+            tmem_ld16(tmem + d + ((quarter * 32) << 16), x);
             tmem_ld_wait();
 #pragma unroll
             for (int j = 0; j < 4; ++j)
@@ -237,11 +238,13 @@ __global__ void __launch_bounds__(kMdThreads) k_memory_delta(const __grid_consta
         }
         fence_before();
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-        if (v < a.vdim_pad)
-            asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(dst + (size_t)v * a.dim_pad), "r"(base + line),
-                         "r"(a.dim_pad * 4)
+        __syncthreads();
+        if (tid < kMdRows && v0 + tid < a.vdim_pad) {
+            asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(dst + (size_t)(v0 + tid) * a.dim_pad),
+                         "r"(base + tid * row_bytes), "r"(a.dim_pad * 4)
                          : "memory");
-        asm volatile("cp.async.bulk.commit_group;\n\tcp.async.bulk.wait_group 0;" ::: "memory");
+            asm volatile("cp.async.bulk.commit_group;\n\tcp.async.bulk.wait_group 0;" ::: "memory");
+        }
     }
     __syncthreads();
     if (warp == 0) {
@@ -293,13 +296,12 @@ __global__ void __launch_bounds__(kMcThreads) k_memory_scan(MatrixMemory a, floa
 }
 
 // ------------------------------------------------------------------ outputs
-constexpr int kMoThreads = 192;      // warp 0: TMA, warp 1: MMA, warps 2-5: a token per thread
+constexpr int kMoThreads = 320;      // warp 0: TMA, warp 1: MMA, warps 2-9: two threads per token, half of the columns each
 constexpr uint32_t kMoSlice = 64;    // value columns at once
 constexpr uint32_t kMoBatch = 4;     // rows whose loads are in flight together
 
-// Tensor memory: scores (then their weighted bf16 form), two buffers each of the state's share and of the
-// chunk's own, n . q.
-constexpr uint32_t kMoState = 128, kMoOwn = 256, kMoNorm = 384, kMoCols = 512;
+// Tensor memory: scores, two buffers each of the state's share and of the chunk's own, n . q, the weighted scores.
+constexpr uint32_t kMoState = 128, kMoOwn = 256, kMoNorm = 384, kMoWeights = 416, kMoCols = 512;
 
 // One whole 32-byte sector.
 __device__ __forceinline__ void store8(float *p, const float *v) {
@@ -318,7 +320,8 @@ __global__ void __launch_bounds__(kMoThreads) k_memory_output(const __grid_const
     __shared__ __align__(8) uint64_t bars[14];
     __shared__ uint32_t tmem_slot;
     __shared__ volatile int dead;
-    __shared__ float a_s[kMemChunk], r_s[kMemChunk];
+    __shared__ float red_s[3][kMemChunk];  // a, then sums of squares in the first two; n . q of the chunk's own in the last two
+    float *a_s = red_s[0];
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const uint32_t chunk = blockIdx.x % chunks, head = blockIdx.x / chunks;
     const HeadBox bd = head_box(a.dim_pad);
@@ -335,12 +338,12 @@ __global__ void __launch_bounds__(kMoThreads) k_memory_output(const __grid_const
     if (tid == 0) {
         dead = 0;
         for (uint32_t bar : {qk_full, n_full, s_full, nq_full, drained}) bar_init(bar, 1);
-        bar_init(p_full, 4);
+        bar_init(p_full, 8);
         for (uint32_t i = 0; i < 2; ++i) {
             bar_init(st_full + i * 8, 1);
             bar_init(st_empty + i * 8, 1);
             bar_init(o_full + i * 8, 1);
-            bar_init(o_empty + i * 8, 4);
+            bar_init(o_empty + i * 8, 8);
         }
         bar_init_fence();
     }
@@ -422,7 +425,7 @@ __global__ void __launch_bounds__(kMoThreads) k_memory_output(const __grid_const
                 const uint64_t dv = smem_desc_mn(v_s + o * v_bytes, 128, v_bytes);
 #pragma unroll
                 for (uint32_t k = 0; k < kMemChunk / 16; ++k)
-                    mma_f16_ts(tmem + kMoOwn + o * kMoSlice, tmem + k * 8, dv + k * (16 * 128 / 16), idesc_v, k > 0);
+                    mma_f16_ts(tmem + kMoOwn + o * kMoSlice, tmem + kMoWeights + k * 8, dv + k * (16 * 128 / 16), idesc_v, k > 0);
                 commit(st_empty + o * 8);
                 commit(o_full + o * 8);
             }
@@ -432,19 +435,20 @@ __global__ void __launch_bounds__(kMoThreads) k_memory_output(const __grid_const
             }
         }
     } else {
-        const uint32_t quarter = warp & 3, row = quarter * 32 + lane, lanes = (quarter * 32) << 16, tok = chunk * kMemChunk + row;
+        const uint32_t quarter = warp & 3, part = (warp - 2) >> 2, row = quarter * 32 + lane, lanes = (quarter * 32) << 16,
+                       tok = chunk * kMemChunk + row;
         const MemScan sc = mem_scan(w.scan, a.heads, chunks, head);
-        a_s[row] = sc.a[tok] * kLog2e;
+        if (part == 0) a_s[row] = sc.a[tok] * kLog2e;
         const float M = sc.M[tok], Ml = M * kLog2e, floor = sc.floor[tok];
         const float scale = 1.0f / sqrtf((float)a.dim), from_state = expf(sc.chunk[chunk * 2] - M) * scale;
-        asm volatile("bar.sync 1, 128;" ::: "memory");
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        // `ok` may differ between warps: the barriers below are passed by all of them
         bool ok = __all_sync(0xffffffffu, bar_wait(s_full, 0, &dead));
-        float nq = 0.f;
         if (ok) {
+            float nq = 0.f;
             fence_after();
-            // a block of 32 scores becomes 16 columns of weights, left of every score still to be read
 #pragma unroll 1
-            for (uint32_t b = 0; b < kMemChunk / 32; ++b) {
+            for (uint32_t b = part * 2; b < part * 2 + 2; ++b) {
                 float s[32];
                 tmem_ld32(tmem + b * 32 + lanes, s);
                 tmem_ld_wait();
@@ -458,55 +462,53 @@ __global__ void __launch_bounds__(kMoThreads) k_memory_output(const __grid_const
                     const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
                     p[j / 2] = *reinterpret_cast<const float *>(&h);
                 }
-                tmem_st16(tmem + b * 16 + lanes, p);
+                tmem_st16(tmem + kMoWeights + b * 16 + lanes, p);
             }
+            red_s[1 + part][row] = nq;
             tmem_st_wait();
             fence_before();
             __syncwarp();
             if (lane == 0) bar_arrive(p_full);
             ok = __all_sync(0xffffffffu, bar_wait(nq_full, 0, &dead));
         }
+        asm volatile("bar.sync 1, 256;" ::: "memory");
         float inv = 0.f, sq = 0.f;
         if (ok) {
             fence_after();
             float n[16];
             tmem_ld16(tmem + kMoNorm + lanes, n);
             tmem_ld_wait();
-            nq = fmaf(from_state, n[0], nq);
+            const float nq = fmaf(from_state, n[0], red_s[1][row] + red_s[2][row]);
             inv = 1.0f / (fmaxf(fabsf(nq), floor) + 1e-6f);
         }
+        asm volatile("bar.sync 1, 256;" ::: "memory");
         float *raw_row = w.raw + ((size_t)tok * a.heads + head) * a.vdim_pad;
         for (uint32_t j = 0; j < slices && ok; ++j) {
-            const uint32_t o = j & 1;
+            const uint32_t o = j & 1, c = part * 32, v = j * kMoSlice + c;  // vdim_pad is a multiple of 16
             if (!(ok = __all_sync(0xffffffffu, bar_wait(o_full + o * 8, (j >> 1) & 1, &dead)))) break;
             fence_after();
-#pragma unroll 1
-            for (uint32_t c = 0; c < kMoSlice; c += 32) {
-                float x[32], y[32];
-                tmem_ld32(tmem + kMoState + o * kMoSlice + c + lanes, x);
-                tmem_ld32(tmem + kMoOwn + o * kMoSlice + c + lanes, y);
-                tmem_ld_wait();
-#pragma unroll
-                for (int i = 0; i < 32; ++i) x[i] = fmaf(from_state, x[i], y[i]) * inv;
-                const uint32_t v = j * kMoSlice + c;  // vdim_pad is a multiple of 16
-#pragma unroll
-                for (int i = 0; i < 32; i += 16)
-                    if (v + i < a.vdim_pad && tok < m)
-#pragma unroll
-                        for (int k = 0; k < 16; k += 8) {
-#pragma unroll
-                            for (int e = 0; e < 8; e += 2) sq += x[i + k + e] * x[i + k + e] + x[i + k + e + 1] * x[i + k + e + 1];
-                            store8(raw_row + v + i + k, x + i + k);
-                        }
-            }
+            float x[32], y[32];
+            tmem_ld32(tmem + kMoState + o * kMoSlice + c + lanes, x);
+            tmem_ld32(tmem + kMoOwn + o * kMoSlice + c + lanes, y);
+            tmem_ld_wait();
             fence_before();
             __syncwarp();
             if (lane == 0) bar_arrive(o_empty + o * 8);
+#pragma unroll
+            for (int i = 0; i < 32; ++i) x[i] = fmaf(from_state, x[i], y[i]) * inv;
+#pragma unroll
+            for (int i = 0; i < 32; i += 8)
+                if (v + i < a.vdim_pad && tok < m) {
+#pragma unroll
+                    for (int e = 0; e < 8; e += 2) sq += x[i + e] * x[i + e] + x[i + e + 1] * x[i + e + 1];
+                    store8(raw_row + v + i, x + i);
+                }
         }
-        if (ok) {  // norm and output gate: the warp goes through its rows, a lane holds eight values
-            r_s[row] = 1.0f / sqrtf(sq / (float)a.vdim + a.eps);
-            __syncwarp();
-            const uint32_t t0 = chunk * kMemChunk + quarter * 32, n = t0 < m ? min(32u, m - t0) : 0;
+        red_s[part][row] = sq;
+        __threadfence_block();
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        if (ok) {  // norm and output gate: a warp goes through sixteen rows, a lane holds eight values
+            const uint32_t r0 = (warp - 2) * 16, t0 = chunk * kMemChunk + r0, n = t0 < m ? min(16u, m - t0) : 0;
             const size_t ld = (size_t)a.heads * a.vdim_pad;
             for (uint32_t v = lane * 8; v < a.vdim_pad; v += 256) {
                 float nw[8];
@@ -529,7 +531,7 @@ __global__ void __launch_bounds__(kMoThreads) k_memory_output(const __grid_const
                     for (uint32_t k = 0; k < kMoBatch; ++k)
                         if (k0 + k < n) {
                             const uint32_t gw[4] = {g[k].x, g[k].y, g[k].z, g[k].w};
-                            const float r = r_s[quarter * 32 + k0 + k];
+                            const float r = 1.0f / sqrtf((red_s[0][r0 + k0 + k] + red_s[1][r0 + k0 + k]) / (float)a.vdim + a.eps);
                             __nv_bfloat162 h[4];
 #pragma unroll
                             for (int i = 0; i < 4; ++i) {

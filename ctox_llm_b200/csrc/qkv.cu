@@ -6,7 +6,7 @@ namespace ctox {
 constexpr int kQkvThreads = 512;
 
 // One CTA per (position, share of the outputs). Every CTA of a position brings the projections into shared memory and
-// forms the norms over the whole query and key projection itself; a thread then makes groups of eight outputs.
+// forms the norms over the whole query and key projection itself; a thread then makes groups of four outputs.
 __global__ void __launch_bounds__(kQkvThreads) k_qkv_prep(QkvPrep a) {
     pdl_launch();
     extern __shared__ __align__(16) float sm[];
@@ -70,10 +70,23 @@ __global__ void __launch_bounds__(kQkvThreads) k_qkv_prep(QkvPrep a) {
         for (uint32_t c = tid; c < nk; c += kQkvThreads) x[nq + c] *= k_inv * a.k_norm[c];
     }
     __syncthreads();
-    // values d .. d + 8 of the head at h, rotated
+    // values d .. d + 4 of the head at h, rotated
+    const bool vec = a.dim % 4 == 0 && half % 4 == 0;  // then a group lies in one half, and so does its pair
     auto turned = [&](const float *h, uint32_t d, float *r) {
+        if (vec && d < a.dim) {
+            *reinterpret_cast<float4 *>(r) = *reinterpret_cast<const float4 *>(h + d);
+            if (d < a.rot_dim) {
+                const bool low = d < half;
+                const float4 p = *reinterpret_cast<const float4 *>(low ? h + d + half : h + d - half);
+                const float pv[4] = {p.x, p.y, p.z, p.w};
+                const float2 *cs = cs_s + (low ? d : d - half);
 #pragma unroll
-        for (uint32_t j = 0; j < 8; ++j) {
+                for (int j = 0; j < 4; ++j) r[j] = low ? r[j] * cs[j].x - pv[j] * cs[j].y : r[j] * cs[j].x + pv[j] * cs[j].y;
+            }
+            return;
+        }
+#pragma unroll
+        for (uint32_t j = 0; j < 4; ++j) {
             const uint32_t i = d + j;
             r[j] = i < a.dim ? h[i] : 0.f;
             if (i < half) {
@@ -87,32 +100,29 @@ __global__ void __launch_bounds__(kQkvThreads) k_qkv_prep(QkvPrep a) {
     };
     auto store = [&](__nv_bfloat16 *b16, float *f32, size_t at, const float *r) {
         if (b16) {
-            __nv_bfloat162 h[4];
-#pragma unroll
-            for (int j = 0; j < 4; ++j) h[j] = __floats2bfloat162_rn(r[2 * j], r[2 * j + 1]);
-            *reinterpret_cast<uint4 *>(b16 + at) = *reinterpret_cast<const uint4 *>(h);
+            const __nv_bfloat162 h[2] = {__floats2bfloat162_rn(r[0], r[1]), __floats2bfloat162_rn(r[2], r[3])};
+            *reinterpret_cast<uint2 *>(b16 + at) = *reinterpret_cast<const uint2 *>(h);
         } else {
             *reinterpret_cast<float4 *>(f32 + at) = make_float4(r[0], r[1], r[2], r[3]);
-            *reinterpret_cast<float4 *>(f32 + at + 4) = make_float4(r[4], r[5], r[6], r[7]);
         }
     };
-    const uint32_t q_groups = a.heads * a.dim_pad / 8, part = a.dim_pad + a.vdim_pad, slot_cols = a.kv_heads * part;
+    const uint32_t q_groups = a.heads * a.dim_pad / 4, part = a.dim_pad + a.vdim_pad, slot_cols = a.kv_heads * part;
     const size_t base = paged_slot(a.page_table, a.page_tokens, pos) * slot_cols;
     const float mix = a.v_mix ? *a.v_mix : 0.f;
-    for (uint32_t g = blockIdx.x * kQkvThreads + tid; g < q_groups + slot_cols / 8; g += gridDim.x * kQkvThreads) {
-        float r[8];
+    for (uint32_t g = blockIdx.x * kQkvThreads + tid; g < q_groups + slot_cols / 4; g += gridDim.x * kQkvThreads) {
+        __align__(16) float r[4];
         if (g < q_groups) {
-            const uint32_t c = g * 8;
+            const uint32_t c = g * 4;
             turned(x + c / a.dim_pad * a.dim, c % a.dim_pad, r);
             store(a.q_b16, a.q_f32, (size_t)m * a.heads * a.dim_pad + c, r);
             continue;
         }
-        const uint32_t c = (g - q_groups) * 8, head = c / part, d = c % part;
+        const uint32_t c = (g - q_groups) * 4, head = c / part, d = c % part;
         if (d < a.dim_pad) {
             turned(x + nq + head * a.dim, d, r);
         } else {
 #pragma unroll
-            for (uint32_t j = 0; j < 8; ++j) {
+            for (uint32_t j = 0; j < 4; ++j) {
                 const uint32_t i = d - a.dim_pad + j, at = head * a.vdim + i;
                 r[j] = i < a.vdim ? x[nq + nk + at] : 0.f;
                 if (i < a.vdim && a.v_mix)
@@ -126,7 +136,7 @@ __global__ void __launch_bounds__(kQkvThreads) k_qkv_prep(QkvPrep a) {
 }
 
 ctox_status launch_qkv_prep(ctox_ctx *ctx, const QkvPrep &a, uint32_t m) {
-    const uint32_t outs = (a.heads * a.dim_pad + a.kv_heads * (a.dim_pad + a.vdim_pad)) / 8;
+    const uint32_t outs = (a.heads * a.dim_pad + a.kv_heads * (a.dim_pad + a.vdim_pad)) / 4;
     uint32_t parts = m <= kDensePass ? (outs + kQkvThreads - 1) / kQkvThreads : 1;
     if (parts > 16) parts = 16;
     const size_t all = (size_t)(a.heads + a.kv_heads) * a.dim + (size_t)a.kv_heads * a.vdim;
