@@ -89,7 +89,10 @@ __device__ void latent_append_row(const LatentAppend &a, uint32_t m, uint32_t ti
 // rows. The activations sit in shared memory in the order the lanes read them: blocks of LPR * 8
 // columns as [half][lane][4]. The first weights of every warp are requested before the dependency
 // wait (they are constants), so they arrive while the prologue forms the input.
-template <int M, int R>
+// IN: how the prologue forms the input (InKind); one kernel each, since every launch reads its code anew.
+enum InKind : int { IN_PLAIN, IN_RMS, IN_LAYER, IN_MERGE };
+
+template <int M, int R, int IN>
 __global__ void __launch_bounds__(kDvThreads, 2)
     k_dense_matvec(const __nv_bfloat16 *__restrict__ W, uint32_t ld, uint32_t rows_per_group, uint32_t units_per_group,
                    uint32_t units, uint32_t ks, uint32_t lpr_log2, uint32_t npos, VecIn in, VecOut out,
@@ -98,7 +101,7 @@ __global__ void __launch_bounds__(kDvThreads, 2)
     extern __shared__ __align__(16) float xs[];  // [M][ldx]
     __shared__ float red[kDvWarps];
     __shared__ float part[kDvWarps][32 * 4];  // partial sums of the column parts: [warp][subgroup rows x positions]
-    __shared__ float mw[M][kAttnSplitsDense];
+    __shared__ float mw[IN == IN_MERGE ? M : 1][kAttnSplitsDense];
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const uint32_t grid = gridDim.x - append_positions;
     if (blockIdx.x >= grid) {
@@ -138,7 +141,7 @@ __global__ void __launch_bounds__(kDvThreads, 2)
     auto stage = [&](uint32_t group) {
         const bool live = pm < npos;
         const uint32_t end = live ? cols : 0;
-        if (in.ws_o) {
+        if constexpr (IN == IN_MERGE) {
             const size_t row = (size_t)pm * in.groups + group;
             if (live) {  // every warp forms the weights of the splits: lane = split and split + 32
                 float mv[kSplitLanes], sv[kSplitLanes], mx = -INFINITY, den = 0.f;
@@ -206,7 +209,7 @@ __global__ void __launch_bounds__(kDvThreads, 2)
                 }
             }
         };
-        if (in.norm == NORM_NONE) {
+        if constexpr (IN == IN_PLAIN) {
             stream(x, nullptr, ldx, [&](uint32_t c, const float4 &v, const float4 &) { slot4(c) = v; });
             return;
         }
@@ -214,7 +217,7 @@ __global__ void __launch_bounds__(kDvThreads, 2)
         auto sq4 = [](const float4 &v) { return (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); };
         const float n = (float)cols;
         float s = 0.f;
-        if (in.norm == NORM_RMS) {
+        if constexpr (IN == IN_RMS) {
             stream(x, in.y ? in.y + (size_t)pm * in.y_stride : nullptr, ldx, [&](uint32_t c, const float4 &xv, const float4 &yv) {
                 float4 v = xv;
                 if (in.y) {
@@ -277,10 +280,10 @@ __global__ void __launch_bounds__(kDvThreads, 2)
         });
     };
     // norm weights are constants: bring their lines in before the wait
-    if (in.w)
+    if constexpr (IN == IN_RMS || IN == IN_LAYER)
         each(cols, [&](uint32_t c) {
             prefetch_l1(in.w + c);
-            if (in.y && in.wb) prefetch_l1(in.wb + c);
+            if (IN == IN_LAYER && in.y && in.wb) prefetch_l1(in.wb + c);
         });
 
     uint32_t staged = 0xffffffffu;
@@ -395,8 +398,8 @@ __global__ void __launch_bounds__(kDvThreads, 2)
 
 namespace {
 
-template <int M, int R>
-ctox_status matvec_launch(ctox_ctx *ctx, const DenseMat &w, uint32_t groups, uint32_t m, const VecIn &in,
+template <int M, int R, int IN>
+ctox_status matvec_kernel(ctox_ctx *ctx, const DenseMat &w, uint32_t groups, uint32_t m, const VecIn &in,
                           const VecOut &out, const LatentAppend *append, uint32_t append_positions, size_t smem,
                           uint32_t ks, uint32_t lpr_log2) {
     static std::mutex mu;
@@ -406,9 +409,9 @@ ctox_status matvec_launch(ctox_ctx *ctx, const DenseMat &w, uint32_t groups, uin
         std::lock_guard<std::mutex> lock(mu);
         auto it = resident.find({ctx->device, smem});
         if (it == resident.end()) {
-            CTOX_CUDA(ctx, cudaFuncSetAttribute(k_dense_matvec<M, R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+            CTOX_CUDA(ctx, cudaFuncSetAttribute(k_dense_matvec<M, R, IN>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                 ctx->max_smem_optin - 8192));
-            CTOX_CUDA(ctx, cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, k_dense_matvec<M, R>, kDvThreads, smem));
+            CTOX_CUDA(ctx, cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, k_dense_matvec<M, R, IN>, kDvThreads, smem));
             if (per_sm < 1) return fail(ctx, CTOX_MEMORY_BUDGET, "dense matvec: %zu bytes of shared memory", smem);
             resident[{ctx->device, smem}] = per_sm;
         } else {
@@ -421,11 +424,19 @@ ctox_status matvec_launch(ctox_ctx *ctx, const DenseMat &w, uint32_t groups, uin
     const uint32_t grid = (units + waves - 1) / waves;
     const LatentAppend ap = append ? *append : LatentAppend{};
     timing_begin(ctx);
-    CTOX_CUDA(ctx, launch_pdl(k_dense_matvec<M, R>, dim3(grid + append_positions), dim3(kDvThreads), smem, ctx->stream,
+    CTOX_CUDA(ctx, launch_pdl(k_dense_matvec<M, R, IN>, dim3(grid + append_positions), dim3(kDvThreads), smem, ctx->stream,
                               (const __nv_bfloat16 *)w.w, w.ld, rows_per_group, units_per_group, units, ks, lpr_log2, m,
                               in, out, ap, append_positions));
     timing_end(ctx, KC_DENSE_MATVEC, 2.0 * w.rows * w.ld, 2.0 * w.rows * w.ld * m);
     return CTOX_OK;
+}
+
+template <int M, int R, typename... Args>
+ctox_status matvec_launch(ctox_ctx *ctx, const DenseMat &w, uint32_t groups, uint32_t m, const VecIn &in, Args... args) {
+    if (in.ws_o) return matvec_kernel<M, R, IN_MERGE>(ctx, w, groups, m, in, args...);
+    if (in.norm == NORM_NONE) return matvec_kernel<M, R, IN_PLAIN>(ctx, w, groups, m, in, args...);
+    if (in.norm == NORM_RMS) return matvec_kernel<M, R, IN_RMS>(ctx, w, groups, m, in, args...);
+    return matvec_kernel<M, R, IN_LAYER>(ctx, w, groups, m, in, args...);
 }
 
 }  // namespace

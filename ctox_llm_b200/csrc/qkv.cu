@@ -20,6 +20,11 @@ __global__ void __launch_bounds__(kQkvThreads) k_qkv_prep(QkvPrep a) {
         sincosf((float)pos * a.freq[i], &s, &c);
         cs_s[i] = make_float2(c, s);
     }
+    // the norms' weights are constants: bring their lines in before the wait
+    for (uint32_t c = tid * 32; c < nq + nk; c += kQkvThreads * 32) {
+        const float *w = c < nq ? a.q_norm : a.k_norm;
+        if (w) asm volatile("prefetch.global.L1 [%0];" ::"l"(w + (c < nq ? c : c - nq)));
+    }
     pdl_wait();
     const float *row = a.fan + (size_t)m * a.fan_stride;
     float sq = 0.f, sk = 0.f;

@@ -24,17 +24,21 @@ __device__ __forceinline__ bool key_visible(uint32_t key, uint32_t pos, uint32_t
 }
 
 // Query rows of one part of the cache: r = position * (heads per part) + head within the part.
+// Without GROUPED there is one part, and r is the row.
+template <bool GROUPED>
 struct PartRows {
     uint32_t share, part, heads, n;
-    __device__ __forceinline__ PartRows(const CacheAttn &a, uint32_t p)
-        : share(a.heads / a.kv_heads), part(p), heads(a.heads), n(a.m * (a.heads / a.kv_heads)) {}
+    __device__ __forceinline__ PartRows(const CacheAttn &a)
+        : share(GROUPED ? a.heads / a.kv_heads : a.heads), part(GROUPED ? blockIdx.z : 0), heads(a.heads), n(a.m * share) {}
     __device__ __forceinline__ uint32_t position(uint32_t r) const { return r / share; }
-    __device__ __forceinline__ uint32_t row(uint32_t r) const { return r / share * heads + part * share + r % share; }
+    __device__ __forceinline__ uint32_t row(uint32_t r) const {
+        return GROUPED ? r / share * heads + part * share + r % share : r;
+    }
 };
 
 // The CTA that delivers the last split of a tile of query rows merges the tile: a warp per row, the splits in
 // their order, the sink as one more term of the denominator.
-__device__ void merge_splits(const CacheAttn &a, const PartRows &pr, uint32_t splits, uint32_t row0, uint32_t tile_rows) {
+__device__ void merge_splits(const CacheAttn &a, const PartRows<true> &pr, uint32_t splits, uint32_t row0, uint32_t tile_rows) {
     __shared__ uint32_t last;
     __threadfence();
     __syncthreads();
@@ -112,12 +116,12 @@ __device__ __forceinline__ float cache_value<__nv_bfloat16>(const __nv_bfloat16 
 
 // CUDA cores, fp32 throughout: eight query rows against 32-token tiles; a warp scores one row (lane =
 // token), then every thread owns J value columns of all eight rows.
-template <typename T, int J>
+template <typename T, int J, bool GROUPED>
 __global__ void __launch_bounds__(kCaThreads) k_cache_attention(CacheAttn a, uint32_t splits) {
     pdl_launch();
     pdl_wait();
     extern __shared__ __align__(16) float sm[];
-    const PartRows pr(a, blockIdx.z);
+    const PartRows<GROUPED> pr(a);
     const uint32_t D = a.key_cols, ldk = a.head_cols + 1, rows = a.m * a.heads;
     float *q_s = sm;                           // [8][D]
     float *k_s = q_s + kCaRowsFma * D;          // [32][head_cols + 1]
@@ -208,7 +212,7 @@ __global__ void __launch_bounds__(kCaThreads) k_cache_attention(CacheAttn a, uin
             const uint32_t c = tid + j * kCaThreads;
             if (c < a.val_cols && row0 + r < pr.n) a.ws_o[((size_t)sp * rows + pr.row(row0 + r)) * a.val_cols + c] = o[r][j];
         }
-    if (a.out) merge_splits(a, pr, splits, row0, kCaRowsFma);
+    if constexpr (GROUPED) merge_splits(a, pr, splits, row0, kCaRowsFma);
 }
 
 // ------------------------------------------------------------------ tensor cores, bf16 cache
@@ -244,12 +248,12 @@ __device__ __forceinline__ void split_bf16(float v, __nv_bfloat16 &hi, __nv_bflo
 __host__ __device__ constexpr int ca_steps(int nt) { return nt <= 2 ? 2 : nt / 2 + 1; }  // 16-value steps of a row per warp
 constexpr uint32_t kCaLdP = kCaTileMma + 8, kCaLdS = kCaTileMma + 4;
 
-template <int NT>
-__global__ void __launch_bounds__(kCaThreads, 1) k_cache_attention_mma(CacheAttn a, uint32_t splits, uint32_t stages) {
+template <int NT, bool GROUPED>
+__global__ void __launch_bounds__(kCaThreads, NT <= 2 ? 2 : 1) k_cache_attention_mma(CacheAttn a, uint32_t splits, uint32_t stages) {
     constexpr int NK = ca_steps(NT), JG = NT < 4 ? NT : 4;
     pdl_launch();
     extern __shared__ __align__(16) uint8_t smraw[];
-    const PartRows pr(a, blockIdx.z);
+    const PartRows<GROUPED> pr(a);
     const uint32_t D = a.key_cols, ld = a.head_cols + 8, rows = a.m * a.heads;
     __nv_bfloat16 *k_s = reinterpret_cast<__nv_bfloat16 *>(smraw);           // [stages][64][ld]
     float *s_s = reinterpret_cast<float *>(k_s + (size_t)stages * kCaTileMma * ld);  // [8 warps][16][kCaLdS]
@@ -441,7 +445,7 @@ __global__ void __launch_bounds__(kCaThreads, 1) k_cache_attention_mma(CacheAttn
                     make_float2(o[j][i * 2], o[j][i * 2 + 1]);
         }
     }
-    if (a.out) merge_splits(a, pr, splits, row0, kCaRowsMma);
+    if constexpr (GROUPED) merge_splits(a, pr, splits, row0, kCaRowsMma);
 }
 
 namespace {
@@ -467,18 +471,29 @@ size_t fma_smem(const CacheAttn &a) {
     return ((size_t)kCaRowsFma * a.key_cols + kCaTileFma * (a.head_cols + 1) + kCaRowsFma * kCaTileFma + kCaRowsFma) * 4;
 }
 
+template <typename T, int J, bool GROUPED>
+ctox_status fma_kernel(ctox_ctx *ctx, const CacheAttn &a, uint32_t splits, uint32_t row_tiles, size_t smem) {
+    CTOX_CUDA(ctx, cudaFuncSetAttribute(k_cache_attention<T, J, GROUPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    CTOX_CUDA(ctx, launch_pdl(k_cache_attention<T, J, GROUPED>, dim3(row_tiles, splits, a.kv_heads), dim3(kCaThreads), smem, ctx->stream, a, splits));
+    return CTOX_OK;
+}
+template <int NT, bool GROUPED>
+ctox_status mma_kernel(ctox_ctx *ctx, const CacheAttn &a, uint32_t splits, uint32_t row_tiles, size_t smem, uint32_t stages) {
+    CTOX_CUDA(ctx, cudaFuncSetAttribute(k_cache_attention_mma<NT, GROUPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    CTOX_CUDA(ctx, launch_pdl(k_cache_attention_mma<NT, GROUPED>, dim3(row_tiles, splits, a.kv_heads), dim3(kCaThreads), smem, ctx->stream, a,
+                              splits, stages));
+    return CTOX_OK;
+}
+
+// A grouped cache is the one whose splits are merged here (out).
 template <typename T, int J>
 ctox_status fma_launch(ctox_ctx *ctx, const CacheAttn &a, uint32_t splits, uint32_t row_tiles, size_t smem) {
-    CTOX_CUDA(ctx, cudaFuncSetAttribute(k_cache_attention<T, J>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    CTOX_CUDA(ctx, launch_pdl(k_cache_attention<T, J>, dim3(row_tiles, splits, a.kv_heads), dim3(kCaThreads), smem, ctx->stream, a, splits));
-    return CTOX_OK;
+    return a.out ? fma_kernel<T, J, true>(ctx, a, splits, row_tiles, smem) : fma_kernel<T, J, false>(ctx, a, splits, row_tiles, smem);
 }
 template <int NT>
 ctox_status mma_launch(ctox_ctx *ctx, const CacheAttn &a, uint32_t splits, uint32_t row_tiles, size_t smem, uint32_t stages) {
-    CTOX_CUDA(ctx, cudaFuncSetAttribute(k_cache_attention_mma<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    CTOX_CUDA(ctx, launch_pdl(k_cache_attention_mma<NT>, dim3(row_tiles, splits, a.kv_heads), dim3(kCaThreads), smem, ctx->stream, a,
-                              splits, stages));
-    return CTOX_OK;
+    return a.out ? mma_kernel<NT, true>(ctx, a, splits, row_tiles, smem, stages)
+                 : mma_kernel<NT, false>(ctx, a, splits, row_tiles, smem, stages);
 }
 
 }  // namespace
@@ -497,7 +512,9 @@ uint32_t cache_attn_splits(const ctox_ctx *ctx, const CacheAttn &a) {
     const uint32_t tile = mma ? kCaTileMma : kCaTileFma, row_tiles = row_tiles_of(a, mma) * a.kv_heads;
     const KeyRange kr = key_range(a.pos0, a.m, a.window);
     const uint32_t tiles = (kr.hi - kr.lo + tile - 1) / tile;
-    uint32_t s = (uint32_t)ctx->sm_count / row_tiles;
+    // a CTA waits at several barriers per tile: two of them on an SM where their buffers fit
+    const bool two = mma && mma_form(a) <= 2 && 2 * (mma_smem(a, mma_stages(ctx, a)) + 1280) <= (size_t)ctx->max_smem_optin + 1024;
+    uint32_t s = (uint32_t)ctx->sm_count * (two ? 2 : 1) / row_tiles;
     // whoever merges the splits reads them all: many only where they shorten a long chain of tiles
     const uint32_t most = tiles >= 256 ? kAttnSplitsDense : kAttnSplitsDense / 2;
     if (s > most) s = most;

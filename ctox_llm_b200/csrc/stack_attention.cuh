@@ -23,7 +23,7 @@ struct CacheAttn {
     uint32_t pos0, m, window;  // window 0: every earlier token
     float scale;
     float *ws_o, *ws_ml;   // [split][row][val_cols], [split][row]{max, sum}
-    float *out;            // [row][val_cols]; null: the splits stay as they are
+    float *out;            // [row][val_cols]; null: the splits stay as they are (one part only)
     const float *sink;     // [heads], may be null (with out only)
     uint32_t *arrived;     // zero on entry and on return, one per tile of query rows (cache_attn_tiles)
 };
