@@ -89,6 +89,14 @@ __device__ void latent_append_row(const LatentAppend &a, uint32_t m, uint32_t ti
 // rows. The activations sit in shared memory in the order the lanes read them: blocks of LPR * 8
 // columns as [half][lane][4]. The first weights of every warp are requested before the dependency
 // wait (they are constants), so they arrive while the prologue forms the input.
+// Weights are read once: their lines stay out of L1. Volatile, so that requests made ahead of the dependency wait stay
+// ahead of it.
+__device__ __forceinline__ uint4 load_weights(const __nv_bfloat16 *p) {
+    uint4 v;
+    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+    return v;
+}
+
 // IN: how the prologue forms the input (InKind); one kernel each, since every launch reads its code anew.
 enum InKind : int { IN_PLAIN, IN_RMS, IN_LAYER, IN_MERGE };
 
@@ -124,7 +132,7 @@ __global__ void __launch_bounds__(kDvThreads, 2)
         for (int r = 0; r < R; ++r) {
             dst[r] = make_uint4(0, 0, 0, 0);
             if (i < cnt && c < ld && row0 + r < rows_per_group)
-                dst[r] = __ldg(reinterpret_cast<const uint4 *>(base + (size_t)(row0 + r) * ld + c));
+                dst[r] = load_weights(base + (size_t)(row0 + r) * ld + c);
         }
     };
     // ---- the input of `group`, normalised, into xs. Loads are issued in batches of kBatch vectors before
@@ -411,6 +419,9 @@ ctox_status matvec_kernel(ctox_ctx *ctx, const DenseMat &w, uint32_t groups, uin
         if (it == resident.end()) {
             CTOX_CUDA(ctx, cudaFuncSetAttribute(k_dense_matvec<M, R, IN>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                 ctx->max_smem_optin - 8192));
+            // One split of the SM's memory into L1 and shared for all of them: kernels that ask for different ones
+            // do not overlap on an SM.
+            CTOX_CUDA(ctx, cudaFuncSetAttribute(k_dense_matvec<M, R, IN>, cudaFuncAttributePreferredSharedMemoryCarveout, 75));
             CTOX_CUDA(ctx, cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, k_dense_matvec<M, R, IN>, kDvThreads, smem));
             if (per_sm < 1) return fail(ctx, CTOX_MEMORY_BUDGET, "dense matvec: %zu bytes of shared memory", smem);
             resident[{ctx->device, smem}] = per_sm;
