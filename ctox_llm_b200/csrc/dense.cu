@@ -621,8 +621,10 @@ ctox_status launch_latent_split(ctox_ctx *ctx, const float *fan, uint32_t fan_st
                                 const float *q_norm, float eps, __nv_bfloat16 *cq, uint32_t cq_ld,
                                 const LatentAppend *append, uint32_t m) {
     const LatentAppend ap = append ? *append : LatentAppend{};
+    timing_begin(ctx);
     CTOX_CUDA(ctx, launch_pdl(k_latent_split, dim3(m), dim3(kSnThreads), 0, ctx->stream, fan, fan_stride, q_rank, q_norm,
                               eps, cq, cq_ld, ap, (int)(append != nullptr)));
+    timing_end(ctx, KC_QKV, (double)m * (fan_stride * 4.0 + q_rank * 2.0 + (ap.kv_pad + ap.rot_pad) * 2.0), 0);
     return CTOX_OK;
 }
 
